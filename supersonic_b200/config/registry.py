@@ -19,6 +19,7 @@ from .sotavik import ARCHITECTURE as _SOTAVIK, SotavikConfig
 from .ronelorn import ARCHITECTURE as _RONELORN, RonelornConfig
 from .vufadra import ARCHITECTURE as _VUFADRA, VufadraConfig
 from .kilisun import ARCHITECTURE as _KILISUN, KilisunConfig
+from .ruzunex import ARCHITECTURE as _RUZUNEX, RuzunexConfig
 
 _ARCHITECTURES: Dict[str, Type] = {}
 
@@ -72,6 +73,7 @@ register_architecture(_SOTAVIK, SotavikConfig)
 register_architecture(_VUFADRA, VufadraConfig)
 register_architecture(_RONELORN, RonelornConfig)
 register_architecture(_KILISUN, KilisunConfig)
+register_architecture(_RUZUNEX, RuzunexConfig)
 
 
 _PRESET_DIR = os.path.join(os.path.dirname(os.path.abspath(__file__)), "presets")

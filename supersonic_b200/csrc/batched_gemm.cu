@@ -206,7 +206,7 @@ SSB_API int ssb_grouped_gemm_mma(const void* A, int lda, const int* a_index, int
     // n_rows: the rows of all groups together (what the host knows of their sizes); gate_kind, gate_limit: the
     // gated unit's inner step in mode 1 (0: silu(g) u)
     if (max_tiles <= 0 || N <= 0) return 0;
-    if (a_div <= 0 || gate_kind < 0 || gate_kind > SSB_GATE_CLAMPED_SWISH) return SSB_ERR_BAD_SIZE;
+    if (a_div <= 0 || gate_kind < 0 || gate_kind > SSB_GATE_LAST) return SSB_ERR_BAD_SIZE;
     BgArgs a = {};
     a.A = (const bf16*)A; a.lda = lda; a.a_batch = 0; a.a_index = a_index; a.a_div = a_div;
     a.W = (const bf16*)W; a.ldw = ldw; a.w_batch = w_expert;

@@ -52,6 +52,7 @@ LIBRARIES: Dict[str, Dict[str, List[str]]] = {
     "window_attention": {"sources": ["window_attention.cu"], "flags": [], "link": []},
     "window_attention_mma": {"sources": ["window_attention_mma.cu"], "flags": [], "link": []},
     "mingru_ops": {"sources": ["mingru_ops.cu"], "flags": [], "link": []},
+    "stream_ops": {"sources": ["stream_ops.cu"], "flags": [], "link": []},
     "random_fill": {"sources": ["random_fill.cu"], "flags": [], "link": []},
     # the host side's native core: no CUDA in it, so it is compiled by the C++ compiler alone
     "host_runtime": {"sources": ["runtime.cpp"], "flags": [], "link": [], "dir": os.path.join(os.path.dirname(_HERE), "host"),

@@ -44,10 +44,12 @@ __device__ __forceinline__ float ssb_activate(float u, int kind) {
 
 // A gated unit's inner step between its two products, in float32: what becomes of a gate value g and an up value u.
 //   kind 0: silu(g) * u;
-//   kind 1: with g' = min(g, limit) and u' = clamp(u, -limit, limit):  g' * sigmoid(1.702 g') * (u' + 1)
-enum { SSB_GATE_SILU = 0, SSB_GATE_CLAMPED_SWISH = 1 };
+//   kind 1: with g' = min(g, limit) and u' = clamp(u, -limit, limit):  g' * sigmoid(1.702 g') * (u' + 1);
+//   kind 2: gelu(g) * u, the form of gelu with tanh (see ssb_activate)
+enum { SSB_GATE_SILU = 0, SSB_GATE_CLAMPED_SWISH = 1, SSB_GATE_GELU_TANH = 2, SSB_GATE_LAST = SSB_GATE_GELU_TANH };
 __device__ __forceinline__ float ssb_gate(float g, float u, int kind, float limit) {
     if (kind == SSB_GATE_SILU) return g / (1.0f + expf(-g)) * u;
+    if (kind == SSB_GATE_GELU_TANH) return ssb_activate(g, SSB_ACT_GELU_TANH) * u;
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
@@ -56,6 +58,9 @@ __device__ __forceinline__ float ssb_gate(float g, float u, int kind, float limi
 // The same where a product finishes its float32 sums (fast exponential: the result is rounded to bfloat16 next).
 __device__ __forceinline__ float ssb_gate_fast(float g, float u, int kind, float limit) {
     if (kind == SSB_GATE_SILU) return __fdividef(g, 1.0f + __expf(-g)) * u;
+    // (1 + tanh(y)) / 2 = 1 / (1 + exp(-2 y))
+    if (kind == SSB_GATE_GELU_TANH)
+        return __fdividef(g, 1.0f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u;
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);

@@ -142,6 +142,83 @@ SSB_API int ssb_route_sigmoid_groups(const float* z, int ld, const float* correc
 }
 
 // ---------------------------------------------------------------------------------------
+// softmax router.  s = softmax(z) over all experts (float32); the `top` experts with the largest scores win, the lower
+// index at equal scores; an expert's weight is its s times `scale`, with `renormalize` divided by the sum of the
+// chosen scores (+ 1e-20).  One warp per token, lanes over experts.
+// ---------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(RG_THREADS)
+route_softmax_kernel(const float* __restrict__ z, int ld, int n_tokens, int n_experts, int top, int renormalize, float scale,
+                     int* __restrict__ expert_of, float* __restrict__ pair_weight) {
+    extern __shared__ float rs_smem[];                   // per warp: [n_experts] scores, [top] chosen scores
+    ssb_pdl_launch_dependents();
+    ssb_pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.x * (RG_THREADS / 32) + warp;
+    if (t >= n_tokens) return;
+    float* s_s = rs_smem + (size_t)warp * (n_experts + top);
+    float* w_s = s_s + n_experts;
+    const float* zr = z + (size_t)t * ld;
+    float m = -INFINITY;
+    for (int e = lane; e < n_experts; e += 32) m = fmaxf(m, zr[e]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+    float sum = 0.f;
+    for (int e = lane; e < n_experts; e += 32) {
+        const float p = expf(zr[e] - m);
+        s_s[e] = p;
+        sum += p;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    const float inv = 1.0f / sum;
+    for (int e = lane; e < n_experts; e += 32) s_s[e] *= inv;
+    __syncwarp();
+    float chosen = 0.f;
+    for (int k = 0; k < top; ++k) {
+        float bv = -1.0f;                                 // below every score; a taken expert's mark is lower still
+        int best = 0x7fffffff;
+        for (int e = lane; e < n_experts; e += 32) {
+            const float v = s_s[e];
+            if (v > bv) { bv = v; best = e; }             // rising e: the lower index stays at equal scores
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+            const int oe = __shfl_xor_sync(0xffffffffu, best, o);
+            if (ov > bv || (ov == bv && oe < best)) { bv = ov; best = oe; }
+        }
+        if (best == 0x7fffffff) {                         // only where scores are not numbers: some expert in range, weight 0
+            best = k;
+            bv = 0.f;
+        }
+        chosen += bv;
+        if (lane == 0) {
+            expert_of[(size_t)t * top + k] = best;
+            w_s[k] = bv;
+            s_s[best] = -2.0f;                            // taken
+        }
+        __syncwarp();
+    }
+    const float f = renormalize ? scale / (chosen + 1e-20f) : scale;
+    for (int k = lane; k < top; k += 32) pair_weight[(size_t)t * top + k] = w_s[k] * f;
+}
+
+SSB_API int ssb_route_softmax(const float* z, int ld, int n_tokens, int n_experts, int top, int renormalize, float scale,
+                              int* expert_of, float* pair_weight, int pdl, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (n_experts <= 0 || top < 1 || top > n_experts || n_experts > 2048 || ld < n_experts) return SSB_ERR_BAD_SIZE;
+    const size_t smem = (size_t)(RG_THREADS / 32) * (n_experts + top) * sizeof(float);
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(route_softmax_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
+    const int rc = ssb_launch(route_softmax_kernel, dim3((n_tokens + RG_THREADS / 32 - 1) / (RG_THREADS / 32)),
+                              dim3(RG_THREADS), smem, stream, pdl != 0, z, ld, n_tokens, n_experts, top, renormalize, scale,
+                              expert_of, pair_weight);
+    return rc ? rc : ssb_launch_status();
+}
+
+// ---------------------------------------------------------------------------------------
 // pairs sorted by expert.  One block: counts in shared memory, offsets and the tile list by one
 // thread, then every pair takes the next free row of its expert.  The order inside a group is
 // whatever the adds give; nothing downstream depends on it.

@@ -417,12 +417,14 @@ class FastKernels(PlainKernels):
                                       chunk, window, scale)
 
     def window_attention(self, q, kv, pooled_kv, batch, out, n_q, n_kv, dim, vdim, page_shift, window, keep_first, pool,
-                         scale, softcap, sinks, value_position, out_scale=1.0, v_share=1, gate=None):
+                         scale, softcap, sinks, value_position, out_scale=1.0, v_share=1, gate=None, gate_elems=False,
+                         slopes=None, head_mul=None):
         k_cache, v_cache, table, _ = kv
         pooled = None if pooled_kv is None else pooled_kv[:3]
         if not ops.window_attention_mma_ok(q, k_cache, v_cache, pooled, out, dim, vdim, page_shift):
             super().window_attention(q, kv, pooled_kv, batch, out, n_q, n_kv, dim, vdim, page_shift, window, keep_first,
-                                     pool, scale, softcap, sinks, value_position, out_scale, v_share, gate)
+                                     pool, scale, softcap, sinks, value_position, out_scale, v_share, gate, gate_elems,
+                                     slopes, head_mul)
             return
         vcos = vsin = None
         v_inter = False
@@ -432,7 +434,7 @@ class FastKernels(PlainKernels):
         ops.window_attention_mma(q, k_cache, v_cache, table, pooled, batch.cu_new, batch.seq_start, batch.seq_slot, out,
                                  batch.max_new, n_q, n_kv, dim, vdim, page_shift, window, keep_first, pool, scale, softcap,
                                  sinks, vcos, vsin, v_inter, out_scale, pdl=self._chain(batch.n_tokens), v_share=v_share,
-                                 gate=gate)
+                                 gate=gate, gate_elems=gate_elems, slopes=slopes, head_mul=head_mul)
 
     def gated_linear_scan(self, proj, q_off, k_off, v_off, z, z_bias, tau, q_scale, state, batch, out, n_heads,
                           dim, vdim):

@@ -617,7 +617,7 @@ SSB_API int ssb_gemm_tc_act(const void* A, int lda, const void* W, int ldw, void
 SSB_API int ssb_gemm_tc_gate(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K,
                              int gate_kind, float gate_limit, const float* row_scale, int tile_n, int* error_word,
                              cudaStream_t stream) {
-    if (gate_kind < 0 || gate_kind > SSB_GATE_CLAMPED_SWISH) return SSB_ERR_BAD_SIZE;
+    if (gate_kind < 0 || gate_kind > SSB_GATE_LAST) return SSB_ERR_BAD_SIZE;
     TcRope extra{};
     extra.gate_kind = gate_kind; extra.gate_limit = gate_limit; extra.row_scale = row_scale;
     return gemm_tc_any(A, lda, W, ldw, C, ldc, SSB_BF16, M, N, K, TC_SWIGLU, tile_n, 1, error_word, extra, stream);

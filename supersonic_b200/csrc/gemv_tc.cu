@@ -317,7 +317,7 @@ SSB_API int ssb_gemv_tc(const void* x, int ldx, const void* W, int ldw, void* ou
 SSB_API int ssb_gemv_tc_gate(const void* x, int ldx, const void* W, int ldw, void* out, int ldo, int n_rows, int N, int K,
                              int gate_kind, float gate_limit, const float* row_scale, int* error_word, int pdl,
                              cudaStream_t stream) {
-    if (gate_kind < 0 || gate_kind > SSB_GATE_CLAMPED_SWISH) return SSB_ERR_BAD_SIZE;
+    if (gate_kind < 0 || gate_kind > SSB_GATE_LAST) return SSB_ERR_BAD_SIZE;
     return gemv_tc_any(x, ldx, W, ldw, out, ldo, SSB_BF16, n_rows, N, K, TC_SWIGLU, 1, nullptr, nullptr, error_word, pdl,
                        stream, gate_kind, gate_limit, row_scale);
 }

@@ -95,6 +95,29 @@ class PlainKernels:
         ops.rms_add(residual, branch, weight, eps, clear, None if next_norm is None else next_norm.weight_f32,
                     0.0 if next_norm is None else next_norm.eps, next_out, pdl=self._chain(residual.shape[0]))
 
+    def stream_enter(self, src, streams, in_weights, branch, write, dst, norm, conv, tail, batch, out):
+        """A sublayer's entry over several residual streams: the write of the sublayer before (``write`` = (mix,
+        out_weights) with its ``branch``, or None), the next read, its RMS norm and the short convolution behind it
+        (``conv`` [width, taps] float32, ``tail`` its per-slot rows), into ``out``."""
+        mix, out_w = write if write is not None else (None, None)
+        if write is None:
+            branch = dst = None
+        pdl = self._chain(batch.n_tokens)
+        if batch.is_decode:                    # one token a sequence: the convolution reads its kept rows alone
+            ops.stream_cross(src, streams, in_weights, out, branch, mix, out_w, dst, True, norm.weight_f32, norm.eps, conv,
+                             tail, batch.slot_of_token, pdl=pdl)
+            return
+        normed = torch.empty_like(out)
+        ops.stream_cross(src, streams, in_weights, normed, branch, mix, out_w, dst, True, norm.weight_f32, norm.eps, pdl=pdl)
+        ops.causal_conv(normed, None, conv, None, tail if conv.shape[1] > 1 else conv[:1, :0], batch.cu_new, batch.seq_slot,
+                        out, batch.max_new, pdl=pdl)
+
+    def stream_sum(self, src, streams, branch, write, out, clear=True):
+        """The sum of the streams with the last write applied (``clear``: the branch is zeroed behind the read)."""
+        mix, out_w = write if write is not None else (None, None)
+        ops.stream_cross(src, streams, None, out, branch if write is not None else None, mix, out_w, None, clear,
+                         pdl=self._chain(out.shape[0]))
+
     def project_rope_append(self, x, w_qkv, qkv, position, kv, batch, n_q, n_kv, head_dim, page_shift) -> bool:
         """The q/k/v projection with position encoding and cache append in one kernel: rotated q
         into ``qkv``'s first columns, k and v into the cache.  False: not taken, nothing was done."""
@@ -162,6 +185,22 @@ class PlainKernels:
         float32 path's scan); unit keys and removal vectors into ``unit`` (see ``ops.state_scan_prepare``)."""
         ops.state_scan_prepare(z, z_bias, decay_kind, decay_scale, n_heads, dim, proj, k_off, a_off, a_bias, unit_eps,
                                unit, log_decay=log_decay, pdl=self._chain(z.shape[0]))
+
+    def tied_scan(self, proj, q_off, f_off, v_off, z_bias, lower, state, batch, norm_w, eps, y, n_heads, dim, vdim):
+        """The recurrence whose forget gate also says what is written, with the head norm behind it, into ``y``."""
+        if batch.is_decode and vdim <= ops.TIED_STEP_MAX_VDIM:
+            ops.tied_step(proj, q_off, f_off, v_off, z_bias, lower, state, batch.cu_new, batch.seq_slot, norm_w, eps, y,
+                          n_heads, dim, vdim, pdl=self._chain(batch.n_tokens))
+            return
+        chunk, n_sums, n_decays = ops.scan_chunking(batch.n_seqs, batch.max_new, n_heads, dim, vdim)
+        sums = decays = None
+        if chunk:                             # a long prompt: its chunks in parallel
+            scratch = self._scan_scratch(n_sums + n_decays, y.device)
+            sums, decays = scratch[:n_sums], scratch[n_sums: n_sums + n_decays]
+        o = torch.empty((batch.n_tokens, n_heads * vdim), dtype=torch.float32, device=y.device)
+        ops.tied_scan(proj, q_off, f_off, v_off, z_bias, lower, state, batch.cu_new, batch.seq_slot, o, n_heads, dim, vdim,
+                      pdl=self._chain(batch.n_tokens), chunk=chunk, max_new=batch.max_new, sums=sums, decays=decays)
+        ops.head_norm_gate(o, norm_w, eps, None, y, n_heads, vdim, pdl=self._chain(batch.n_tokens))
 
     def matrix_state_scan(self, proj, r_off, k_off, v_off, decay, kind, state, batch, out, n_heads, dim, vdim,
                           unit=None, bonus=None):
@@ -247,7 +286,8 @@ class PlainKernels:
         self.activation(u, out, kind, scale)
 
     def qkv_prepare(self, qkv, q_weight, k_weight, norm, eps, position, value_position, kv, batch, n_q, n_kv, dim, vdim,
-                    page_shift, write_cache=True, pooled_kv=None, pool=0, v_off=None, q_temp=None, n_v=None) -> bool:
+                    page_shift, write_cache=True, pooled_kv=None, pool=0, v_off=None, q_temp=None, n_v=None,
+                    v_mix=None) -> bool:
         """Norm of q and k (``norm`` ``"head"``, ``"row"`` or None), rotation of their first coordinates by
         ``position``, of the values over their whole width by ``value_position`` (either may be None), k and v into
         the cache.  With a pooled store and a step of one token a sequence, the tokens that end a run of ``pool``
@@ -267,7 +307,7 @@ class PlainKernels:
         ops.qkv_prepare(qkv, q_weight, k_weight, norm, eps, cos, sin, rot_dims, inter, vcos, vsin, v_inter, batch.pos,
                         batch.slot_of_token, table, k_cache, v_cache, n_q, n_kv, dim, vdim, page_shift, write_cache,
                         pdl=self._chain(batch.n_tokens), pooled=pooled_kv[:3] if pools else None, pool=pool if pools else 0,
-                        v_off=v_off, q_temp=q_temp, n_v=n_v)
+                        v_off=v_off, q_temp=q_temp, n_v=n_v, v_mix=v_mix)
         return pools
 
     def pool_rows(self, kv, pooled_kv, batch, n_kv, dim, vdim, page_shift, pool):
@@ -278,7 +318,8 @@ class PlainKernels:
                       batch.max_new, n_kv, dim, vdim, page_shift, pool, pdl=self._chain(batch.n_tokens))
 
     def window_attention(self, q, kv, pooled_kv, batch, out, n_q, n_kv, dim, vdim, page_shift, window, keep_first, pool,
-                         scale, softcap, sinks, value_position, out_scale=1.0, v_share=1, gate=None):
+                         scale, softcap, sinks, value_position, out_scale=1.0, v_share=1, gate=None, gate_elems=False,
+                         slopes=None, head_mul=None):
         vcos = vsin = None
         v_inter = False
         if value_position is not None:
@@ -288,7 +329,8 @@ class PlainKernels:
         pooled = None if pooled_kv is None else pooled_kv[:3]
         ops.window_attention_plain(q, k_cache, v_cache, table, pooled, batch.pos, batch.slot_of_token, out, n_q, n_kv,
                                    dim, vdim, page_shift, window, keep_first, pool, scale, softcap, sinks, vcos, vsin,
-                                   v_inter, out_scale, pdl=self._chain(batch.n_tokens), v_share=v_share, gate=gate)
+                                   v_inter, out_scale, pdl=self._chain(batch.n_tokens), v_share=v_share, gate=gate,
+                                   gate_elems=gate_elems, slopes=slopes, head_mul=head_mul)
 
     def map_difference(self, maps, out, n_heads, n_kv, vdim, lam, eps, mult):
         ops.map_difference(maps, out, n_heads, n_kv, vdim, lam, eps, mult, pdl=self._chain(maps.shape[0]))
@@ -311,6 +353,9 @@ class PlainKernels:
                              extra_col=None, extra_out=None):
         ops.route_sigmoid_groups(logits, n_experts, correction, n_groups, keep, scale, expert_of, pair_weight, extra_col,
                                  extra_out, pdl=self._chain(logits.shape[0]))
+
+    def route_softmax(self, logits, n_experts, renormalize, scale, expert_of, pair_weight):
+        ops.route_softmax(logits, n_experts, renormalize, scale, expert_of, pair_weight, pdl=self._chain(logits.shape[0]))
 
     def group_by_expert(self, expert_of, n_experts, groups):
         """``groups``: the dict of int32 tensors a grouped product reads (offsets, order, tile_expert,

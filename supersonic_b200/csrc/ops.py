@@ -225,14 +225,14 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False) 
         _stream()), "swiglu")
 
 
-GATE_KINDS_FF = {"silu": 0, "clamped_swish": 1}
+GATE_KINDS_FF = {"silu": 0, "clamped_swish": 1, "gelu_tanh": 2}
 
 
 def gated_activation(gate_up: torch.Tensor, out: torch.Tensor, kind: str = "silu", limit: float = 0.0,
                      interleaved: bool = False, row_scale: Optional[torch.Tensor] = None, pdl: bool = False) -> None:
     """out[t, c] = f(gate[t, c], up[t, c]) * row_scale[t] in float32 arithmetic.  ``kind`` ``"silu"``: silu(g) u;
-    ``"clamped_swish"``: with g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(1.702 g') (u' + 1).  Gate and up
-    are the halves of a row of ``gate_up``, or (interleaved) alternate as [8 gate | 8 up] per 16 columns."""
+    ``"clamped_swish"``: with g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(1.702 g') (u' + 1);
+    ``"gelu_tanh"``: gelu(g) u, gelu in the form with tanh.  Gate and up are the halves of a row of ``gate_up``, or (interleaved) alternate as [8 gate | 8 up] per 16 columns."""
     _need(gate_up, "gate_up", None, 2); _need(out, "out", gate_up.dtype, 2)
     if kind not in GATE_KINDS_FF:
         raise KernelError(f"gated_activation: kind {kind!r} is not known (known: {sorted(GATE_KINDS_FF)})")
@@ -497,6 +497,120 @@ def gated_linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, z:
         "gated_linear_scan")
 
 
+TIED_STEP_MAX_VDIM = 256
+
+
+def _tied_args(proj, q_off, f_off, v_off, z_bias, lower, state, cu_new, seq_slot, n_heads, dim, vdim, what):
+    _need(proj, "proj", None, 2); _need(z_bias, "z_bias", torch.float32, 1); _need(lower, "lower", torch.float32, 1)
+    _need(state, "state", torch.float32, 2); _need(cu_new, "cu_new", torch.int32, 1); _need(seq_slot, "seq_slot", torch.int32, 1)
+    if z_bias.shape[0] != n_heads * dim or lower.shape[0] != n_heads * dim or cu_new.shape[0] != seq_slot.shape[0] + 1 \
+            or max(q_off, f_off) + n_heads * dim > proj.shape[1] or v_off + n_heads * vdim > proj.shape[1] \
+            or state.shape[1] != n_heads * dim * vdim or not state.is_contiguous() or dim > SCAN_MAX_DIM:
+        raise KernelError(f"{what}: sizes (state rows of heads x dim x vdim, dim up to {SCAN_MAX_DIM})")
+
+
+def tied_scan(proj: torch.Tensor, q_off: int, f_off: int, v_off: int, z_bias: torch.Tensor, lower: torch.Tensor,
+              state: torch.Tensor, cu_new: torch.Tensor, seq_slot: torch.Tensor, out: torch.Tensor, n_heads: int, dim: int,
+              vdim: int, pdl: bool = False, chunk: int = 0, max_new: int = 0, sums: Optional[torch.Tensor] = None,
+              decays: Optional[torch.Tensor] = None) -> None:
+    """Per sequence and head, over the sequence's new tokens in order, with the gate f = lower + (1 - lower) *
+    sigmoid(z + z_bias) per head and channel:  S = diag(f) S + (1 - f) v^T;  out = S^T silu(q).  q and z (heads x dim)
+    and v (heads x vdim) are columns of ``proj``; ``state``, ``chunk``, ``sums`` and ``decays`` as in ``gated_linear_scan``."""
+    _tied_args(proj, q_off, f_off, v_off, z_bias, lower, state, cu_new, seq_slot, n_heads, dim, vdim, "tied_scan")
+    _need(out, "out", torch.float32, 2)
+    T, B = proj.shape[0], seq_slot.shape[0]
+    if out.shape[0] != T or out.shape[1] < n_heads * vdim:
+        raise KernelError("tied_scan: one output row per token")
+    max_chunks = 0
+    if chunk > 0:
+        max_chunks = -(-max_new // chunk)
+        _need(sums, "sums", torch.float32); _need(decays, "decays", torch.float32)
+        if max_chunks < 1 or sums.numel() < B * max_chunks * n_heads * dim * vdim \
+                or decays.numel() < B * max_chunks * n_heads * dim:
+            raise KernelError("tied_scan: the scratch of the chunked run is too small")
+    _check(_fn("recurrence_ops", "ssb_tied_scan")(
+        _ptr(proj), c_int(proj.stride(0)), c_int(dtype_code(proj.dtype)), c_int(q_off), c_int(f_off), c_int(v_off),
+        _ptr(z_bias), _ptr(lower), _ptr(state), _ptr(cu_new), _ptr(seq_slot), _ptr(out), c_int(out.stride(0)), c_int(B),
+        c_int(T), c_int(n_heads), c_int(dim), c_int(vdim), c_int(chunk), c_int(max_chunks), _ptr(sums), _ptr(decays),
+        c_int(1 if pdl else 0), _stream()), "tied_scan")
+
+
+def tied_step(proj: torch.Tensor, q_off: int, f_off: int, v_off: int, z_bias: torch.Tensor, lower: torch.Tensor,
+              state: torch.Tensor, cu_new: torch.Tensor, seq_slot: torch.Tensor, weight: torch.Tensor, eps: float,
+              out: torch.Tensor, n_heads: int, dim: int, vdim: int, pdl: bool = False) -> None:
+    """``tied_scan`` for steps of one token a sequence, with the head norm behind it: out = o / rms(o) * weight per head
+    (``weight`` [vdim] float32, for all heads)."""
+    _tied_args(proj, q_off, f_off, v_off, z_bias, lower, state, cu_new, seq_slot, n_heads, dim, vdim, "tied_step")
+    _need(out, "out", proj.dtype, 2); _need(weight, "weight", torch.float32, 1)
+    B = seq_slot.shape[0]
+    if proj.shape[0] != B or out.shape[0] != B or out.shape[1] < n_heads * vdim or weight.shape[0] != vdim \
+            or vdim > TIED_STEP_MAX_VDIM:
+        raise KernelError(f"tied_step: one row per sequence, heads of up to {TIED_STEP_MAX_VDIM} values")
+    _check(_fn("recurrence_ops", "ssb_tied_step")(
+        _ptr(proj), c_int(proj.stride(0)), c_int(dtype_code(proj.dtype)), c_int(q_off), c_int(f_off), c_int(v_off),
+        _ptr(z_bias), _ptr(lower), _ptr(state), _ptr(cu_new), _ptr(seq_slot), _ptr(weight), c_float(eps), _ptr(out),
+        c_int(out.stride(0)), c_int(B), c_int(n_heads), c_int(dim), c_int(vdim), c_int(1 if pdl else 0), _stream()), "tied_step")
+
+
+STREAMS_MAX = 16
+
+
+def stream_cross(src: torch.Tensor, streams: int, in_weights: Optional[torch.Tensor], out: torch.Tensor,
+                 branch: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
+                 out_weights: Optional[torch.Tensor] = None, dst: Optional[torch.Tensor] = None, clear: bool = False,
+                 norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0, conv: Optional[torch.Tensor] = None,
+                 tail: Optional[torch.Tensor] = None, slot: Optional[torch.Tensor] = None, pdl: bool = False) -> None:
+    """One pass over S residual streams ``src`` [S or 1, tokens, width] float32 (1: the one row that all streams equal).
+    With a ``branch`` y [tokens, width] the streams become x_t = sum_s mix[s, t] x_s + out_weights[t] y, all at once from
+    the old ones, stored into ``dst`` (``src`` itself, another tensor, or None: not stored), and ``clear`` zeroes the
+    branch behind the read.  Then u = sum_t in_weights[t] x_t (None: their sum); ``out`` gets u (float32) or, with
+    ``norm_weight``, u / sqrt(mean(u^2) + eps) * norm_weight.  With ``conv`` [width, taps] (one token a sequence only) the
+    normed row n passes a causal convolution, out = sum_j conv[:, j] n_(t - taps + 1 + j), whose earlier rows are
+    ``tail[slot]`` ([taps - 1, width], oldest first), brought up to date."""
+    _need(src, "src", torch.float32, 3); _need(out, "out", None, 2)
+    n_src, T, W = src.shape
+    if not 1 <= streams <= STREAMS_MAX or n_src not in (1, streams) or tuple(out.shape) != (T, W) \
+            or not (src.is_contiguous() and out.is_contiguous()):
+        raise KernelError(f"stream_cross: src [streams or 1, tokens, width] of up to {STREAMS_MAX} streams, out [tokens, width]")
+    if in_weights is not None:
+        _need(in_weights, "in_weights", torch.float32, 1)
+        if in_weights.shape[0] != streams:
+            raise KernelError("stream_cross: one reading weight per stream")
+    if branch is not None:
+        _need(branch, "branch", torch.float32, 2); _need(mix, "mix", torch.float32, 2)
+        _need(out_weights, "out_weights", torch.float32, 1)
+        if tuple(branch.shape) != (T, W) or not branch.is_contiguous() or tuple(mix.shape) != (streams, streams) \
+                or not mix.is_contiguous() or out_weights.shape[0] != streams:
+            raise KernelError("stream_cross: branch [tokens, width], mix [streams, streams], one writing weight per stream")
+        if dst is not None:
+            _need(dst, "dst", torch.float32, 3)
+            if tuple(dst.shape) != (streams, T, W) or not dst.is_contiguous():
+                raise KernelError("stream_cross: dst [streams, tokens, width], contiguous")
+    elif dst is not None:
+        raise KernelError("stream_cross: without a branch the streams stay as they are")
+    if norm_weight is not None:
+        _need(norm_weight, "norm_weight", torch.float32, 1)
+        if norm_weight.shape[0] != W:
+            raise KernelError("stream_cross: a norm weight per column")
+    elif out.dtype != torch.float32 or conv is not None:
+        raise KernelError("stream_cross: without a norm the result is float32, and no convolution stands behind it")
+    taps = 0
+    if conv is not None:
+        _need(conv, "conv", torch.float32, 2); _need(slot, "slot", torch.int32, 1)
+        taps = conv.shape[1]
+        if conv.shape[0] != W or not conv.is_contiguous() or not 1 <= taps <= CONV_MAX_TAPS or slot.shape[0] != T:
+            raise KernelError(f"stream_cross: conv [width, taps] of up to {CONV_MAX_TAPS} taps, one slot per token")
+        if taps > 1:
+            _need(tail, "tail", torch.float32, 2)
+            if tail.shape[1] != (taps - 1) * W or not tail.is_contiguous():
+                raise KernelError("stream_cross: tail rows of (taps - 1) x width")
+    _check(_fn("stream_ops", "ssb_stream_cross")(
+        _ptr(src), c_int(n_src), c_longlong(T * W), _ptr(branch), c_int(1 if clear else 0), _ptr(mix if branch is not None else None),
+        _ptr(out_weights if branch is not None else None), _ptr(dst), _ptr(in_weights), _ptr(norm_weight), c_float(eps),
+        _ptr(out), c_int(dtype_code(out.dtype)), _ptr(conv), _ptr(tail if taps > 1 else None), _ptr(slot if conv is not None else None),
+        c_int(taps), c_int(T), c_int(W), c_int(streams), c_int(1 if pdl else 0), _stream()), "stream_cross")
+
+
 SCAN_CHUNK = 128                 # tokens of a chunk when a long prompt's recurrence runs chunk-parallel (2,048 tokens of
                                  # 4 heads x 256 x 512: 1.18 ms in chunks of 64, 1.00 ms in chunks of 128, 4.4 ms in one go)
 SCAN_CHUNK_MIN_NEW = 256         # shorter runs of new tokens are walked in one go
@@ -517,21 +631,24 @@ def scan_chunking(n_seqs: int, max_new: int, n_heads: int, dim: int, vdim: int):
     return chunk, n_seqs * n * per, n_seqs * n * n_heads * dim
 
 
-def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate: torch.Tensor, out: torch.Tensor,
+def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate: Optional[torch.Tensor], out: torch.Tensor,
                    n_heads: int, vdim: int, pdl: bool = False, gate_kind: str = "silu") -> None:
     """out[t, h] = o[t, h] / sqrt(mean(o[t, h]^2) + eps) * weight * act(gate[t, h]): every head's ``vdim``
     outputs normalised on their own, weighted (``weight`` [vdim]: one vector for all heads; [heads x vdim]: one
-    per head), then gated; ``gate_kind``: ``"silu"``, ``"sigmoid"`` or ``"none"`` (the gate as given).  ``o`` float32."""
-    _need(o, "o", torch.float32, 2); _need(weight, "weight", None, 1); _need(gate, "gate", None, 2)
-    _need(out, "out", gate.dtype, 2)
+    per head), then gated; ``gate_kind``: ``"silu"``, ``"sigmoid"`` or ``"none"`` (the gate as given); ``gate`` None: the product ends at the weight.  ``o`` float32."""
+    _need(o, "o", torch.float32, 2); _need(weight, "weight", None, 1); _need(out, "out", None, 2)
     T = o.shape[0]
-    if gate.shape[0] != T or out.shape[0] != T or min(o.shape[1], gate.shape[1], out.shape[1]) < n_heads * vdim \
+    if gate is not None:
+        _need(gate, "gate", out.dtype, 2)
+        if gate.shape[0] != T or gate.shape[1] < n_heads * vdim:
+            raise KernelError("head_norm_gate: one gate row per token")
+    if out.shape[0] != T or min(o.shape[1], out.shape[1]) < n_heads * vdim \
             or weight.shape[0] not in (vdim, n_heads * vdim) or not weight.is_contiguous():
         raise KernelError("head_norm_gate: sizes")
     w_stride = vdim if weight.shape[0] == n_heads * vdim and n_heads > 1 else 0
     _check(_fn("recurrence_ops", "ssb_head_norm_gate")(
         _ptr(o), c_int(o.stride(0)), _ptr(weight), c_int(dtype_code(weight.dtype)), c_int(w_stride), c_float(eps),
-        _ptr(gate), c_int(gate.stride(0)), c_int(GATE_KINDS[gate_kind]), _ptr(out), c_int(out.stride(0)),
+        _ptr(gate), c_int(gate.stride(0) if gate is not None else 0), c_int(GATE_KINDS[gate_kind]), _ptr(out), c_int(out.stride(0)),
         c_int(dtype_code(out.dtype)), c_int(T), c_int(n_heads), c_int(vdim), c_int(1 if pdl else 0), _stream()),
         "head_norm_gate")
 
@@ -968,7 +1085,8 @@ def qkv_prepare(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: O
                 v_cos: Optional[torch.Tensor], v_sin: Optional[torch.Tensor], v_interleaved: bool, pos: torch.Tensor,
                 slot: torch.Tensor, page_table: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, n_q: int,
                 n_kv: int, dim: int, vdim: int, page_shift: int, write_cache: bool = True, pdl: bool = False,
-                pooled=None, pool: int = 0, v_off: Optional[int] = None, q_temp=None, n_v: Optional[int] = None) -> None:
+                pooled=None, pool: int = 0, v_off: Optional[int] = None, q_temp=None, n_v: Optional[int] = None,
+                v_mix=None) -> None:
     """Rows [q (n_q x dim) | k (n_kv x dim) | v (n_kv x vdim)].  ``norm`` ``"head"``: every q and k head is divided
     by its root mean square (eps inside the root) and multiplied by a weight vector [dim] shared by the heads;
     ``"row"``: all heads of q (of k) together are divided by one root mean square, weights [heads x dim]; None:
@@ -979,7 +1097,8 @@ def qkv_prepare(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: O
     run writes the run's pooled row as ``pool_rows`` would.  ``v_off``: the column where the values start (default:
     behind the keys; the keys' own column for values that are the keys as projected, before their norm).  ``q_temp`` =
     (coef, every): the queries at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1).  ``n_v``:
-    value heads, if fewer than key heads (several score maps over the same values)."""
+    value heads, if fewer than key heads (several score maps over the same values).  ``v_mix`` = (values [tokens, >= n_v x
+    vdim] of another layer for the same tokens, lambda): v <- (1 - lambda) v + lambda values before anything else."""
     _need(qkv, "qkv", None, 2); _need(pos, "pos", torch.int32, 1); _need(slot, "slot", torch.int32, 1)
     _need(page_table, "page_table", torch.int32, 2)
     if norm not in QK_NORM_MODES:
@@ -1014,6 +1133,11 @@ def qkv_prepare(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: O
         _need(k_cache, "k_cache", qkv.dtype); _need(v_cache, "v_cache", qkv.dtype)
         if not (k_cache.is_contiguous() and v_cache.is_contiguous()) or k_cache.shape[-1] != dim or v_cache.shape[-1] != vdim:
             raise KernelError("qkv_prepare: cache rows of dim and vdim, contiguous")
+    v_first, v_lambda = v_mix if v_mix is not None else (None, 0.0)
+    if v_first is not None:
+        _need(v_first, "mixed values", qkv.dtype, 2)
+        if v_first.shape[0] != T or v_first.shape[1] < n_v * vdim:
+            raise KernelError("qkv_prepare: the values mixed in have a row of all value heads per token")
     pk = pv = ptable = None
     if pool:
         if not write_cache or pooled is None:
@@ -1029,7 +1153,8 @@ def qkv_prepare(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: O
         c_int(page_table.shape[1]), _ptr(k_cache), _ptr(v_cache), c_int(T), c_int(n_q), c_int(n_kv), c_int(dim), c_int(vdim),
         c_int(page_shift), c_int(1 if write_cache else 0), _ptr(pk), _ptr(pv), _ptr(ptable),
         c_int(ptable.shape[1] if ptable is not None else 0), c_int(int(pool) if pool else 0), c_int(v_off), c_int(n_v),
-        c_float(coef), c_int(every), c_int(1 if pdl else 0), _stream()), "qkv_prepare")
+        c_float(coef), c_int(every), _ptr(v_first), c_int(v_first.stride(0) if v_first is not None else 0), c_float(v_lambda),
+        c_int(1 if pdl else 0), _stream()), "qkv_prepare")
 
 
 def pool_rows(k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor, pk_cache: torch.Tensor,
@@ -1056,7 +1181,7 @@ def pool_rows(k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Te
 
 
 def _window_attention_args(q, k_cache, v_cache, page_table, pooled, out, n_q, n_kv, dim, vdim, window, keep_first, pool,
-                           sinks, v_cos, v_sin, what, v_share=1, gate=None):
+                           sinks, v_cos, v_sin, what, v_share=1, gate=None, gate_elems=False, slopes=None, head_mul=None):
     _need(q, "q", None, 2); _need(out, "out", q.dtype, 2); _need(k_cache, "k_cache", q.dtype); _need(v_cache, "v_cache", q.dtype)
     _need(page_table, "page_table", torch.int32, 2)
     T = q.shape[0]
@@ -1067,8 +1192,15 @@ def _window_attention_args(q, k_cache, v_cache, page_table, pooled, out, n_q, n_
         raise KernelError(f"{what}: {n_kv} key heads do not share values {v_share} at a time (and not with pooled runs)")
     if gate is not None:
         _need(gate, "gate", q.dtype, 2)
-        if gate.shape[0] != T or gate.shape[1] < n_q:
-            raise KernelError(f"{what}: one gate per token and head")
+        if gate.shape[0] != T or gate.shape[1] < (n_q * vdim if gate_elems else n_q):
+            raise KernelError(f"{what}: one gate per token and head, or per token and element of its heads")
+    for v, name in ((slopes, "slope"), (head_mul, "score factor")):
+        if v is not None:
+            _need(v, name, torch.float32, 1)
+            if v.shape[0] != n_q:
+                raise KernelError(f"{what}: one {name} per query head")
+    if pool and slopes is not None:
+        raise KernelError(f"{what}: a pooled run has no one distance to take a bias from")
     pk = pv = ptable = None
     if pool:
         if not window:
@@ -1092,7 +1224,8 @@ def window_attention_plain(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
                            vdim: int, page_shift: int, window: Optional[int], keep_first: int, pool: int, scale: float,
                            softcap: Optional[float], sinks, v_cos: Optional[torch.Tensor], v_sin: Optional[torch.Tensor],
                            v_interleaved: bool, out_scale: float = 1.0, pdl: bool = False, v_share: int = 1,
-                           gate: Optional[torch.Tensor] = None) -> None:
+                           gate: Optional[torch.Tensor] = None, gate_elems: bool = False,
+                           slopes: Optional[torch.Tensor] = None, head_mul: Optional[torch.Tensor] = None) -> None:
     """Softmax attention of every token over its slot's cache: the keys j with pos - window < j <= pos, the first
     ``keep_first`` tokens, and (``pool`` > 0, ``pooled`` = (keys, values, page table) of the pooled store) the
     pooled row of every run of ``pool`` tokens that ends at or before pos - window.  Scores times ``scale``, then
@@ -1100,10 +1233,11 @@ def window_attention_plain(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
     denominator) or one float per query head.  With ``v_cos``/``v_sin`` the head's sum is turned back by the
     token's position.  ``out`` is multiplied by ``out_scale``.  ``v_share``: that many key heads in a row read one
     value head (the value store has n_kv / v_share heads).  ``gate`` [tokens, >= n_q]: head h of token t is
-    multiplied by sigmoid(gate[t, h])."""
+    multiplied by sigmoid(gate[t, h]); with ``gate_elems`` [tokens, >= n_q x vdim], a gate per element of the result.
+    ``head_mul``: a factor per query head on its scores; ``slopes``: slope_h * (pos - j) is taken off them (after a cap)."""
     pk, pv, ptable, positions = _window_attention_args(q, k_cache, v_cache, page_table, pooled, out, n_q, n_kv, dim, vdim,
                                                        window, keep_first, pool, sinks, v_cos, v_sin, "window_attention",
-                                                       v_share, gate)
+                                                       v_share, gate, gate_elems, slopes, head_mul)
     _need(pos, "pos", torch.int32, 1); _need(slot, "slot", torch.int32, 1)
     zero_sink = sinks is True
     _check(_fn("window_attention", "ssb_window_attention_plain")(
@@ -1114,7 +1248,8 @@ def window_attention_plain(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
         c_int(int(pool or 0)), c_float(scale), c_float(float(softcap) if softcap else 0.0),
         _ptr(None if (sinks is None or isinstance(sinks, bool)) else sinks), c_int(1 if zero_sink else 0), _ptr(v_cos),
         _ptr(v_sin), c_int(1 if v_interleaved else 0), c_int(positions), c_float(out_scale), c_int(v_share), _ptr(gate),
-        c_int(gate.stride(0) if gate is not None else 0), c_int(1 if pdl else 0), _stream()), "window_attention_plain")
+        c_int(gate.stride(0) if gate is not None else 0), c_int(1 if gate_elems else 0), _ptr(slopes), _ptr(head_mul),
+        c_int(1 if pdl else 0), _stream()), "window_attention_plain")
 
 
 def window_attention_mma_ok(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, pooled, out: torch.Tensor,
@@ -1135,7 +1270,8 @@ def window_attention_mma(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
                          keep_first: int, pool: int, scale: float, softcap: Optional[float], sinks,
                          v_cos: Optional[torch.Tensor], v_sin: Optional[torch.Tensor], v_interleaved: bool,
                          out_scale: float = 1.0, split: Optional[bool] = None, pdl: bool = False, v_share: int = 1,
-                         gate: Optional[torch.Tensor] = None) -> None:
+                         gate: Optional[torch.Tensor] = None, gate_elems: bool = False,
+                         slopes: Optional[torch.Tensor] = None, head_mul: Optional[torch.Tensor] = None) -> None:
     """``window_attention_plain`` on mma.sync for bfloat16: a block streams what a tile of (token, head of one kv
     group) rows can see once (pooled rows, kept first tokens, the window's pages); scores, weights and sums
     float32, the weights entering the second product as hi + lo bfloat16.  ``split`` (default: steps of one
@@ -1144,7 +1280,7 @@ def window_attention_mma(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         raise KernelError(f"window_attention_mma: dim {dim}, vdim {vdim} or operands not supported")
     pk, pv, ptable, positions = _window_attention_args(q, k_cache, v_cache, page_table, pooled, out, n_q, n_kv, dim, vdim,
                                                        window, keep_first, pool, sinks, v_cos, v_sin, "window_attention_mma",
-                                                       v_share, gate)
+                                                       v_share, gate, gate_elems, slopes, head_mul)
     _need(cu_new, "cu_new", torch.int32, 1); _need(seq_start, "seq_start", torch.int32, 1); _need(seq_slot, "seq_slot", torch.int32, 1)
     B = seq_slot.shape[0]
     if cu_new.shape[0] != B + 1 or seq_start.shape[0] != B:
@@ -1159,8 +1295,8 @@ def window_attention_mma(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         c_int(int(pool or 0)), c_float(scale), c_float(float(softcap) if softcap else 0.0),
         _ptr(None if (sinks is None or isinstance(sinks, bool)) else sinks), c_int(1 if sinks is True else 0), _ptr(v_cos),
         _ptr(v_sin), c_int(1 if v_interleaved else 0), c_int(positions), c_float(out_scale), c_int(v_share), _ptr(gate),
-        c_int(gate.stride(0) if gate is not None else 0), c_int(1 if split else 0), c_int(1 if pdl else 0), _stream()),
-        "window_attention_mma")
+        c_int(gate.stride(0) if gate is not None else 0), c_int(1 if gate_elems else 0), _ptr(slopes), _ptr(head_mul),
+        c_int(1 if split else 0), c_int(1 if pdl else 0), _stream()), "window_attention_mma")
 
 
 def map_difference(maps: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv: int, vdim: int, lam: float, eps: float,
@@ -1263,6 +1399,21 @@ def route_sigmoid_groups(logits: torch.Tensor, n_experts: int, correction: Optio
         _ptr(logits), c_int(logits.stride(0)), _ptr(correction), c_int(T), c_int(n_experts), c_int(n_groups), c_int(keep),
         c_int(top), c_float(scale), c_int(-1 if extra_col is None else extra_col), _ptr(expert_of), _ptr(pair_weight),
         _ptr(extra_out if extra_col is not None else None), c_int(1 if pdl else 0), _stream()), "route_sigmoid_groups")
+
+
+def route_softmax(logits: torch.Tensor, n_experts: int, renormalize: bool, scale: float, expert_of: torch.Tensor,
+                  pair_weight: torch.Tensor, pdl: bool = False) -> None:
+    """Per token, from float32 router logits [tokens, >= n_experts]: s = softmax(z) over all experts; the ``top`` experts
+    with the largest s; pair_weight = s * scale, with ``renormalize`` divided by the chosen scores' sum (+ 1e-20)."""
+    _need(logits, "logits", torch.float32, 2)
+    _need(expert_of, "expert_of", torch.int32, 2); _need(pair_weight, "pair_weight", torch.float32, 2)
+    T, top = logits.shape[0], expert_of.shape[1]
+    if logits.shape[1] < n_experts or not 1 <= top <= n_experts or tuple(expert_of.shape) != (T, top) \
+            or tuple(pair_weight.shape) != (T, top) or not (expert_of.is_contiguous() and pair_weight.is_contiguous()):
+        raise KernelError("route_softmax: logits [tokens, >= experts]; expert_of and pair_weight [tokens, top], contiguous")
+    _check(_fn("expert_ops", "ssb_route_softmax")(
+        _ptr(logits), c_int(logits.stride(0)), c_int(T), c_int(n_experts), c_int(top), c_int(1 if renormalize else 0),
+        c_float(scale), _ptr(expert_of), _ptr(pair_weight), c_int(1 if pdl else 0), _stream()), "route_softmax")
 
 
 def expert_tiles_bound(n_pairs: int, n_experts: int, tile_rows: int) -> int:

@@ -459,7 +459,7 @@ SSB_API int ssb_attention_plain(const void* q, int ldq, int dtype, const void* k
 
 // ---------------------------------------------------------------------------------------
 // A gated unit's inner step: z[t, c] = gate_fn(gate[t, c], up[t, c]) * row_scale[t] (ssb_gate: silu(g) u, or the
-// clamped form g' sigmoid(1.702 g') (u' + 1)).  Gate and up are the two halves of a row, or (interleaved) come as
+// clamped form g' sigmoid(1.702 g') (u' + 1), or gelu(g) u).  Gate and up are the two halves of a row, or (interleaved) come as
 // [8 gate | 8 up] per 16 columns.  row_scale: one float32 factor per row, or none.
 // ---------------------------------------------------------------------------------------
 template <typename T>
@@ -483,7 +483,7 @@ __global__ void gated_activation_kernel(const T* __restrict__ gu, int ld, T* __r
 SSB_API int ssb_gated_activation(const void* gate_up, int ld, void* z, int ldz, int dtype, int n_tokens, int inter,
                                  int interleaved, int kind, float limit, const float* row_scale, int pdl,
                                  cudaStream_t stream) {
-    if ((interleaved && inter % 8) || kind < 0 || kind > SSB_GATE_CLAMPED_SWISH) return SSB_ERR_BAD_SIZE;
+    if ((interleaved && inter % 8) || kind < 0 || kind > SSB_GATE_LAST) return SSB_ERR_BAD_SIZE;
     const size_t total = (size_t)n_tokens * inter;
     if (total == 0) return 0;
     const unsigned blocks = (unsigned)((total + 255) / 256);

@@ -8,6 +8,11 @@
 // The scan walks a sequence's new tokens in order, from the state the sequence's slot holds, and
 // leaves the state there; a block owns a tile of value columns of one head of one sequence, so no
 // sum depends on what else is in the batch.
+//
+// Tied form (HGRN2): the forget gate f_t per key channel also says what is written,
+//     f_t = l + (1 - l) sigmoid(z_t),    S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T,    o_t = S_t^T silu(q_t)
+// walked as S <- S + k (v - S) with k = 1 - f = (1 - l) sigmoid(-z): a gate close to one loses nothing to the
+// rounding of 1 - f.
 #include "common.cuh"
 #include <math.h>
 #include <type_traits>
@@ -49,13 +54,19 @@ __global__ void decay_kernel(float* __restrict__ z, int ldz, const float* __rest
     *p = expf(log_sigmoid(*p + z_bias[c]) * inv_tau);
 }
 
-template <typename T>
+// The written share 1 - f of the tied form, from the gate's pre-activation (bias included) and the lower bound.
+__device__ __forceinline__ float tied_share(float z, float lower) { return (1.0f - lower) / (1.0f + expf(z)); }
+
+// TIED: k_off names the columns of the gate's pre-activation (bias z_bias, lower bounds `lower`, per head and channel),
+// z is not read, and q passes silu.
+template <typename T, bool TIED>
 __global__ void __launch_bounds__(SCAN_COLS * SCAN_GROUPS)
 gated_linear_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v_off,
                          const float* __restrict__ z, int ldz, float q_scale, float* __restrict__ state,
                          const int* __restrict__ cu_new, const int* __restrict__ seq_slot,
                          float* __restrict__ out, int ldo, int n_heads, int dim, int vdim,
-                         int chunk, int max_chunks, float* __restrict__ sums, float* __restrict__ decays) {
+                         int chunk, int max_chunks, float* __restrict__ sums, float* __restrict__ decays,
+                         const float* __restrict__ z_bias, const float* __restrict__ lower) {
     constexpr int NT = SCAN_COLS * SCAN_GROUPS;
     extern __shared__ __align__(16) float sm[];
     // rows per thread, a multiple of four: thread (g, j) owns rows g * rpt .. + rpt - 1 of column j, and reads
@@ -93,11 +104,14 @@ gated_linear_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
     // a turn stages SCAN_TOKENS tokens: item (token, channel) n * NT + tid of the turn is this thread's
     float zz[SCAN_ITEMS], kk[SCAN_ITEMS], qq[SCAN_ITEMS], vv = 0.f, a_prod = 1.f;
     int item_tt[SCAN_ITEMS], item_i[SCAN_ITEMS];         // the same in every turn: divided once
+    float item_bias[SCAN_ITEMS], item_low[SCAN_ITEMS];
 #pragma unroll
     for (int n = 0; n < SCAN_ITEMS; ++n) {
         const int item = n * NT + tid;
         item_tt[n] = item < SCAN_TOKENS * dim ? item / dim : SCAN_TOKENS;
         item_i[n] = item % dim;
+        item_bias[n] = TIED ? z_bias[h * dim + item_i[n]] : 0.f;
+        item_low[n] = TIED ? lower[h * dim + item_i[n]] : 0.f;
     }
     auto fetch = [&](int t) {
         const int n_tok = min(SCAN_TOKENS, t1 - t);
@@ -106,7 +120,7 @@ gated_linear_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
             const int tt = item_tt[n], i = item_i[n];
             if (tt < n_tok) {
                 const T* row = proj + (size_t)(t + tt) * ld;
-                zz[n] = z[(size_t)(t + tt) * ldz + h * dim + i];
+                zz[n] = TIED ? 0.f : z[(size_t)(t + tt) * ldz + h * dim + i];
                 kk[n] = ssb_to_float(row[k_off + h * dim + i]);
                 qq[n] = ssb_to_float(row[q_off + h * dim + i]);
             }
@@ -124,16 +138,21 @@ gated_linear_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
         for (int n = 0; n < SCAN_ITEMS; ++n) {
             const int tt = item_tt[n], i = item_i[n];
             if (tt < n_tok) {
-                a_s[tt * dimp + i] = zz[n];
-                k_s[tt * dimp + i] = kk[n];
-                q_s[tt * dimp + i] = qq[n] * q_scale;
+                if (TIED) {
+                    k_s[tt * dimp + i] = tied_share(kk[n] + item_bias[n], item_low[n]);
+                    q_s[tt * dimp + i] = qq[n] / (1.0f + expf(-qq[n])) * q_scale;
+                } else {
+                    a_s[tt * dimp + i] = zz[n];
+                    k_s[tt * dimp + i] = kk[n];
+                    q_s[tt * dimp + i] = qq[n] * q_scale;
+                }
             }
         }
         if (tid < SCAN_TOKENS * SCAN_COLS) v_s[tid] = vv;
         __syncthreads();
         if (t + SCAN_TOKENS < t1) fetch(t + SCAN_TOKENS);
         if (decays != nullptr && tid < dim)
-            for (int tt = 0; tt < n_tok; ++tt) a_prod *= a_s[tt * dimp + tid];
+            for (int tt = 0; tt < n_tok; ++tt) a_prod *= TIED ? 1.0f - k_s[tt * dimp + tid] : a_s[tt * dimp + tid];
         for (int tt = 0; tt < n_tok; ++tt) {
             const float v = v_s[tt * SCAN_COLS + j];
             const float4* a4 = reinterpret_cast<const float4*>(a_s + tt * dimp + g * rpt);
@@ -143,7 +162,15 @@ gated_linear_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
 #pragma unroll
             for (int r = 0; r < SCAN_MAX_ROWS; r += 4)
                 if (r < rpt) {
-                    const float4 a = a4[r >> 2], k = k4[r >> 2], q = q4[r >> 2];
+                    const float4 k = k4[r >> 2], q = q4[r >> 2];
+                    if (TIED) {
+                        s_reg[r] = fmaf(k.x, v - s_reg[r], s_reg[r]);              o = fmaf(s_reg[r], q.x, o);
+                        s_reg[r + 1] = fmaf(k.y, v - s_reg[r + 1], s_reg[r + 1]);  o = fmaf(s_reg[r + 1], q.y, o);
+                        s_reg[r + 2] = fmaf(k.z, v - s_reg[r + 2], s_reg[r + 2]);  o = fmaf(s_reg[r + 2], q.z, o);
+                        s_reg[r + 3] = fmaf(k.w, v - s_reg[r + 3], s_reg[r + 3]);  o = fmaf(s_reg[r + 3], q.w, o);
+                        continue;
+                    }
+                    const float4 a = a4[r >> 2];
                     s_reg[r] = fmaf(a.x, s_reg[r], k.x * v);          o = fmaf(s_reg[r], q.x, o);
                     s_reg[r + 1] = fmaf(a.y, s_reg[r + 1], k.y * v);  o = fmaf(s_reg[r + 1], q.y, o);
                     s_reg[r + 2] = fmaf(a.z, s_reg[r + 2], k.z * v);  o = fmaf(s_reg[r + 2], q.z, o);
@@ -205,21 +232,13 @@ gated_linear_carry_kernel(float* __restrict__ state, float* __restrict__ sums, c
     state[(size_t)slot * per + e] = cur;
 }
 
-// proj [T, ld] holds q, k (n_heads x dim each) and v (n_heads x vdim) from the given columns;
-// z [T, ldz] float32 is the decay's pre-activation without its bias z_bias [n_heads x dim], and is overwritten
-// with the decays;
-// state [slots, n_heads, dim, vdim] float32; out [T, ldo] float32 gets o (n_heads x vdim).
-// chunk > 0: sequences are run in chunks of that many tokens, in parallel, through ``sums``
-// (n_seqs x max_chunks x n_heads x dim x vdim floats) and ``decays`` (n_seqs x max_chunks x n_heads x dim);
-// max_chunks = ceil(longest run of new tokens / chunk).
-SSB_API int ssb_gated_linear_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off,
-                                  float* z, int ldz, const float* z_bias, float tau, float q_scale,
-                                  float* state, const int* cu_new, const int* seq_slot, float* out, int ldo,
-                                  int n_seqs, int n_tokens, int n_heads, int dim, int vdim, int chunk, int max_chunks,
-                                  float* sums, float* decays, int pdl, cudaStream_t stream) {
-    if (n_seqs <= 0 || n_tokens <= 0) return 0;
-    if (dim <= 0 || dim > SCAN_MAX_ROWS * SCAN_GROUPS || vdim <= 0 || !(tau > 0.f)) return SSB_ERR_BAD_SIZE;
-    if (chunk < 0 || (chunk > 0 && (max_chunks <= 0 || sums == nullptr || decays == nullptr))) return SSB_ERR_BAD_SIZE;
+// The launches of a scan over prepared decays (or, TIED, over the gate's pre-activations): one walk, or chunk sums, carry
+// and chunk outputs.
+template <bool TIED>
+static int gated_scan_launches(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off, const float* z, int ldz,
+                               float q_scale, float* state, const int* cu_new, const int* seq_slot, float* out, int ldo,
+                               int n_seqs, int n_heads, int dim, int vdim, int chunk, int max_chunks, float* sums,
+                               float* decays, const float* z_bias, const float* lower, int pdl, cudaStream_t stream) {
     const long long items = chunk > 0 ? (long long)n_seqs * max_chunks : n_seqs;
     if (items > 0x7fffffffll) return SSB_ERR_BAD_SIZE;
     const dim3 grid((unsigned)items, n_heads, (vdim + SCAN_COLS - 1) / SCAN_COLS);
@@ -227,17 +246,10 @@ SSB_API int ssb_gated_linear_scan(const void* proj, int ld, int dtype, int q_off
     const int rpt = ((dim + SCAN_GROUPS - 1) / SCAN_GROUPS + 3) & ~3;
     const size_t smem = (size_t)SCAN_TOKENS * (3 * rpt * SCAN_GROUPS + SCAN_COLS + SCAN_COLS * SCAN_GROUPS) * sizeof(float);
     int rc = 0;
-    {
-        const size_t total = (size_t)n_tokens * n_heads * dim;
-        rc = ssb_launch(decay_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, pdl != 0, z, ldz, z_bias,
-                        1.0f / tau, n_heads * dim, total);
-        if (!rc) rc = ssb_launch_status();
-        if (rc) return rc;
-    }
 #define SSB_SCAN(T, OUT) \
-    rc = ssb_launch(gated_linear_scan_kernel<T>, grid, dim3(SCAN_COLS * SCAN_GROUPS), smem, stream, pdl != 0, \
+    rc = ssb_launch(gated_linear_scan_kernel<T, TIED>, grid, dim3(SCAN_COLS * SCAN_GROUPS), smem, stream, pdl != 0, \
                     (const T*)proj, ld, q_off, k_off, v_off, (const float*)z, ldz, q_scale, state, cu_new, seq_slot, \
-                    OUT, ldo, n_heads, dim, vdim, chunk, max_chunks, sums, decays)
+                    OUT, ldo, n_heads, dim, vdim, chunk, max_chunks, sums, decays, z_bias, lower)
 #define SSB_SCAN_BOTH(OUT) do { \
         if (dtype == SSB_F32) SSB_SCAN(float, OUT); \
         else if (dtype == SSB_BF16) SSB_SCAN(bf16, OUT); \
@@ -261,11 +273,159 @@ SSB_API int ssb_gated_linear_scan(const void* proj, int ld, int dtype, int q_off
     return 0;
 }
 
+// proj [T, ld] holds q, k (n_heads x dim each) and v (n_heads x vdim) from the given columns;
+// z [T, ldz] float32 is the decay's pre-activation without its bias z_bias [n_heads x dim], and is overwritten
+// with the decays;
+// state [slots, n_heads, dim, vdim] float32; out [T, ldo] float32 gets o (n_heads x vdim).
+// chunk > 0: sequences are run in chunks of that many tokens, in parallel, through ``sums``
+// (n_seqs x max_chunks x n_heads x dim x vdim floats) and ``decays`` (n_seqs x max_chunks x n_heads x dim);
+// max_chunks = ceil(longest run of new tokens / chunk).
+SSB_API int ssb_gated_linear_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off,
+                                  float* z, int ldz, const float* z_bias, float tau, float q_scale,
+                                  float* state, const int* cu_new, const int* seq_slot, float* out, int ldo,
+                                  int n_seqs, int n_tokens, int n_heads, int dim, int vdim, int chunk, int max_chunks,
+                                  float* sums, float* decays, int pdl, cudaStream_t stream) {
+    if (n_seqs <= 0 || n_tokens <= 0) return 0;
+    if (dim <= 0 || dim > SCAN_MAX_ROWS * SCAN_GROUPS || vdim <= 0 || !(tau > 0.f)) return SSB_ERR_BAD_SIZE;
+    if (chunk < 0 || (chunk > 0 && (max_chunks <= 0 || sums == nullptr || decays == nullptr))) return SSB_ERR_BAD_SIZE;
+    const long long items = chunk > 0 ? (long long)n_seqs * max_chunks : n_seqs;
+    if (items > 0x7fffffffll || n_seqs > 65535 || n_heads > 65535) return SSB_ERR_BAD_SIZE;
+    int rc = 0;
+    {
+        const size_t total = (size_t)n_tokens * n_heads * dim;
+        rc = ssb_launch(decay_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, pdl != 0, z, ldz, z_bias,
+                        1.0f / tau, n_heads * dim, total);
+        if (!rc) rc = ssb_launch_status();
+        if (rc) return rc;
+    }
+    return gated_scan_launches<false>(proj, ld, dtype, q_off, k_off, v_off, z, ldz, q_scale, state, cu_new, seq_slot, out, ldo,
+                                      n_seqs, n_heads, dim, vdim, chunk, max_chunks, sums, decays, nullptr, nullptr, pdl, stream);
+}
+
+// The tied form: f_off names the gate's pre-activation among proj's columns (bias z_bias, lower bounds `lower`, both
+// [n_heads x dim]); otherwise as ssb_gated_linear_scan.
+SSB_API int ssb_tied_scan(const void* proj, int ld, int dtype, int q_off, int f_off, int v_off, const float* z_bias,
+                          const float* lower, float* state, const int* cu_new, const int* seq_slot, float* out, int ldo,
+                          int n_seqs, int n_tokens, int n_heads, int dim, int vdim, int chunk, int max_chunks, float* sums,
+                          float* decays, int pdl, cudaStream_t stream) {
+    if (n_seqs <= 0 || n_tokens <= 0) return 0;
+    if (dim <= 0 || dim > SCAN_MAX_ROWS * SCAN_GROUPS || vdim <= 0 || n_heads <= 0 || z_bias == nullptr || lower == nullptr)
+        return SSB_ERR_BAD_SIZE;
+    if (chunk < 0 || (chunk > 0 && (max_chunks <= 0 || sums == nullptr || decays == nullptr))) return SSB_ERR_BAD_SIZE;
+    return gated_scan_launches<true>(proj, ld, dtype, q_off, f_off, v_off, nullptr, 0, 1.0f, state, cu_new, seq_slot, out, ldo,
+                                     n_seqs, n_heads, dim, vdim, chunk, max_chunks, sums, decays, z_bias, lower, pdl, stream);
+}
+
+// ---------------------------------------------------------------------------------------
+// One token a sequence (a decode step) of the tied form with the head norm behind it, in one launch: a block takes a
+// sequence and a head, its warps share the state's rows (lanes along the value columns, so that a row is read and
+// written in one piece), the partial sums S^T q meet in shared memory, and the head's output is normed and weighted
+// (y = o / rms(o) * w, w [vdim] shared by the heads, a norm's constant factor already in it).
+// ---------------------------------------------------------------------------------------
+constexpr int TS_THREADS = 512;
+constexpr int TS_WARPS = TS_THREADS / 32;
+constexpr int TS_MAX_VDIM = 256;
+
+template <typename T, int NC>                              // NC: columns a lane owns
+__global__ void __launch_bounds__(TS_THREADS)
+tied_step_kernel(const T* __restrict__ proj, int ld, int q_off, int f_off, int v_off, const float* __restrict__ z_bias,
+                 const float* __restrict__ lower, float* __restrict__ state, const int* __restrict__ cu_new,
+                 const int* __restrict__ seq_slot, const float* __restrict__ w, float eps, T* __restrict__ y, int ldy,
+                 int n_heads, int dim, int vdim) {
+    __shared__ float k_s[SCAN_MAX_ROWS * SCAN_GROUPS], q_s[SCAN_MAX_ROWS * SCAN_GROUPS];
+    __shared__ float o_s[TS_WARPS][NC * 32];
+    __shared__ float red[TS_WARPS];
+    const int b = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    ssb_pdl_launch_dependents();
+    ssb_pdl_wait();
+    const int slot = seq_slot[b];
+    if (slot < 0) return;
+    const int t = cu_new[b];
+    const T* row = proj + (size_t)t * ld;
+    for (int i = tid; i < dim; i += TS_THREADS) {
+        k_s[i] = tied_share(ssb_to_float(row[f_off + h * dim + i]) + z_bias[h * dim + i], lower[h * dim + i]);
+        const float q = ssb_to_float(row[q_off + h * dim + i]);
+        q_s[i] = q / (1.0f + expf(-q));
+    }
+    float* S = state + ((size_t)slot * n_heads + h) * dim * vdim;
+    float o[NC], v[NC];
+#pragma unroll
+    for (int n = 0; n < NC; ++n) {
+        const int c = lane + n * 32;
+        o[n] = 0.f;
+        v[n] = c < vdim ? ssb_to_float(row[v_off + h * vdim + c]) : 0.f;
+    }
+    __syncthreads();
+    constexpr int RF = 4;                                  // rows of the state a warp has in flight
+    for (int i0 = warp; i0 < dim; i0 += RF * TS_WARPS) {
+        float s[RF][NC];
+#pragma unroll
+        for (int r = 0; r < RF; ++r)
+#pragma unroll
+            for (int n = 0; n < NC; ++n) {
+                const int i = i0 + r * TS_WARPS, c = lane + n * 32;
+                s[r][n] = (i < dim && c < vdim) ? S[(size_t)i * vdim + c] : 0.f;
+            }
+#pragma unroll
+        for (int r = 0; r < RF; ++r)
+#pragma unroll
+            for (int n = 0; n < NC; ++n) {
+                const int i = i0 + r * TS_WARPS, c = lane + n * 32;
+                if (i < dim && c < vdim) {
+                    const float x = fmaf(k_s[i], v[n] - s[r][n], s[r][n]);
+                    S[(size_t)i * vdim + c] = x;
+                    o[n] = fmaf(x, q_s[i], o[n]);
+                }
+            }
+    }
+#pragma unroll
+    for (int n = 0; n < NC; ++n) o_s[warp][lane + n * 32] = o[n];
+    __syncthreads();
+    float sum = 0.f;                                      // vdim <= 256 < TS_THREADS: a column a thread
+    if (tid < vdim) {
+#pragma unroll
+        for (int g = 0; g < TS_WARPS; ++g) sum += o_s[g][tid];
+    }
+    float sq = sum * sum;
+#pragma unroll
+    for (int m = 16; m > 0; m >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, m);
+    if (lane == 0) red[warp] = sq;
+    __syncthreads();
+    float total = 0.f;
+#pragma unroll
+    for (int g = 0; g < TS_WARPS; ++g) total += red[g];
+    if (tid < vdim)
+        y[(size_t)t * ldy + (size_t)h * vdim + tid] = ssb_from_float<T>(sum / sqrtf(total / (float)vdim + eps) * w[tid]);
+}
+
+SSB_API int ssb_tied_step(const void* proj, int ld, int dtype, int q_off, int f_off, int v_off, const float* z_bias,
+                          const float* lower, float* state, const int* cu_new, const int* seq_slot, const float* w, float eps,
+                          void* y, int ldy, int n_seqs, int n_heads, int dim, int vdim, int pdl, cudaStream_t stream) {
+    if (n_seqs <= 0) return 0;
+    if (dim <= 0 || dim > SCAN_MAX_ROWS * SCAN_GROUPS || vdim <= 0 || n_heads <= 0 || n_heads > 65535 || z_bias == nullptr ||
+        lower == nullptr)
+        return SSB_ERR_BAD_SIZE;
+    if (vdim > TS_MAX_VDIM) return SSB_ERR_UNSUPPORTED;
+    const dim3 grid(n_seqs, n_heads);
+    int rc;
+#define SSB_TS(T, NC_) \
+    rc = ssb_launch(tied_step_kernel<T, NC_>, grid, dim3(TS_THREADS), 0, stream, pdl != 0, (const T*)proj, ld, q_off, f_off, \
+                    v_off, z_bias, lower, state, cu_new, seq_slot, w, eps, (T*)y, ldy, n_heads, dim, vdim)
+#define SSB_TS_NC(T) \
+    if (vdim <= 32) SSB_TS(T, 1); else if (vdim <= 64) SSB_TS(T, 2); else if (vdim <= 128) SSB_TS(T, 4); else SSB_TS(T, 8)
+    if (dtype == SSB_F32) { SSB_TS_NC(float); }
+    else if (dtype == SSB_BF16) { SSB_TS_NC(bf16); }
+    else return SSB_ERR_BAD_DTYPE;
+#undef SSB_TS_NC
+#undef SSB_TS
+    return rc ? rc : ssb_launch_status();
+}
+
 // ---------------------------------------------------------------------------------------
 // y[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * w * act(gate[t, h, :]): a head's
 // output normalised over its own width, weighted (one weight vector for all heads, or w_stride = vdim:
 // one per head), then gated; act is silu (gate_kind 0), sigmoid (1), or the gate as it is (2: the
-// caller has applied its activation already)
+// caller has applied its activation already); without a gate (null) the product ends at w
 // ---------------------------------------------------------------------------------------
 template <typename T, typename TW>
 __global__ void __launch_bounds__(128)
@@ -282,9 +442,13 @@ head_norm_gate_kernel(const float* __restrict__ o, int ldo, const TW* __restrict
 #pragma unroll
     for (int m = 16; m > 0; m >>= 1) part += __shfl_xor_sync(0xffffffffu, part, m);
     const float inv = 1.0f / sqrtf(part / (float)vdim + eps);
-    const T* gr = gate + (size_t)t * ldg + (size_t)h * vdim;
     const TW* wr = w + (size_t)h * w_stride;
     T* dst = y + (size_t)t * ldy + (size_t)h * vdim;
+    if (gate == nullptr) {
+        for (int c = lane; c < vdim; c += 32) dst[c] = ssb_from_float<T>(src[c] * inv * ssb_to_float(wr[c]));
+        return;
+    }
+    const T* gr = gate + (size_t)t * ldg + (size_t)h * vdim;
     for (int c = lane; c < vdim; c += 32) {
         const float gv = ssb_to_float(gr[c]);
         const float sg = 1.0f / (1.0f + expf(-gv));

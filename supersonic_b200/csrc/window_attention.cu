@@ -5,7 +5,9 @@
 // all in one softmax:  s = (q . k) * scale,  optionally s <- cap * tanh(s / cap),  w = exp(s - m) / (sum + sink),
 // where a sink adds exp(sink - m) to the denominator and nothing to the numerator.  The values of a position may
 // be stored turned by that position (pairs over the whole value width); the head's sum is then turned back by
-// the query's position, so that a value enters by the distance between the two.
+// the query's position, so that a value enters by the distance between the two.  A head may multiply its scores by
+// a number of its own (head_mul) and take off a bias that grows with the distance, slope_h * (p - j), which is
+// applied last, after the cap.
 //
 // Here: the preparation of the projected rows [q | k | v] (norm of q and k per head or over the whole row,
 // rotation, append), the pooling of finished runs, the plain kernel (float32 throughout, keys in a fixed order),
@@ -76,6 +78,8 @@ __device__ __forceinline__ void wa_pair(int c, int dims, int interleaved, int& o
 // sequence, the token that ends a run of `pool` tokens may write the run's pooled row as well (see pool_rows).
 //   v_off: the column of the row where the values start (behind the keys; at the keys themselves for a mixer whose
 //   values are its keys as projected, before their norm).
+//   v_first: the values of another layer for the same tokens, mixed in: v <- (1 - v_lambda) v + v_lambda v_first (before
+//   anything else happens to v; the mixed values are what is cached).
 //   q_temp_every > 0: the queries of position p are multiplied by 1 + q_temp_coef * ln(floor((p + 1) / every) + 1).
 // ---------------------------------------------------------------------------------------
 constexpr int WP_THREADS = 256;
@@ -89,7 +93,7 @@ qkv_prepare_kernel(T* __restrict__ qkv, int ld, const float* __restrict__ q_w, c
                    const int* __restrict__ page_table, int max_pages, T* __restrict__ k_cache, T* __restrict__ v_cache,
                    int n_q, int n_kv, int dim, int vdim, int page_shift, int write_cache, T* __restrict__ pk_cache,
                    T* __restrict__ pv_cache, const int* __restrict__ pool_table, int pool_max_pages, int pool, int v_off,
-                   int n_v, float q_temp_coef, int q_temp_every) {
+                   int n_v, float q_temp_coef, int q_temp_every, const T* __restrict__ v_first, int ld_first, float v_lambda) {
     extern __shared__ float wp_row[];                      // the part's row, then one factor per head
     __shared__ float red[WP_THREADS / 32];
     ssb_pdl_launch_dependents();
@@ -120,7 +124,12 @@ qkv_prepare_kernel(T* __restrict__ qkv, int ld, const float* __restrict__ q_w, c
         const T* src = base + v_off;
         const int n = n_v * vdim;                          // n_v value heads (fewer than key heads where several maps share them)
         const bool turn = vcos_t != nullptr && p < table_positions;
-        for (int c = tid; c < n; c += WP_THREADS) wp_row[c] = ssb_to_float(src[c]);
+        const T* other_v = v_first == nullptr ? nullptr : v_first + (size_t)t * ld_first;
+        for (int c = tid; c < n; c += WP_THREADS) {
+            float v = ssb_to_float(src[c]);
+            if (other_v != nullptr) v = (1.0f - v_lambda) * v + v_lambda * ssb_to_float(other_v[c]);
+            wp_row[c] = v;
+        }
         __syncthreads();
         for (int c = tid; c < n; c += WP_THREADS) {
             const int h = c / vdim, d = c - h * vdim;
@@ -194,7 +203,8 @@ SSB_API int ssb_qkv_prepare(void* qkv, int ld, int dtype, const float* q_w, cons
                             const int* page_table, int max_pages, void* k_cache, void* v_cache, int n_tokens, int n_q,
                             int n_kv, int dim, int vdim, int page_shift, int write_cache, void* pk_cache, void* pv_cache,
                             const int* pool_table, int pool_max_pages, int pool, int v_off, int n_v, float q_temp_coef,
-                            int q_temp_every, int pdl, cudaStream_t stream) {
+                            int q_temp_every, const void* v_first, int ld_first, float v_lambda, int pdl,
+                            cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (v_off < 0) v_off = (n_q + n_kv) * dim;
     if (n_v <= 0) n_v = n_kv;
@@ -219,7 +229,7 @@ SSB_API int ssb_qkv_prepare(void* qkv, int ld, int dtype, const float* q_w, cons
                         cos_t, sin_t, rot_dims, interleaved, vcos_t, vsin_t, v_interleaved, table_positions, pos, slot,   \
                         page_table, max_pages, (TYPE*)k_cache, (TYPE*)v_cache, n_q, n_kv, dim, vdim, page_shift,          \
                         write_cache, (TYPE*)pk_cache, (TYPE*)pv_cache, pool_table, pool_max_pages, pool, v_off, n_v,      \
-                        q_temp_coef, q_temp_every);                                                                       \
+                        q_temp_coef, q_temp_every, (const TYPE*)v_first, ld_first, v_lambda);                                                                       \
     }
     if (dtype == SSB_F32) SSB_WP(float)
     else if (dtype == SSB_BF16) SSB_WP(bf16)
@@ -310,7 +320,8 @@ window_attention_plain_kernel(const T* __restrict__ q, int ldq, const T* __restr
                               int n_q, int n_kv, int dim, int vdim, int page_shift, int window, int keep_first, int pool,
                               float scale, float softcap, const float* __restrict__ sinks, int zero_sink,
                               const float* __restrict__ vcos_t, const float* __restrict__ vsin_t, int v_interleaved,
-                              int table_positions, float out_scale, int v_share, const T* __restrict__ gate, int ldg) {
+                              int table_positions, float out_scale, int v_share, const T* __restrict__ gate, int ldg,
+                              int gate_elems, const float* __restrict__ slopes, const float* __restrict__ head_mul) {
     __shared__ float q_s[WA_MAX_DIM];
     __shared__ float p_s[WA_THREADS];
     __shared__ float red[WA_THREADS / 32];
@@ -327,8 +338,13 @@ window_attention_plain_kernel(const T* __restrict__ q, int ldq, const T* __restr
     const WaKeys keys = wa_keys_of(p, window, keep_first, pool);
     // v_share key heads in a row read the values of one value head (several score maps over the same values)
     const int kvh = h / (n_q / n_kv), vh = kvh / v_share, n_v = n_kv / v_share;
-    // a gate per (token, head): the head's result is multiplied by sigmoid(gate)
-    const float gmul = (gate != nullptr ? 1.0f / (1.0f + expf(-ssb_to_float(gate[(size_t)t * ldg + h]))) : 1.0f) * out_scale;
+    // a gate per (token, head), or per element of the head's result: the result is multiplied by sigmoid(gate)
+    const T* gp = gate == nullptr ? nullptr : gate + (size_t)t * ldg + (gate_elems ? (size_t)h * vdim : (size_t)h);
+    auto gmul_of = [&](int d) {
+        return (gp != nullptr ? 1.0f / (1.0f + expf(-ssb_to_float(gp[gate_elems ? d : 0]))) : 1.0f) * out_scale;
+    };
+    const float h_scale = head_mul != nullptr ? scale * head_mul[h] : scale;
+    const float slope = slopes != nullptr ? slopes[h] : 0.f;
     const T* qp = q + (size_t)t * ldq + (size_t)h * dim;
     for (int d = tid; d < dim; d += WA_THREADS) q_s[d] = ssb_to_float(qp[d]);
     __syncthreads();
@@ -358,8 +374,12 @@ window_attention_plain_kernel(const T* __restrict__ q, int ldq, const T* __restr
             rows_of(i, kr, vr);
             float dot = 0.f;
             for (int d = 0; d < dim; ++d) dot = fmaf(q_s[d], ssb_to_float(kr[d]), dot);
-            sc = dot * scale;
+            sc = dot * h_scale;
             if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);
+            if (slopes != nullptr) {                             // no pooled runs here: key i is a token
+                const int j = i < keys.n_keep ? i : keys.lo + (i - keys.n_keep);
+                sc -= slope * (float)(p - j);
+            }
         }
         const float cm = wa_block_max<WA_THREADS>(sc, red);
         const float m_new = fmaxf(m, cm);
@@ -399,7 +419,7 @@ window_attention_plain_kernel(const T* __restrict__ q, int ldq, const T* __restr
 #pragma unroll
         for (int c = 0; c < WA_MAX_DIM / WA_THREADS; ++c) {
             const int d = tid + c * WA_THREADS;
-            if (d < vdim) o[d] = ssb_from_float<T>(acc[c] * inv * gmul);
+            if (d < vdim) o[d] = ssb_from_float<T>(acc[c] * inv * gmul_of(d));
         }
         return;
     }
@@ -417,7 +437,7 @@ window_attention_plain_kernel(const T* __restrict__ q, int ldq, const T* __restr
         const float cs = vcos_t[(size_t)p * (vdim >> 1) + pair], sn = vsin_t[(size_t)p * (vdim >> 1) + pair];
         const float v = q_s[d], ov = q_s[other];
         const float r = first ? v * cs + ov * sn : v * cs - ov * sn;
-        o[d] = ssb_from_float<T>(r * gmul);
+        o[d] = ssb_from_float<T>(r * gmul_of(d));
     }
 }
 
@@ -427,10 +447,11 @@ SSB_API int ssb_window_attention_plain(const void* q, int ldq, int dtype, const 
                                        int ldo, int n_tokens, int n_q, int n_kv, int dim, int vdim, int page_shift, int window,
                                        int keep_first, int pool, float scale, float softcap, const float* sinks,
                                        int zero_sink, const float* vcos_t, const float* vsin_t, int v_interleaved,
-                                       int table_positions, float out_scale, int v_share, const void* gate, int ldg, int pdl,
+                                       int table_positions, float out_scale, int v_share, const void* gate, int ldg,
+                                       int gate_elems, const float* slopes, const float* head_mul, int pdl,
                                        cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (v_share < 1 || n_kv % v_share) return SSB_ERR_BAD_SIZE;
+    if (v_share < 1 || n_kv % v_share || (pool > 0 && slopes != nullptr)) return SSB_ERR_BAD_SIZE;
     if (dim <= 0 || dim > WA_MAX_DIM || vdim <= 0 || vdim > WA_MAX_DIM || n_kv <= 0 || n_q % n_kv || n_q > 65535 ||
         window < 0 || keep_first < 0 || pool < 0 || (pool > 0 && (window <= 0 || pk_cache == nullptr || pool_table == nullptr)) ||
         (vcos_t != nullptr && (vdim & 1)))
@@ -442,13 +463,13 @@ SSB_API int ssb_window_attention_plain(const void* q, int ldq, int dtype, const 
                         (const float*)k_cache, (const float*)v_cache, page_table, max_pages, (const float*)pk_cache,
                         (const float*)pv_cache, pool_table, pool_max_pages, pos, slot, (float*)out, ldo, n_q, n_kv, dim, vdim,
                         page_shift, window, keep_first, pool, scale, softcap, sinks, zero_sink, vcos_t, vsin_t, v_interleaved,
-                        table_positions, out_scale, v_share, (const float*)gate, ldg);
+                        table_positions, out_scale, v_share, (const float*)gate, ldg, gate_elems, slopes, head_mul);
     else if (dtype == SSB_BF16)
         rc = ssb_launch(window_attention_plain_kernel<bf16>, grid, dim3(WA_THREADS), 0, stream, pdl != 0, (const bf16*)q, ldq,
                         (const bf16*)k_cache, (const bf16*)v_cache, page_table, max_pages, (const bf16*)pk_cache,
                         (const bf16*)pv_cache, pool_table, pool_max_pages, pos, slot, (bf16*)out, ldo, n_q, n_kv, dim, vdim,
                         page_shift, window, keep_first, pool, scale, softcap, sinks, zero_sink, vcos_t, vsin_t, v_interleaved,
-                        table_positions, out_scale, v_share, (const bf16*)gate, ldg);
+                        table_positions, out_scale, v_share, (const bf16*)gate, ldg, gate_elems, slopes, head_mul);
     else
         return SSB_ERR_BAD_DTYPE;
     return rc ? rc : ssb_launch_status();

@@ -43,6 +43,9 @@ struct WmArgs {
     float out_scale;
     int v_share;                  // key heads in a row that read the values of one value head (several score maps over the same values)
     const bf16* gate; int ldg;    // one gate per (token, head), or none: the head's result is multiplied by sigmoid(gate)
+    int gate_elems;               // ... or one per element of a head's result
+    const float* slopes;          // per query head, or none: slope * (p - j) is taken off the score (after the cap)
+    const float* head_mul;        // per query head, or none: a factor on the scale
 };
 
 template <int DIM, int VDIM, bool SPLIT, int ST>          // ST: pages in the ring
@@ -123,6 +126,7 @@ window_attention_mma_kernel(const WmArgs a) {
     const int wrow0 = row0 + (SPLIT ? 0 : warp * 16);
     int r_tok[2], r_head[2], r_pos[2], r_lo[2], r_npool[2], r_nkeep[2];
     bool r_ok[2];
+    float r_scale[2], r_slope[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
         const int R = wrow0 + g + e * 8;
@@ -133,6 +137,8 @@ window_attention_mma_kernel(const WmArgs a) {
         r_lo[e] = (window > 0 && r_pos[e] - window + 1 > 0) ? r_pos[e] - window + 1 : 0;
         r_npool[e] = pool > 0 ? r_lo[e] / pool : 0;
         r_nkeep[e] = min(a.keep_first, r_lo[e]);
+        r_scale[e] = a.head_mul != nullptr ? a.scale * a.head_mul[r_head[e]] : a.scale;
+        r_slope[e] = a.slopes != nullptr ? a.slopes[r_head[e]] : 0.f;
     }
     const bool warp_live = wrow0 < n_rows;
     // the queries as A fragments: [k step][a0 a1 a2 a3]; columns past the real head size are zero
@@ -210,8 +216,9 @@ window_attention_mma_kernel(const WmArgs a) {
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int rr = e >> 1, kk = key + (e & 1);
-                    float x = s[j][e] * a.scale;
+                    float x = s[j][e] * r_scale[rr];
                     if (a.softcap > 0.f) x = a.softcap * wm_tanh(x * inv_cap);
+                    x = fmaf(r_slope[rr], (float)(kk - r_pos[rr]), x);     // pooled runs come without slopes: 0 times a number
                     const bool vis = r_ok[rr] && kk >= v_lo[rr] && kk <= v_hi[rr];
                     x = vis ? x : -INFINITY;
                     s[j][e] = x;
@@ -364,10 +371,17 @@ window_attention_mma_kernel(const WmArgs a) {
                 }
             }
         }
-        float mul = a.out_scale;
-        if (a.gate != nullptr) mul *= 1.0f / (1.0f + __expf(-__bfloat162float(a.gate[(size_t)(t0 + tok) * a.ldg + head])));
+        float mul = a.out_scale, mul1 = mul;
+        if (a.gate != nullptr && a.gate_elems) {
+            const bf16* gp = a.gate + (size_t)(t0 + tok) * a.ldg + (size_t)head * vdim + c;
+            mul *= 1.0f / (1.0f + __expf(-__bfloat162float(gp[0])));
+            mul1 *= 1.0f / (1.0f + __expf(-__bfloat162float(gp[1])));
+        } else if (a.gate != nullptr) {
+            mul *= 1.0f / (1.0f + __expf(-__bfloat162float(a.gate[(size_t)(t0 + tok) * a.ldg + head])));
+            mul1 = mul;
+        }
         bf16* o = a.out + (size_t)(t0 + tok) * a.ldo + (size_t)head * vdim + c;
-        *reinterpret_cast<uint32_t*>(o) = pack2(x0 * mul, x1 * mul);
+        *reinterpret_cast<uint32_t*>(o) = pack2(x0 * mul, x1 * mul1);
     }
 }
 
@@ -398,9 +412,10 @@ SSB_API int ssb_window_attention_mma(const void* q, int ldq, const void* k_cache
                                      int page_shift, int window, int keep_first, int pool, float scale, float softcap,
                                      const float* sinks, int zero_sink, const float* vcos_t, const float* vsin_t,
                                      int v_interleaved, int table_positions, float out_scale, int v_share, const void* gate,
-                                     int ldg, int split, int pdl, cudaStream_t stream) {
+                                     int ldg, int gate_elems, const float* slopes, const float* head_mul, int split,
+                                     int pdl, cudaStream_t stream) {
     if (n_seqs <= 0 || max_new <= 0) return 0;
-    if (v_share < 1 || n_kv <= 0 || n_kv % v_share || (pool > 0 && v_share > 1)) return SSB_ERR_BAD_SIZE;
+    if (v_share < 1 || n_kv <= 0 || n_kv % v_share || (pool > 0 && (v_share > 1 || slopes != nullptr))) return SSB_ERR_BAD_SIZE;
     if (page_shift != 6 || n_kv <= 0 || n_q % n_kv || (ldq & 1) || (ldo & 1) || window < 0 || keep_first < 0 || pool < 0 ||
         (pool > 0 && (window <= 0 || pk_cache == nullptr || pv_cache == nullptr || pool_table == nullptr)) ||
         dim <= 0 || vdim <= 0 || (dim & 7) || (vdim & 7))
@@ -420,6 +435,7 @@ SSB_API int ssb_window_attention_mma(const void* q, int ldq, const void* k_cache
     a.vcos = vcos_t; a.vsin = vsin_t; a.v_interleaved = v_interleaved; a.table_positions = table_positions;
     a.out_scale = out_scale;
     a.v_share = v_share; a.gate = (const bf16*)gate; a.ldg = ldg;
+    a.gate_elems = gate_elems; a.slopes = slopes; a.head_mul = head_mul;
     const int D = dim <= 64 ? 64 : 128, V = vdim <= 64 ? 64 : 128;
     const long long blocks = (long long)((max_new * (n_q / n_kv) + 15) / 16) * n_kv * n_seqs;     // of the decode form
     const bool deep = split && blocks <= WM_DEEP_MAX_BLOCKS;

@@ -14,7 +14,7 @@ for one token (crates/runner/src/decode_engine.rs:3631-3993), one sequence each.
 from __future__ import annotations
 
 import os
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Any, Dict, Optional, Sequence
 
 import numpy as np
@@ -62,6 +62,7 @@ class StepContext:
     streams: Any = None        # what a block arrangement keeps from layer to layer within one step (the stack of
                                # earlier layers' results for a weighted sum over depth)
     embedded: Any = None       # the embedding's output of the step, for stream adapters that read it again
+    carried: Dict[str, Any] = field(default_factory=dict)   # what a layer leaves for later layers of the same step, by name
 
 
 class DecodeGraph:
@@ -472,7 +473,8 @@ class Model:
                 if moved is not None:
                     residual = moved
                 if self.layer_probe is not None:            # a debugging hook: the stream after every stop
-                    self.layer_probe(stop, residual)
+                    view = getattr(self.blocks[stop.layer], "stream_view", None)
+                    self.layer_probe(stop, residual if view is None else view(ctx, residual))
         if batch.n_want == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=self.device)
         ctx.stage = "head"

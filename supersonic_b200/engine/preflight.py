@@ -120,6 +120,8 @@ def workspace_bytes(spec, dtype: torch.dtype, step_tokens: int, decode_rows: int
     # an arrangement that keeps every layer's result within a step says how many float32 streams it holds
     streams = max([int(b.params.get("depth_average", {}).get("layers", 0)) + 2 if b.params.get("depth_average") else 1
                    for b in spec.blocks] + [1])
+    # several residual streams: their planes, the branch and the stream they are summed into
+    streams = max([streams] + [int(b.params.get("streams") or 0) + 2 for b in spec.blocks if b.params.get("streams")])
     per_token = 4 * spec.hidden_size * streams + item * (2 * spec.hidden_size + widest)
     return step_tokens * per_token + 2 * decode_rows * spec.vocab_size * 4
 

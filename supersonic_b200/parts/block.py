@@ -4,7 +4,9 @@ the residual stream kept and summed in float32 (crates/runner/src/prefill_engine
 norm of its own before it joins the stream.
 ``parallel``: h += mixer(n) + feed_forward(n) with the one n = norm(h), or with a norm each (both of the
 same h); optionally the mixer's input is mixed with the previous token's (token shift), and optionally the
-layer is followed by a learned weighted sum over the results of all layers so far."""
+layer is followed by a learned weighted sum over the results of all layers so far.
+``hyper_connections``: several residual streams; a sublayer reads a weighted sum of them and its result is written into
+all of them, which are mixed with one another at the same time."""
 from __future__ import annotations
 
 import torch
@@ -199,3 +201,114 @@ class ParallelBlock:
         out = ctx.streams[self.index + 2]
         ctx.kernels.stream_mix(ctx.streams, self.depth_weights, self.index + 2, out)
         return out
+
+
+class _Streams:
+    """The residual streams within one step: ``x`` [streams, T, width], or [1, T, width] while all of them still equal the
+    embedding's output; ``branch`` [T, width], which sublayers add into; ``write``, the (mix, out) of the last sublayer
+    whose result still waits in the branch (None: nothing waits)."""
+
+    def __init__(self, embedded):
+        self.x, self.branch, self.write = embedded.unsqueeze(0), torch.zeros_like(embedded), None
+
+
+@register_block("hyper_connections")
+class HyperConnectionBlock:
+    """Residual streams x_1 .. x_S, all equal to the embedding's output at the start.  For each of the two sublayers
+
+        u = sum_s in[s] x_s,    n = norm(u),    h = n + conv(n),    y = sublayer(h)
+        x_t <- sum_s mix[s, t] x_s + out[t] y        (all streams at once from the old ones; mix is [from, to])
+
+    with conv a causal convolution over time on each channel, conv(n)_t = sum_j w[:, j] n_(t - taps + 1 + j), whose last
+    taps - 1 inputs are per-sequence state of the block, one row for each sublayer.  Behind the last layer the stream is
+    the sum of the streams.
+
+    ``params``: ``size``, ``streams``, ``taps`` (0: no convolution), ``last`` (the layer that sums the streams); tensors per
+    sublayer ``s`` in ``mixer``, ``ff``: ``<s>_in`` [S], ``<s>_mix`` [S, S], ``<s>_out`` [S], with a convolution ``<s>_conv``
+    [size, taps].  A sublayer's write waits until the next one's read: both are one pass over the streams, which also
+    takes the norm (and, in steps of one token a sequence, the convolution).  1 is added to the convolution's last tap
+    when the part is built, so that n + conv(n) is one convolution."""
+
+    def __init__(self, mixer, feed_forward, mixer_norm, feed_forward_norm, position, params=None, weights=None, build=None):
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.mixer_norm, self.feed_forward_norm, self.position = mixer_norm, feed_forward_norm, position
+        self.size, self.streams = int(params["size"]), int(params["streams"])
+        self.taps, self.last = int(params.get("taps") or 0), bool(params.get("last"))
+        from ..csrc.ops import CONV_MAX_TAPS, STREAMS_MAX
+        if not 1 <= self.streams <= STREAMS_MAX or not 0 <= self.taps <= CONV_MAX_TAPS:
+            raise ValueError(f"hyper_connections: {self.streams} streams (1 to {STREAMS_MAX}), {self.taps} taps (0 to {CONV_MAX_TAPS})")
+        S = self.streams
+
+        def stored(role, shape):
+            t = build.weights.stored(weights[role]).float().contiguous()
+            if tuple(t.shape) != shape:
+                raise ValueError(f"{weights[role]} has shape {tuple(t.shape)}, expected {shape}")
+            return t
+        self.reads, self.writes, self.convs = [], [], []
+        for sub, norm in (("mixer", mixer_norm), ("ff", feed_forward_norm))[: 1 if feed_forward is None else 2]:
+            if not getattr(norm, "fusable_rms", False):
+                raise ValueError("hyper_connections: the norm behind a read of the streams is an RMS norm")
+            self.reads.append(stored(f"{sub}_in", (S,)))
+            self.writes.append((stored(f"{sub}_mix", (S, S)), stored(f"{sub}_out", (S,))))
+            if self.taps:
+                w = stored(f"{sub}_conv", (self.size, self.taps)).clone()
+                w[:, -1] += 1.0
+                self.convs.append(w)
+            else:
+                self.convs.append(torch.ones((self.size, 1), dtype=torch.float32, device=build.device))
+        self.dtype = build.dtype
+
+    @staticmethod
+    def _needs(mixer_need, size, taps, sublayers):
+        if taps < 2:
+            return mixer_need
+        return {"mixer": mixer_need, **{f"conv{i}": StateNeed((taps - 1) * size) for i in range(sublayers)}}
+
+    def cache_need(self):
+        return self._needs(self.mixer.cache_need(), self.size, self.taps, len(self.reads))
+
+    @staticmethod
+    def cache_need_from(params, mixer_need):
+        return HyperConnectionBlock._needs(mixer_need, int(params["size"]), int(params.get("taps") or 0),
+                                           2 if params.get("feed_forward", True) else 1)
+
+    def _enter(self, ctx, st, i, norm, cache_id):
+        """Finish the write that waits, read the streams for sublayer i, norm and convolve."""
+        T, dev = st.branch.shape[0], st.branch.device
+        h = torch.empty((T, self.size), dtype=self.dtype, device=dev)
+        dst = None
+        if st.write is not None:
+            # written over the old streams, except where those are the one row all of them equal
+            dst = st.x if st.x.shape[0] == self.streams and self.streams > 1 else \
+                torch.empty((self.streams, T, self.size), dtype=torch.float32, device=dev)
+        tail = ctx.cache.state((cache_id, f"conv{i}")) if self.taps > 1 else None
+        ctx.kernels.stream_enter(st.x, self.streams, self.reads[i], st.branch, st.write, dst, norm, self.convs[i], tail,
+                                 ctx.batch, h)
+        if dst is not None:
+            st.x = dst
+        st.write = self.writes[i]
+        return h
+
+    def forward(self, ctx, residual, cache_id, writes_cache):
+        if not writes_cache:
+            raise ValueError("hyper_connections: the block keeps state: its stop must write its cache entry")
+        if not isinstance(ctx.streams, _Streams):
+            ctx.streams = _Streams(residual)
+        st = ctx.streams
+        ctx.stage = "mixer"
+        h = self._enter(ctx, st, 0, self.mixer_norm, cache_id)
+        self.mixer.forward(ctx, h, st.branch, (cache_id, "mixer") if self.taps > 1 else cache_id, writes_cache, self.position)
+        if self.feed_forward is not None:
+            ctx.stage = "feed_forward"
+            h = self._enter(ctx, st, 1, self.feed_forward_norm, cache_id)
+            self.feed_forward.forward(ctx, h, st.branch)
+        return self._sum(ctx, st) if self.last else None
+
+    def _sum(self, ctx, st, clear=True):
+        out = torch.empty_like(st.branch)
+        ctx.kernels.stream_sum(st.x, self.streams, st.branch, st.write, out, clear)
+        return out
+
+    def stream_view(self, ctx, residual):
+        """The stream behind this layer, for probes: the sum of the streams with the waiting write applied."""
+        return residual if self.last else self._sum(ctx, ctx.streams, clear=False)

@@ -10,6 +10,8 @@ chosen experts and their weights:
 * ``sigmoid_groups``: scores s = sigmoid(W x) in float32; experts are chosen by s + correction (a stored vector),
   but only among the experts of the ``keep`` best of ``groups`` equal groups of neighbours, a group's score being
   the sum of its two largest choice scores; the weights are the chosen experts' s times ``scale``, not renormalized.
+* ``softmax``: scores s = softmax(W x) over all experts in float32; the experts with the largest scores are chosen;
+  the weights are their s times ``scale``, with ``renormalize`` divided by their sum (+ 1e-20).
 
 A shared expert runs for every token; with ``shared.gate`` its result is multiplied by sigmoid(w_sg . x), one number
 per token.
@@ -106,6 +108,30 @@ class SigmoidGroupRouter:
         ctx.kernels.linear(x, self.weight, logits)
         ctx.kernels.route_sigmoid_groups(logits, self.n_experts, self.correction, self.groups, self.keep, self.scale,
                                          expert_of, pair_weight, self.extra_col if extra_out is not None else None, extra_out)
+
+
+@register_router("softmax")
+class SoftmaxRouter:
+    """params: ``renormalize`` (True), ``scale`` (1.0); weights: ``weight`` [experts, hidden].  The logits are a product of
+    their own with a float32 result, as ``sigmoid_groups``'."""
+
+    def __init__(self, params, weights, build: BuildContext, n_experts: int, top: int):
+        self.n_experts, self.top = n_experts, top
+        self.renormalize, self.scale = bool(params.get("renormalize", True)), float(params.get("scale", 1.0))
+        if not 1 <= top <= n_experts:
+            raise ValueError(f"softmax router: {top} experts a token of {n_experts}")
+        w = build.weights.as_dtype(weights["weight"], build.dtype)
+        if w.dim() != 2 or w.shape[0] != n_experts:
+            raise ValueError(f"{weights['weight']} has shape {tuple(w.shape)}, expected [{n_experts}, hidden]")
+        pad = (-n_experts) % 8                   # rows of the product's result stay a multiple of 8 wide
+        if pad:
+            w = torch.cat([w, torch.zeros((pad, w.shape[1]), dtype=w.dtype, device=w.device)], dim=0)
+        self.weight = w.contiguous()
+
+    def route(self, ctx, x, expert_of, pair_weight):
+        logits = torch.empty((x.shape[0], self.weight.shape[0]), dtype=torch.float32, device=x.device)
+        ctx.kernels.linear(x, self.weight, logits)
+        ctx.kernels.route_softmax(logits, self.n_experts, self.renormalize, self.scale, expert_of, pair_weight)
 
 
 @register_feed_forward("experts")

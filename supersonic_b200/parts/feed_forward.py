@@ -25,8 +25,8 @@ def gated_activation_of(spec):
 @register_feed_forward("swiglu")
 class SwiGLU:
     """params: ``hidden_size``, ``intermediate_size``, ``activation`` (None: silu(g) u; ``{"kind": "clamped_swish",
-    "limit": L}``: with g' = min(g, L) and u' = clamp(u, -L, L), g' sigmoid(1.702 g') (u' + 1)); weights: ``gate``,
-    ``up``, ``down``.
+    "limit": L}``: with g' = min(g, L) and u' = clamp(u, -L, L), g' sigmoid(1.702 g') (u' + 1); ``{"kind": "gelu_tanh"}``:
+    gelu(g) u, gelu in the form with tanh); weights: ``gate``, ``up``, ``down``.
 
     Interface of a feed-forward: ``forward(ctx, x, residual)`` reads the normed
     activations ``x`` [T, hidden] and adds its output into ``residual`` (float32).

@@ -2,7 +2,9 @@
 
     result = scale * (rms(left) * w_left + rms(right) * w_right)
 
-with the root mean square taken over the model width (eps inside the root) and a weight vector each.
+with the root mean square taken over the model width (eps inside the root) and a weight vector each, or, with
+``join`` = ``"add"``, added as they are, result = left + right, each half with the constant factor its own parameters
+give it (``out_scale``): both then add straight into the stream.
 Either half is any registered mixer; each keeps what it needs in the cache under the pair's id
 (``(cache_id, "left")`` and ``(cache_id, "right")``), and each gets the position encoding only if it asks for it.
 """
@@ -15,17 +17,22 @@ from .registry import MIXERS, BuildContext, lookup, register_mixer
 
 @register_mixer("mixer_pair")
 class MixerPair:
-    """params: ``hidden_size``, ``norm_eps``, ``scale`` (default 1/2), ``left`` and ``right``: each
-    ``{"kind", "params", "weights", "position": bool}``; weights: ``left_out``, ``right_out`` [hidden]."""
+    """params: ``hidden_size``, ``join`` (``"normed"``, the default, or ``"add"``), for normed halves ``norm_eps`` and ``scale``
+    (default 1/2), ``left`` and ``right``: each ``{"kind", "params", "weights", "position": bool}``; weights, for normed
+    halves: ``left_out``, ``right_out`` [hidden]."""
 
     def __init__(self, params, weights, build: BuildContext):
-        self.hidden, self.eps = int(params["hidden_size"]), float(params["norm_eps"])
-        self.scale = float(params.get("scale", 0.5))
+        self.hidden, self.join = int(params["hidden_size"]), params.get("join") or "normed"
+        if self.join not in ("normed", "add"):
+            raise ValueError(f"mixer_pair: join {self.join!r} is not known ('normed' or 'add')")
         self.halves = []
         for side in ("left", "right"):
             sub = params[side]
             self.halves.append((side, lookup(MIXERS, sub["kind"], "mixer")(sub["params"], sub["weights"], build),
                                 bool(sub.get("position", False))))
+        if self.join == "add":
+            return
+        self.eps, self.scale = float(params["norm_eps"]), float(params.get("scale", 0.5))
         self.out_w = [build.weights.stored(weights[s + "_out"]).float().contiguous() for s in ("left", "right")]
         for s, t in zip(("left_out", "right_out"), self.out_w):
             if tuple(t.shape) != (self.hidden,):
@@ -44,7 +51,7 @@ class MixerPair:
 
     @staticmethod
     def activation_elements(params) -> int:
-        total = 4 * int(params["hidden_size"])
+        total = 0 if params.get("join") == "add" else 4 * int(params["hidden_size"])
         for side in ("left", "right"):
             hook = getattr(lookup(MIXERS, params[side]["kind"], "mixer"), "activation_elements", None)
             total += int(hook(params[side]["params"])) if hook is not None else 4 * int(params["hidden_size"])
@@ -52,6 +59,10 @@ class MixerPair:
 
     def forward(self, ctx, x, residual, cache_id, writes_cache, position):
         x = x.tensor() if hasattr(x, "tensor") else x
+        if self.join == "add":
+            for side, mixer, wants_position in self.halves:
+                mixer.forward(ctx, x, residual, (cache_id, side), writes_cache, position if wants_position else None)
+            return
         outs = []
         for side, mixer, wants_position in self.halves:
             # a half adds into what it is given: a zeroed stream of its own

@@ -30,6 +30,12 @@ previous token's input, m_s = h_t + (h_(t-1) - h_t) * mu_s:
     S_t = (1 - z) S_(t-1) + z cand                                   S_(-1) = 0
     result = out_scale * Wo (S_t * silu(Wg h))
 
+``hgrn2`` (a matrix state per head whose forget gate also says what is written), with q, z, v = Wq h, Wf h, Wv h:
+
+    f = l + (1 - l) sigmoid(z + b)                     per head and key channel, l the stored lower bound
+    S_t = diag(f) S_(t-1) + (1 - f) v^T,      o = S_t^T silu(q)                                S_(-1) = 0
+    result = out_scale * Wo [rms(o_head) * norm]       norm [vdim], one vector for all heads
+
 Decays, gates of the recurrences, unit keys, the states and o are float32 whatever the activation type; the
 matrix products and the convolution run in the activation type.
 """
@@ -281,4 +287,56 @@ class MinGRU:
         k.linear(x, self.w_in, proj)
         y = torch.empty((T, self.C), dtype=self.dtype, device=dev)
         k.mingru_scan(proj, self.z_bias, self.x_bias, ctx.cache.state(cache_id), ctx.batch, y, self.C, self.out_scale)
+        k.linear(y, self.w_o, residual, accumulate=True)
+
+
+@register_mixer("hgrn2")
+class Hgrn2:
+    """params: ``hidden_size``, ``num_heads``, ``dim``, ``value_dim``, ``norm_eps``, ``out_scale`` (1.0: folded into the norm's
+    weight, in float32); weights: ``q``, ``f``, ``v``, ``f_bias`` [heads x dim], ``lower`` [heads x dim], ``norm``
+    [value_dim], ``o``.  The three input products run as one over [q | f | v]."""
+
+    takes_lazy_input = True
+
+    def __init__(self, params, weights, build: BuildContext):
+        self.hidden, self.H = int(params["hidden_size"]), int(params["num_heads"])
+        self.dim, self.vdim, self.eps = int(params["dim"]), int(params["value_dim"]), float(params["norm_eps"])
+        self.out_scale = float(params.get("out_scale", 1.0))
+        from ..csrc.ops import SCAN_MAX_DIM
+        if self.dim > SCAN_MAX_DIM:
+            raise ValueError(f"hgrn2: {self.dim} key channels a head; the recurrence kernel holds up to {SCAN_MAX_DIM}")
+        w, dt = build.weights, build.dtype
+        HD, HV = self.H * self.dim, self.H * self.vdim
+        got = {r: w.as_dtype(weights[r], dt) for r in ("q", "f", "v", "o")}
+        got.update({r: w.stored(weights[r]).float().contiguous() for r in ("f_bias", "lower", "norm")})
+        _shapes(got, {"q": (HD, self.hidden), "f": (HD, self.hidden), "v": (HV, self.hidden), "o": (self.hidden, HV),
+                      "f_bias": (HD,), "lower": (HD,), "norm": (self.vdim,)}, weights)
+        self.w_in = torch.cat([got["q"], got["f"], got["v"]], dim=0).contiguous()
+        self.w_o, self.f_bias, self.lower = got["o"], got["f_bias"], got["lower"]
+        self.norm_w = (got["norm"] * self.out_scale).contiguous()
+        self.q_off, self.f_off, self.v_off = 0, HD, 2 * HD
+        self.dtype = dt
+
+    def cache_need(self):
+        return StateNeed(self.H * self.dim * self.vdim)
+
+    @staticmethod
+    def cache_need_from(params):
+        return StateNeed(int(params["num_heads"]) * int(params["dim"]) * int(params["value_dim"]))
+
+    @staticmethod
+    def activation_elements(params) -> int:
+        """The projected row, o (float32: counted twice) and the normed output."""
+        H, d, dv = int(params["num_heads"]), int(params["dim"]), int(params["value_dim"])
+        return 2 * H * d + 4 * H * dv
+
+    def forward(self, ctx, x, residual, cache_id, writes_cache, position):
+        if not writes_cache:
+            raise ValueError("a recurrent mixer cannot read another layer's state without advancing it")
+        T, dev, k = ctx.batch.n_tokens, residual.device, ctx.kernels
+        proj = torch.empty((T, self.w_in.shape[0]), dtype=self.dtype, device=dev)
+        k.linear(x, self.w_in, proj)
+        y = torch.empty((T, self.H * self.vdim), dtype=self.dtype, device=dev)
+        k.tied_scan(proj, self.q_off, self.f_off, self.v_off, self.f_bias, self.lower, ctx.cache.state(cache_id), ctx.batch,
+                    self.norm_w, self.eps, y, self.H, self.dim, self.vdim)
         k.linear(y, self.w_o, residual, accumulate=True)

@@ -18,14 +18,23 @@ A token that has left the window while its run is not yet wholly before it is no
 of q and of k with a plain weight: per head over ``dim`` with one weight vector for all heads (``"head"``), or over
 the whole projection of all heads at once with a weight of that size (``"row"``).  ``rot`` turns the first
 coordinates of q and k (the position encoding of the block); ``vrot`` turns every value over its whole width by
-its own position, so that a value enters a head's sum by its distance to the query.  ``sink``: a key of score 0
-that has no value (exp(0) = 1 is added to the denominator).  Scores, weights, norms and rotations are float32.
+its own position, so that a value enters a head's sum by its distance to the query.  ``sink`` (True): a key of score 0
+that has no value (exp(0) = 1 is added to the denominator); ``"learned"``: a key per head with the stored score sink_g,
+to which nothing of the above is done, and no value.  Scores, weights, norms and rotations are float32.
 
 Further options, each usable without the others:
 
 * ``conv`` = taps: a short causal convolution over time on every channel of the projected q and k, straight behind
   the projection and before the norm, y_t = sum_j w[:, j] u_(t - taps + 1 + j) with zeros before the sequence's
-  start; the last taps - 1 projected rows are per-sequence state beside the keys.
+  start; the last taps - 1 projected rows are per-sequence state beside the keys.  With ``conv_values`` the projected
+  v passes one too.
+* ``head_scale``: head g's scores are multiplied by a stored number temp_g, besides ``scale``.
+* ``distance_bias`` = ``"geometric"``: slope_g (p - j) is taken off the score of key j, slope_g = 2^(-8 (g + 1) / H).
+* ``value_mix`` = ``"first"`` or ``"later"``: in a layer that mixes, v <- (1 - lambda) v + lambda v_first before it is cached,
+  with lambda the layer's stored number and v_first the same token's values in the layer marked ``"first"``, as that
+  layer projected them.  Nothing of it is kept from step to step: a later layer needs the values of the step's own
+  tokens alone.
+* ``element_gate``: the concatenated heads are multiplied by sigmoid(Wg h) element by element.
 * ``values`` = ``"keys"``: there is no value projection; a token's value is its key as it leaves the projection (and
   the convolution), before the norm.
 * ``query_temperature`` = {coef, every}: the queries at position p are multiplied by
@@ -56,12 +65,16 @@ from .registry import POSITION_ENCODINGS, BuildContext, lookup, register_mixer
 @register_mixer("window_attention")
 class WindowAttention:
     """params: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``dim``, ``value_dim``, ``scale``, ``window`` (None: all
-    earlier tokens), ``keep_first`` (0), ``pool`` (0: no pooled runs), ``softcap`` (None), ``sink`` (False),
+    earlier tokens), ``keep_first`` (0), ``pool`` (0: no pooled runs), ``softcap`` (None), ``sink`` (False, True or
+    ``"learned"``),
     ``qk_norm`` (``"head"``, ``"row"`` or None), ``norm_eps``, ``value_rotation`` (None, or ``{"theta", "pairing"}``),
     ``out_scale`` (1.0), ``conv`` (0), ``values`` (``"projection"`` or ``"keys"``), ``query_temperature`` (None),
-    ``head_gate`` (False), ``score_maps`` (1 or 2), ``map_offset``, ``own_kv`` (True), ``cache_window``; weights: ``q``,
-    ``k``, ``v``, ``o``, with a norm ``q_norm``, ``k_norm``, with a convolution ``q_conv``, ``k_conv`` [channels, taps],
-    with a gate ``g`` [heads, hidden], with two maps ``lq1``, ``lk1``, ``lq2``, ``lk2`` [dim]."""
+    ``head_gate`` (False), ``element_gate`` (False), ``score_maps`` (1 or 2), ``map_offset``, ``own_kv`` (True),
+    ``cache_window``, ``conv_values`` (False), ``head_scale`` (False), ``distance_bias`` (None), ``value_mix`` (None); weights:
+    ``q``, ``k``, ``v``, ``o``, with a norm ``q_norm``, ``k_norm``, with a convolution ``q_conv``, ``k_conv`` (and ``v_conv``)
+    [channels, taps], with a gate ``g`` [heads, hidden] or [heads x value_dim, hidden], with two maps ``lq1``, ``lk1``,
+    ``lq2``, ``lk2`` [dim], with learned sinks ``sink`` [heads], with a head scale ``temp`` [heads], mixing values of an
+    earlier layer ``vmix`` (one number)."""
 
     def __init__(self, params, weights, build: BuildContext):
         self.hidden = int(params["hidden_size"])
@@ -71,7 +84,9 @@ class WindowAttention:
         self.window = int(params["window"]) if params.get("window") else None
         self.keep_first, self.pool = int(params.get("keep_first") or 0), int(params.get("pool") or 0)
         self.softcap = float(params["softcap"]) if params.get("softcap") else None
-        self.sink = bool(params.get("sink", False))
+        self.sink = params.get("sink", False)
+        if self.sink not in (False, True, "learned", None):
+            raise ValueError(f"window_attention: sink {self.sink!r} is not known (False, True or 'learned')")
         self.qk_norm = params.get("qk_norm")
         self.out_scale = float(params.get("out_scale", 1.0))
         self.taps = int(params.get("conv") or 0)
@@ -79,6 +94,9 @@ class WindowAttention:
         self.maps = int(params.get("score_maps") or 1)
         self.own_kv = bool(params.get("own_kv", True))
         self.head_gate = bool(params.get("head_gate", False))
+        self.element_gate = bool(params.get("element_gate", False))
+        self.conv_values = bool(params.get("conv_values", False))
+        self.value_mix = params.get("value_mix")
         qt = params.get("query_temperature")
         self.q_temp = (float(qt["coef"]), int(qt["every"])) if qt else None
         self.cache_window = self._reach(self.window, params.get("cache_window"))
@@ -92,8 +110,19 @@ class WindowAttention:
             raise ValueError(f"window_attention: values {self.values!r} is not known ('projection' or 'keys')")
         if self.values == "keys" and (self.vdim != self.dim or self.maps != 1):
             raise ValueError("window_attention: values that are the keys have the keys' width, and one score map")
-        if self.maps not in (1, 2) or (self.maps == 2 and (self.pool or self.qk_norm == "row" or self.sink or self.head_gate)):
-            raise ValueError("window_attention: one score map, or two without pooled runs, row norms, a sink or a head gate")
+        per_head = self.head_gate or self.element_gate or params.get("head_scale") or params.get("distance_bias")
+        if self.maps not in (1, 2) or (self.maps == 2 and (self.pool or self.qk_norm == "row" or self.sink or per_head)):
+            raise ValueError("window_attention: one score map, or two without pooled runs, row norms, a sink, a gate, a scale "
+                             "or a bias per head")
+        if self.head_gate and self.element_gate:
+            raise ValueError("window_attention: one gate per head or one per element, not both")
+        if self.conv_values and (not self.taps or self.values == "keys"):
+            raise ValueError("window_attention: convolved values are a projection of their own beside convolved q and k")
+        if self.value_mix not in (None, "first", "later") or (self.value_mix and (not self.own_kv or self.values == "keys")):
+            raise ValueError(f"window_attention: value_mix {self.value_mix!r} ('first' or 'later', for layers with a value "
+                             "projection of their own)")
+        if params.get("distance_bias") not in (None, "geometric") or (params.get("distance_bias") and self.pool):
+            raise ValueError(f"window_attention: distance_bias {params.get('distance_bias')!r} ('geometric', without pooled runs)")
         if self.taps < 0 or (self.taps and not self.own_kv):
             raise ValueError("window_attention: a convolution needs keys of its own behind it")
         if self.q_temp and self.q_temp[1] < 1:
@@ -103,7 +132,7 @@ class WindowAttention:
         q = w.as_dtype(weights["q"], dt)
         self.w_o = w.as_dtype(weights["o"], dt)
         want = {"q": (H * M * D, self.hidden), "k": (G * M * D, self.hidden), "v": (G * V, self.hidden),
-                "o": (self.hidden, H * V), "g": (H, self.hidden)}
+                "o": (self.hidden, H * V), "g": (H * V if self.element_gate else H, self.hidden)}
 
         def checked(role, t):
             if tuple(t.shape) != want[role]:
@@ -122,9 +151,9 @@ class WindowAttention:
                 rows.append(checked("v", w.as_dtype(weights["v"], dt)))
         self.kv_cols = sum(r.shape[0] for r in rows[1:])
         gate_rows = []
-        if self.head_gate:
+        if self.head_gate or self.element_gate:
             g = checked("g", w.as_dtype(weights["g"], dt))
-            pad = (-H) % 8                   # rows of the projection's result stay a multiple of 8 wide
+            pad = (-g.shape[0]) % 8          # rows of the projection's result stay a multiple of 8 wide
             gate_rows = [g] + ([torch.zeros((pad, self.hidden), dtype=dt, device=g.device)] if pad else [])
         self.gate_cols = sum(r.shape[0] for r in gate_rows)
         # [q | k | v | gate]; a stop that does not write the cache projects [q | gate] only
@@ -153,7 +182,29 @@ class WindowAttention:
             if tuple(cq.shape) != (H * M * D, self.taps) or tuple(ck.shape) != (G * M * D, self.taps):
                 raise ValueError(f"{weights['q_conv']} / {weights['k_conv']}: expected [{H * M * D}, {self.taps}] and "
                                  f"[{G * M * D}, {self.taps}]")
-            self.conv_w = torch.cat([cq, ck], dim=0).contiguous()
+            convs = [cq, ck]
+            if self.conv_values:
+                convs.append(w.stored(weights["v_conv"]).float())
+                if tuple(convs[2].shape) != (G * V, self.taps):
+                    raise ValueError(f"{weights['v_conv']}: expected [{G * V}, {self.taps}]")
+            self.conv_w = torch.cat(convs, dim=0).contiguous()
+
+        def per_query_head(role):
+            t = w.stored(weights[role]).float().contiguous()
+            if tuple(t.shape) != (H,):
+                raise ValueError(f"{weights[role]} has shape {tuple(t.shape)}, expected ({H},)")
+            return t
+        self.sinks = per_query_head("sink") if self.sink == "learned" else True if self.sink else None
+        self.head_mul = per_query_head("temp") if params.get("head_scale") else None
+        self.slopes = None
+        if params.get("distance_bias"):
+            self.slopes = torch.tensor([2.0 ** (-8.0 * (g + 1) / H) for g in range(H)], dtype=torch.float64).float().to(build.device)
+        self.mix_share = None
+        if self.value_mix == "later":
+            lam = w.stored(weights["vmix"]).float().reshape(-1)
+            if lam.numel() != 1:
+                raise ValueError(f"{weights['vmix']} has {lam.numel()} values, expected one")
+            self.mix_share = float(lam[0])
         self.lam = None
         if M == 2:
             lq1, lk1, lq2, lk2 = (w.stored(weights[r]).double().cpu() for r in ("lq1", "lk1", "lq2", "lk2"))
@@ -194,7 +245,11 @@ class WindowAttention:
 
     def cache_need(self):
         return self._needs(self.n_kv, self.dim, self.vdim, self.cache_window, self.keep_first, self.pool, self.maps,
-                           self.taps, (self.n_q + self.n_kv) * self.maps * self.dim)
+                           self.taps, self._conv_channels(self.n_q, self.n_kv, self.maps, self.dim, self.vdim, self.conv_values))
+
+    @staticmethod
+    def _conv_channels(n_q, n_kv, maps, dim, vdim, conv_values):
+        return (n_q + n_kv) * maps * dim + (n_kv * vdim if conv_values else 0)
 
     @staticmethod
     def cache_need_from(params):
@@ -202,14 +257,17 @@ class WindowAttention:
         H, G, D = int(params["num_heads"]), int(params["num_kv_heads"]), int(params["dim"])
         return WindowAttention._needs(G, D, int(params["value_dim"]),
                                       WindowAttention._reach(params.get("window"), params.get("cache_window")),
-                                      params.get("keep_first"), params.get("pool"), maps, taps, (H + G) * maps * D)
+                                      params.get("keep_first"), params.get("pool"), maps, taps,
+                                      WindowAttention._conv_channels(H, G, maps, D, int(params["value_dim"]),
+                                                                     bool(params.get("conv_values"))))
 
     @staticmethod
     def activation_elements(params) -> int:
         H, G = int(params["num_heads"]), int(params["num_kv_heads"])
         maps = int(params.get("score_maps") or 1)
         conv = 2 if params.get("conv") else 1
-        return conv * (H + G) * maps * int(params["dim"]) + (H * maps + G) * int(params["value_dim"]) + 2 * H
+        gates = H * int(params["value_dim"]) if params.get("element_gate") else 2 * H
+        return conv * (H + G) * maps * int(params["dim"]) + (H * maps + conv * G) * int(params["value_dim"]) + gates
 
     def _read_weight(self):
         """[q | gate] for a stop that reads another stop's keys."""
@@ -244,18 +302,29 @@ class WindowAttention:
                           pass_cols=qkv.shape[1] - self.conv_w.shape[0])
             qkv = conv
         v_off = q_cols if self.values == "keys" else None
+        v_mix = None
+        if self.value_mix == "first":
+            # the values as projected (and convolved): the preparation below writes them to the cache, not over the row
+            ctx.carried["first_values"] = qkv[:, q_cols + G * M * D: q_cols + G * M * D + G * V]
+        elif self.value_mix == "later":
+            first = ctx.carried.get("first_values")
+            if first is None or first.shape != (T, G * V):
+                raise RuntimeError("window_attention: a layer that mixes values runs behind the layer whose values it mixes in, "
+                                   "and has as many of them")
+            v_mix = (first, self.mix_share)
         pooled_there = k.qkv_prepare(qkv, self.q_norm, self.k_norm, self.qk_norm, self.eps, position, self.value_position, kv,
                                      ctx.batch, H * M, G * M, D, V, PAGE_SHIFT, writes_cache,
                                      pooled_kv=pooled if writes_cache else None, pool=self.pool, v_off=v_off,
-                                     q_temp=self.q_temp, n_v=G)
+                                     q_temp=self.q_temp, n_v=G, v_mix=v_mix)
         if self.pool and writes_cache and not pooled_there:
             k.pool_rows(kv, pooled, ctx.batch, G, D, V, PAGE_SHIFT, self.pool)
-        gate = qkv[:, q_cols + kv_cols: q_cols + kv_cols + H] if self.head_gate else None
+        n_gates = H * V if self.element_gate else H if self.head_gate else 0
+        gate = qkv[:, q_cols + kv_cols: q_cols + kv_cols + n_gates] if n_gates else None
         heads = torch.empty((T, H * M * V), dtype=self.dtype, device=dev)
         k.window_attention(qkv, kv, pooled, ctx.batch, heads, H * M, G * M, D, V, PAGE_SHIFT,
                            self.window, self.keep_first, self.pool, self.scale, self.softcap,
-                           True if self.sink else None, self.value_position, self.out_scale if M == 1 else 1.0,
-                           v_share=M, gate=gate)
+                           self.sinks, self.value_position, self.out_scale if M == 1 else 1.0, v_share=M, gate=gate,
+                           gate_elems=self.element_gate, slopes=self.slopes, head_mul=self.head_mul)
         if M > 1:
             merged = torch.empty((T, H * V), dtype=self.dtype, device=dev)
             k.map_difference(heads, merged, H, G, V, self.lam, self.eps, (1.0 - self.map_offset) * self.out_scale)
