@@ -397,6 +397,34 @@ def _kilisun_sizes(name):
     return kil, ron
 
 
+def _ruzunex_sizes(name):
+    """(Ruzunex config.json, the Kilisun configuration of the same width, layer count, vocabulary and experts: the
+    closest existing design, whose window attention, convolution, gated units and experts run on the same kernels).  Two
+    window layers, one with a dense feed-forward and one with experts, and two layers of attention beside a recurrence
+    with experts; two residual streams."""
+    def window(heads, kv, dim, vdim, size):
+        return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": dim ** -0.5,
+                                               "mask": {"size": size}, "v_mix": True}}
+
+    def both(heads, kv, dim, right):
+        return {"type": "parallel", "mixer": {
+            "left": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "conv": 4,
+                     "rot": {"base": 500000.0, "dims": dim}},
+            "right": {"heads": right[0], "dim": right[1], "vdim": right[2]}, "left_scale": 0.5, "right_scale": 0.5}}
+    kil, _ = _kilisun_sizes(name)
+    width, ff = kil["width"], kil["layers"][0]["mlp"]["ff"]
+    theirs = kil["layers"][1]["mlp"]
+    experts = {"kind": "moe", "expert": dict(theirs["expert"]), "router": {k: theirs["router"][k] for k in ("experts", "top")}}
+    if name == "2048":
+        mixers = [window(16, 4, 64, 128, 512)] * 2 + [both(16, 4, 128, (16, 128, 128))] * 2
+    else:
+        mixers = [window(8, 2, 64, 128, 256)] * 2 + [both(8, 2, 128, (8, 128, 128))] * 2
+    layers = [dict(mixers[0], mlp={"kind": "dense", "ff": ff})] + [dict(m, mlp=experts) for m in mixers[1:]]
+    ruz = {"architecture": "Ruzunex", "vocab": kil["vocab"], "width": width, "norm": {"eps": 1e-5}, "canon": {"taps": 4},
+           "streams": 2, "layers": layers}
+    return ruz, kil
+
+
 def _operation_work(model, tokens):
     """Algorithmic work of one prompt of ``tokens`` tokens per operation of the model's parts: (FLOPs, bytes).
     Matrix products count 2 per multiply-add; attention counts its scores and weighted sums over the causal
@@ -407,6 +435,22 @@ def _operation_work(model, tokens):
         f, b = work.get(name, (0, 0))
         work[name] = (f + flops, b + nbytes)
     T, causal = tokens, tokens * (tokens + 1) // 2
+
+    def window_work(m):
+        maps = getattr(m, "maps", 1)
+        w_in = m.w_qkv if getattr(m, "own_kv", True) else m._read_weight()
+        add("mixer.linear", 2 * T * (w_in.numel() + m.w_o.numel()))
+        w = int(m.window or T)
+        pairs = sum(min(i + 1, w) + (max(0, i - w + 1) // m.pool if m.pool else min(m.keep_first, max(0, i - w + 1)))
+                    for i in range(T))
+        add("mixer.window_attention", 2 * pairs * m.n_q * maps * (m.dim + m.vdim))
+        kv_rows = m.n_kv * (maps * m.dim + m.vdim) if getattr(m, "own_kv", True) else 0
+        add("mixer.qkv_prepare", 0, T * (m.n_q * maps * m.dim * 4 + kv_rows * 4))
+        if getattr(m, "taps", 0):
+            C = m.conv_w.shape[0]
+            add("mixer.causal_conv", 2 * T * C * m.taps, T * w_in.shape[0] * 4)
+        if maps > 1:
+            add("mixer.map_difference", 0, T * m.n_q * m.vdim * (2 * maps + 2))
     # a block runs once per stop of the schedule: a layer that runs with another's weights is a second stop there
     for b in [model.blocks[stop.layer] for stop in model.spec.schedule]:
         m, ff = b.mixer, b.feed_forward
@@ -433,6 +477,13 @@ def _operation_work(model, tokens):
         elif kind == "MixerPair":
             for _, half, _ in m.halves:
                 hk = type(half).__name__
+                if hk == "WindowAttention":
+                    window_work(half)
+                if hk == "Hgrn2":
+                    add("mixer.linear", 2 * T * (half.w_in.numel() + half.w_o.numel()))
+                    # per state element and token: v - s, its multiply-add, the sum S^T q; q, z, v in 16 bits, o out in 16
+                    add("mixer.tied_scan", 5 * T * half.H * half.dim * half.vdim,
+                        T * half.H * (2 * (2 * half.dim + half.vdim) + 2 * half.vdim))
                 if hk == "SigmoidAttention":
                     add("mixer.linear", 2 * T * (half.w_qkv.numel() + half.w_o.numel()))
                     c = int(half.chunk or T)
@@ -443,20 +494,7 @@ def _operation_work(model, tokens):
                     add("mixer.linear", 2 * T * (sum(w.numel() for w in half.w) + half.w2.numel() + half.w_o.numel()))
                     add("mixer.matrix_state_scan", 6 * T * HD * half.dim, T * HD * (3 * 2 + 4 + 4))
         elif kind == "WindowAttention":
-            maps = getattr(m, "maps", 1)
-            w_in = m.w_qkv if getattr(m, "own_kv", True) else m._read_weight()
-            add("mixer.linear", 2 * T * (w_in.numel() + m.w_o.numel()))
-            w = int(m.window or T)
-            pairs = sum(min(i + 1, w) + (max(0, i - w + 1) // m.pool if m.pool else min(m.keep_first, max(0, i - w + 1)))
-                        for i in range(T))
-            add("mixer.window_attention", 2 * pairs * m.n_q * maps * (m.dim + m.vdim))
-            kv_rows = m.n_kv * (maps * m.dim + m.vdim) if getattr(m, "own_kv", True) else 0
-            add("mixer.qkv_prepare", 0, T * (m.n_q * maps * m.dim * 4 + kv_rows * 4))
-            if getattr(m, "taps", 0):
-                C = m.conv_w.shape[0]
-                add("mixer.causal_conv", 2 * T * C * m.taps, T * w_in.shape[0] * 4)
-            if maps > 1:
-                add("mixer.map_difference", 0, T * m.n_q * m.vdim * (2 * maps + 2))
+            window_work(m)
         elif kind == "MinGRU":
             add("mixer.linear", 2 * T * (m.w_in.numel() + m.w_o.numel()))
             add("mixer.mingru_scan", 10 * T * m.C, T * m.C * (3 * 2 + 2))                # z, x, g in; the gated state out
@@ -469,6 +507,12 @@ def _operation_work(model, tokens):
             # behind each sublayer: the float32 branch in, zeros back, the stream in and out; once with the next norm's rows out
             W = model.spec.hidden_size
             add("feed_forward.rms_add", 0, T * W * ((4 * 4 + 2) + (4 * 4 if ff is not None else 0)))
+        if type(b).__name__ == "HyperConnectionBlock":
+            # a sublayer's entry: the streams and the branch in, the streams and zeros out, the normed and convolved row out
+            W, S = model.spec.hidden_size, b.streams
+            add("mixer.stream_enter", 0, T * W * (4 * (2 * S + 2) + 2))
+            if ff is not None:
+                add("feed_forward.stream_enter", 0, T * W * (4 * (2 * S + 2) + 2))
         if fk == "Experts":
             per = ff.w_gate_up[0].numel() + ff.w_down[0].numel()
             add("feed_forward.expert_gate_up", 2 * T * ff.top * ff.w_gate_up[0].numel())
@@ -497,11 +541,11 @@ def design_comparison(args):
     from supersonic_b200.weights import RandomWeightStore
     pk, pk_src = peaks()
     sizes = {"vufadra": _vufadra_sizes, "sotavik": _sotavik_sizes, "ronelorn": _ronelorn_sizes,
-             "kilisun": _kilisun_sizes}[args.design]
+             "kilisun": _kilisun_sizes, "ruzunex": _ruzunex_sizes}[args.design]
     sot, lla = sizes(args.design_size)
-    beside = {"ronelorn": "vufadra", "kilisun": "ronelorn"}.get(args.design, "llama")
+    beside = {"ronelorn": "vufadra", "kilisun": "ronelorn", "ruzunex": "kilisun"}.get(args.design, "llama")
     models = [(args.design, sot), (beside, lla)]
-    if args.design == "kilisun":                              # its experts beside the design whose expert products they run on
+    if args.design in ("kilisun", "ruzunex"):                              # its experts beside the design whose expert products they run on
         models.append(("sotavik", _sotavik_sizes(args.design_size)[0]))
     out = {"metric": "design_comparison", "design": args.design, "beside": beside, "size": args.design_size,
            "layers": len(sot["layers"]), "dtype": "bf16", "data": "synthetic", "peaks": pk, "peaks_source": pk_src,
@@ -676,7 +720,7 @@ def main():
                     help="also time decode and prompts at further sizes (adds a 'sweep' key to the line)")
     ap.add_argument("--deterministic", action="store_true",
                     help="time the bfloat16 path without float atomics and with one kernel choice whatever the batch")
-    ap.add_argument("--design", default=None, choices=["sotavik", "vufadra", "ronelorn", "kilisun"],
+    ap.add_argument("--design", default=None, choices=["sotavik", "vufadra", "ronelorn", "kilisun", "ruzunex"],
                     help="instead of the headline workload: this design beside the closest existing model at equal size")
     ap.add_argument("--design-size", default="2048", help="width of the compared models: 1024 or 2048")
     args = ap.parse_args()

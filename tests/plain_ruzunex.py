@@ -77,8 +77,8 @@ def weighted_sum(scores, values, sink=None):
 
 
 def mixed_values(v, first, lam):
-    """The values of a mixing layer behind the first one."""
-    return (1.0 - lam) * v + lam * first
+    """The values of a mixing layer behind the first one (element by element of a token's values, whatever the heads)."""
+    return (1.0 - lam) * v + lam * first.reshape(v.shape)
 
 
 def biased_attention(h, weights, p, m, eps, first_values=None):
