@@ -361,6 +361,51 @@ def norm_add(args):
             "GB/s": round(nbytes / us / 1e3, 1)}
 
 
+def stream_cross(args):
+    """The pass between two sublayers over --maps residual streams: write the waiting branch, read, norm (zeroing the
+    branch behind the read): --rows tokens of width --n."""
+    T, Wd, S = args.rows, args.n, max(args.maps, 2)
+    xs = [torch.randn(S, T, Wd, device=DEV) for _ in range(4)]        # four sets in turn: larger than L2 at real sizes
+    br = [torch.randn(T, Wd, device=DEV) for _ in range(4)]
+    mix, o, i_, w = torch.eye(S, device=DEV), torch.ones(S, device=DEV), torch.ones(S, device=DEV), torch.ones(Wd, device=DEV)
+    out = torch.empty(T, Wd, device=DEV, dtype=torch.bfloat16)
+    us = _time(lambda i: ops.stream_cross(xs[i % 4], S, i_, out, br[i % 4], mix, o, xs[i % 4], True, w, 1e-6), args.iters)
+    return {"kernel": "stream_cross", "rows": T, "width": Wd, "streams": S, "us": round(us, 2),
+            "GB/s": round(T * Wd * (4 * (2 * S + 2) + 2) / us / 1e3, 1)}
+
+
+def causal_conv(args):
+    """A short convolution of --keep taps (default 4) over --rows bfloat16 rows of --n channels, one sequence."""
+    T, C, taps = args.rows, args.n, args.keep or 4
+    x = [torch.randn(T, C, device=DEV).bfloat16() for _ in range(8)]
+    w, tail = torch.randn(C, taps, device=DEV), torch.zeros(2, (taps - 1) * C, device=DEV)
+    cu, slots = torch.tensor([0, T], dtype=torch.int32, device=DEV), torch.ones(1, dtype=torch.int32, device=DEV)
+    out = torch.empty(T, C, device=DEV, dtype=torch.bfloat16)
+    us = _time(lambda i: ops.causal_conv(x[i % 8], None, w, None, tail, cu, slots, out, T), args.iters)
+    return {"kernel": "causal_conv", "rows": T, "channels": C, "taps": taps, "us": round(us, 2), "GB/s": round(4 * T * C / us / 1e3, 1)}
+
+
+def tied_scan(args):
+    """The recurrence whose gate also says what is written: --heads heads of --head-dim x --vdim (default: --head-dim) over
+    --seqs prompts of --tokens tokens, with the head norm; --chunk 0: one walk, -1: chunks as the kernel set picks them."""
+    H, d, T, B = args.heads, args.head_dim, args.tokens, args.seqs
+    dv = args.vdim or d
+    proj = torch.randn(B * T, H * (2 * d + dv), device=DEV).bfloat16()
+    bias, low, w = torch.randn(H * d, device=DEV), torch.rand(H * d, device=DEV), torch.ones(dv, device=DEV)
+    state = torch.zeros(B + 1, H * d * dv, device=DEV)
+    cu = torch.arange(0, (B + 1) * T, T, dtype=torch.int32, device=DEV)
+    slots = torch.arange(1, B + 1, dtype=torch.int32, device=DEV)
+    out = torch.empty(B * T, H * dv, device=DEV, dtype=torch.bfloat16)
+    chunk = ops.tied_scan_chunking(B, T, H, d, dv, ops.sm_count())[0] if args.chunk < 0 else args.chunk
+    n = -(-T // chunk) if chunk else 0
+    sums = torch.empty(max(B * n * H * d * dv, 1), device=DEV)
+    decays = torch.empty(max(B * n * H * d, 1), device=DEV)
+    us = _time(lambda i: ops.tied_scan(proj, 0, H * d, 2 * H * d, bias, low, state, cu, slots, out, H, d, dv, norm_w=w, eps=1e-6,
+                                       chunk=chunk, max_new=T, sums=sums, decays=decays), args.iters)
+    return {"kernel": "tied_scan", "seqs": B, "tokens": T, "heads": H, "dim": d, "vdim": dv, "chunk": chunk, "us": round(us, 2),
+            "TFLOP/s": round(5.0 * B * T * H * d * dv / us / 1e6, 2)}
+
+
 def mingru_scan(args):
     """minGRU over --seqs prompts of --tokens tokens and --n channels: --kernel walk, tiled or chunked."""
     C, T, B = args.n, args.tokens, args.seqs
@@ -400,7 +445,7 @@ def main(argv=None):
     sub = ap.add_subparsers(dest="what", required=True)
     for name in ("attention_decode", "linear", "gemm", "attention_prefill", "sampling", "latent_attention", "grouped_gemm",
                  "gated_linear_scan", "matrix_state_scan", "gated_unit_scan", "sigmoid_attention", "window_attention",
-                 "mingru_scan", "norm_add"):
+                 "mingru_scan", "norm_add", "stream_cross", "causal_conv", "tied_scan"):
         p = sub.add_parser(name)
         p.add_argument("--iters", type=int, default=20)
         p.add_argument("--heads", type=int, default=32)

@@ -396,6 +396,11 @@ class FastKernels(PlainKernels):
     def _scan_scratch(self, n, device):
         return self._buffer("unit_scan_chunks", n, torch.float32, device)
 
+    def _tied_chunking(self, batch, n_heads, dim, vdim):
+        if self.deterministic:                 # chunks of one length whatever else is in the step
+            return ops.scan_chunking(batch.n_seqs, batch.max_new, n_heads, dim, vdim)
+        return super()._tied_chunking(batch, n_heads, dim, vdim)
+
     def matrix_state_step(self, proj, r_off, k_off, v_off, g_off, a_off, z, z_bias, decay_kind, decay_scale, a_bias,
                           unit_eps, kind, bonus, state, batch, norm_w, eps, gate_kind, y, n_heads, dim, vdim) -> bool:
         if not (batch.is_decode and proj.dtype == torch.bfloat16 and norm_w.dtype == torch.bfloat16

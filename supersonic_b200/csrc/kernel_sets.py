@@ -192,15 +192,21 @@ class PlainKernels:
             ops.tied_step(proj, q_off, f_off, v_off, z_bias, lower, state, batch.cu_new, batch.seq_slot, norm_w, eps, y,
                           n_heads, dim, vdim, pdl=self._chain(batch.n_tokens))
             return
-        chunk, n_sums, n_decays = ops.scan_chunking(batch.n_seqs, batch.max_new, n_heads, dim, vdim)
+        chunk, n_sums, n_decays = self._tied_chunking(batch, n_heads, dim, vdim)
         sums = decays = None
         if chunk:                             # a long prompt: its chunks in parallel
             scratch = self._scan_scratch(n_sums + n_decays, y.device)
             sums, decays = scratch[:n_sums], scratch[n_sums: n_sums + n_decays]
-        o = torch.empty((batch.n_tokens, n_heads * vdim), dtype=torch.float32, device=y.device)
+        fused = vdim <= ops.tied_scan_cols(dim, vdim)
+        o = y if fused else torch.empty((batch.n_tokens, n_heads * vdim), dtype=torch.float32, device=y.device)
         ops.tied_scan(proj, q_off, f_off, v_off, z_bias, lower, state, batch.cu_new, batch.seq_slot, o, n_heads, dim, vdim,
-                      pdl=self._chain(batch.n_tokens), chunk=chunk, max_new=batch.max_new, sums=sums, decays=decays)
-        ops.head_norm_gate(o, norm_w, eps, None, y, n_heads, vdim, pdl=self._chain(batch.n_tokens))
+                      norm_w=norm_w if fused else None, eps=eps, pdl=self._chain(batch.n_tokens), chunk=chunk,
+                      max_new=batch.max_new, sums=sums, decays=decays)
+        if not fused:
+            ops.head_norm_gate(o, norm_w, eps, None, y, n_heads, vdim, pdl=self._chain(batch.n_tokens))
+
+    def _tied_chunking(self, batch, n_heads, dim, vdim):
+        return ops.tied_scan_chunking(batch.n_seqs, batch.max_new, n_heads, dim, vdim, ops.sm_count())
 
     def matrix_state_scan(self, proj, r_off, k_off, v_off, decay, kind, state, batch, out, n_heads, dim, vdim,
                           unit=None, bonus=None):

@@ -509,18 +509,41 @@ def _tied_args(proj, q_off, f_off, v_off, z_bias, lower, state, cu_new, seq_slot
         raise KernelError(f"{what}: sizes (state rows of heads x dim x vdim, dim up to {SCAN_MAX_DIM})")
 
 
+def tied_scan_cols(dim: int, vdim: int) -> int:
+    """Value columns a block of ``tied_scan`` holds; a head of no more takes the head norm along."""
+    return 64 if vdim <= 64 or dim > 128 else 128
+
+
+def tied_scan_chunking(n_seqs: int, max_new: int, n_heads: int, dim: int, vdim: int, sms: int):
+    """(chunk, floats of sums, floats of decays) for ``tied_scan``: as many chunks as fill the SMs with a block each, if
+    that is three or more (a chunked run walks every token twice); chunk 0: one walk a sequence."""
+    blocks = n_seqs * n_heads * (-(-vdim // tied_scan_cols(dim, vdim)))
+    per = n_heads * dim * vdim
+    n = min(sms // max(blocks, 1), max_new // 64, SCAN_SCRATCH_BYTES // (4 * per * n_seqs))
+    if n < 3:
+        return 0, 0, 0
+    chunk = -(-(-(-max_new // n)) // 8) * 8           # whole turns of eight tokens
+    n = -(-max_new // chunk)
+    return chunk, n_seqs * n * per, n_seqs * n * n_heads * dim
+
+
 def tied_scan(proj: torch.Tensor, q_off: int, f_off: int, v_off: int, z_bias: torch.Tensor, lower: torch.Tensor,
               state: torch.Tensor, cu_new: torch.Tensor, seq_slot: torch.Tensor, out: torch.Tensor, n_heads: int, dim: int,
-              vdim: int, pdl: bool = False, chunk: int = 0, max_new: int = 0, sums: Optional[torch.Tensor] = None,
-              decays: Optional[torch.Tensor] = None) -> None:
+              vdim: int, norm_w: Optional[torch.Tensor] = None, eps: float = 0.0, pdl: bool = False, chunk: int = 0,
+              max_new: int = 0, sums: Optional[torch.Tensor] = None, decays: Optional[torch.Tensor] = None) -> None:
     """Per sequence and head, over the sequence's new tokens in order, with the gate f = lower + (1 - lower) *
-    sigmoid(z + z_bias) per head and channel:  S = diag(f) S + (1 - f) v^T;  out = S^T silu(q).  q and z (heads x dim)
-    and v (heads x vdim) are columns of ``proj``; ``state``, ``chunk``, ``sums`` and ``decays`` as in ``gated_linear_scan``."""
+    sigmoid(z + z_bias) per head and channel:  S = diag(f) S + (1 - f) v^T;  o = S^T silu(q).  q and z (heads x dim)
+    and v (heads x vdim) are columns of ``proj``; ``state``, ``chunk``, ``sums`` and ``decays`` as in ``gated_linear_scan``.
+    ``out`` gets o (float32) or, with ``norm_w`` [vdim] (heads of up to ``tied_scan_cols`` values), o / rms(o) * norm_w per head."""
     _tied_args(proj, q_off, f_off, v_off, z_bias, lower, state, cu_new, seq_slot, n_heads, dim, vdim, "tied_scan")
-    _need(out, "out", torch.float32, 2)
+    _need(out, "out", proj.dtype if norm_w is not None else torch.float32, 2)
     T, B = proj.shape[0], seq_slot.shape[0]
     if out.shape[0] != T or out.shape[1] < n_heads * vdim:
         raise KernelError("tied_scan: one output row per token")
+    if norm_w is not None:
+        _need(norm_w, "norm_w", torch.float32, 1)
+        if norm_w.shape[0] != vdim or vdim > tied_scan_cols(dim, vdim):
+            raise KernelError(f"tied_scan: a norm weight per value column, heads of up to {tied_scan_cols(dim, vdim)}")
     max_chunks = 0
     if chunk > 0:
         max_chunks = -(-max_new // chunk)
@@ -530,8 +553,9 @@ def tied_scan(proj: torch.Tensor, q_off: int, f_off: int, v_off: int, z_bias: to
             raise KernelError("tied_scan: the scratch of the chunked run is too small")
     _check(_fn("recurrence_ops", "ssb_tied_scan")(
         _ptr(proj), c_int(proj.stride(0)), c_int(dtype_code(proj.dtype)), c_int(q_off), c_int(f_off), c_int(v_off),
-        _ptr(z_bias), _ptr(lower), _ptr(state), _ptr(cu_new), _ptr(seq_slot), _ptr(out), c_int(out.stride(0)), c_int(B),
-        c_int(T), c_int(n_heads), c_int(dim), c_int(vdim), c_int(chunk), c_int(max_chunks), _ptr(sums), _ptr(decays),
+        _ptr(z_bias), _ptr(lower), _ptr(state), _ptr(cu_new), _ptr(seq_slot), _ptr(None if norm_w is not None else out),
+        c_int(out.stride(0)), _ptr(norm_w), c_float(eps), _ptr(out if norm_w is not None else None), c_int(out.stride(0)),
+        c_int(B), c_int(T), c_int(n_heads), c_int(dim), c_int(vdim), c_int(chunk), c_int(max_chunks), _ptr(sums), _ptr(decays),
         c_int(1 if pdl else 0), _stream()), "tied_scan")
 
 

@@ -8,11 +8,6 @@
 // The scan walks a sequence's new tokens in order, from the state the sequence's slot holds, and
 // leaves the state there; a block owns a tile of value columns of one head of one sequence, so no
 // sum depends on what else is in the batch.
-//
-// Tied form (HGRN2): the forget gate f_t per key channel also says what is written,
-//     f_t = l + (1 - l) sigmoid(z_t),    S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T,    o_t = S_t^T silu(q_t)
-// walked as S <- S + k (v - S) with k = 1 - f = (1 - l) sigmoid(-z): a gate close to one loses nothing to the
-// rounding of 1 - f.
 #include "common.cuh"
 #include <math.h>
 #include <type_traits>
@@ -54,19 +49,13 @@ __global__ void decay_kernel(float* __restrict__ z, int ldz, const float* __rest
     *p = expf(log_sigmoid(*p + z_bias[c]) * inv_tau);
 }
 
-// The written share 1 - f of the tied form, from the gate's pre-activation (bias included) and the lower bound.
-__device__ __forceinline__ float tied_share(float z, float lower) { return (1.0f - lower) / (1.0f + expf(z)); }
-
-// TIED: k_off names the columns of the gate's pre-activation (bias z_bias, lower bounds `lower`, per head and channel),
-// z is not read, and q passes silu.
-template <typename T, bool TIED>
+template <typename T>
 __global__ void __launch_bounds__(SCAN_COLS * SCAN_GROUPS)
 gated_linear_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v_off,
                          const float* __restrict__ z, int ldz, float q_scale, float* __restrict__ state,
                          const int* __restrict__ cu_new, const int* __restrict__ seq_slot,
                          float* __restrict__ out, int ldo, int n_heads, int dim, int vdim,
-                         int chunk, int max_chunks, float* __restrict__ sums, float* __restrict__ decays,
-                         const float* __restrict__ z_bias, const float* __restrict__ lower) {
+                         int chunk, int max_chunks, float* __restrict__ sums, float* __restrict__ decays) {
     constexpr int NT = SCAN_COLS * SCAN_GROUPS;
     extern __shared__ __align__(16) float sm[];
     // rows per thread, a multiple of four: thread (g, j) owns rows g * rpt .. + rpt - 1 of column j, and reads
@@ -104,14 +93,11 @@ gated_linear_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
     // a turn stages SCAN_TOKENS tokens: item (token, channel) n * NT + tid of the turn is this thread's
     float zz[SCAN_ITEMS], kk[SCAN_ITEMS], qq[SCAN_ITEMS], vv = 0.f, a_prod = 1.f;
     int item_tt[SCAN_ITEMS], item_i[SCAN_ITEMS];         // the same in every turn: divided once
-    float item_bias[SCAN_ITEMS], item_low[SCAN_ITEMS];
 #pragma unroll
     for (int n = 0; n < SCAN_ITEMS; ++n) {
         const int item = n * NT + tid;
         item_tt[n] = item < SCAN_TOKENS * dim ? item / dim : SCAN_TOKENS;
         item_i[n] = item % dim;
-        item_bias[n] = TIED ? z_bias[h * dim + item_i[n]] : 0.f;
-        item_low[n] = TIED ? lower[h * dim + item_i[n]] : 0.f;
     }
     auto fetch = [&](int t) {
         const int n_tok = min(SCAN_TOKENS, t1 - t);
@@ -120,7 +106,7 @@ gated_linear_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
             const int tt = item_tt[n], i = item_i[n];
             if (tt < n_tok) {
                 const T* row = proj + (size_t)(t + tt) * ld;
-                zz[n] = TIED ? 0.f : z[(size_t)(t + tt) * ldz + h * dim + i];
+                zz[n] = z[(size_t)(t + tt) * ldz + h * dim + i];
                 kk[n] = ssb_to_float(row[k_off + h * dim + i]);
                 qq[n] = ssb_to_float(row[q_off + h * dim + i]);
             }
@@ -138,21 +124,16 @@ gated_linear_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
         for (int n = 0; n < SCAN_ITEMS; ++n) {
             const int tt = item_tt[n], i = item_i[n];
             if (tt < n_tok) {
-                if (TIED) {
-                    k_s[tt * dimp + i] = tied_share(kk[n] + item_bias[n], item_low[n]);
-                    q_s[tt * dimp + i] = qq[n] / (1.0f + expf(-qq[n])) * q_scale;
-                } else {
-                    a_s[tt * dimp + i] = zz[n];
-                    k_s[tt * dimp + i] = kk[n];
-                    q_s[tt * dimp + i] = qq[n] * q_scale;
-                }
+                a_s[tt * dimp + i] = zz[n];
+                k_s[tt * dimp + i] = kk[n];
+                q_s[tt * dimp + i] = qq[n] * q_scale;
             }
         }
         if (tid < SCAN_TOKENS * SCAN_COLS) v_s[tid] = vv;
         __syncthreads();
         if (t + SCAN_TOKENS < t1) fetch(t + SCAN_TOKENS);
         if (decays != nullptr && tid < dim)
-            for (int tt = 0; tt < n_tok; ++tt) a_prod *= TIED ? 1.0f - k_s[tt * dimp + tid] : a_s[tt * dimp + tid];
+            for (int tt = 0; tt < n_tok; ++tt) a_prod *= a_s[tt * dimp + tid];
         for (int tt = 0; tt < n_tok; ++tt) {
             const float v = v_s[tt * SCAN_COLS + j];
             const float4* a4 = reinterpret_cast<const float4*>(a_s + tt * dimp + g * rpt);
@@ -162,15 +143,7 @@ gated_linear_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_of
 #pragma unroll
             for (int r = 0; r < SCAN_MAX_ROWS; r += 4)
                 if (r < rpt) {
-                    const float4 k = k4[r >> 2], q = q4[r >> 2];
-                    if (TIED) {
-                        s_reg[r] = fmaf(k.x, v - s_reg[r], s_reg[r]);              o = fmaf(s_reg[r], q.x, o);
-                        s_reg[r + 1] = fmaf(k.y, v - s_reg[r + 1], s_reg[r + 1]);  o = fmaf(s_reg[r + 1], q.y, o);
-                        s_reg[r + 2] = fmaf(k.z, v - s_reg[r + 2], s_reg[r + 2]);  o = fmaf(s_reg[r + 2], q.z, o);
-                        s_reg[r + 3] = fmaf(k.w, v - s_reg[r + 3], s_reg[r + 3]);  o = fmaf(s_reg[r + 3], q.w, o);
-                        continue;
-                    }
-                    const float4 a = a4[r >> 2];
+                    const float4 a = a4[r >> 2], k = k4[r >> 2], q = q4[r >> 2];
                     s_reg[r] = fmaf(a.x, s_reg[r], k.x * v);          o = fmaf(s_reg[r], q.x, o);
                     s_reg[r + 1] = fmaf(a.y, s_reg[r + 1], k.y * v);  o = fmaf(s_reg[r + 1], q.y, o);
                     s_reg[r + 2] = fmaf(a.z, s_reg[r + 2], k.z * v);  o = fmaf(s_reg[r + 2], q.z, o);
@@ -232,13 +205,21 @@ gated_linear_carry_kernel(float* __restrict__ state, float* __restrict__ sums, c
     state[(size_t)slot * per + e] = cur;
 }
 
-// The launches of a scan over prepared decays (or, TIED, over the gate's pre-activations): one walk, or chunk sums, carry
-// and chunk outputs.
-template <bool TIED>
-static int gated_scan_launches(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off, const float* z, int ldz,
-                               float q_scale, float* state, const int* cu_new, const int* seq_slot, float* out, int ldo,
-                               int n_seqs, int n_heads, int dim, int vdim, int chunk, int max_chunks, float* sums,
-                               float* decays, const float* z_bias, const float* lower, int pdl, cudaStream_t stream) {
+// proj [T, ld] holds q, k (n_heads x dim each) and v (n_heads x vdim) from the given columns;
+// z [T, ldz] float32 is the decay's pre-activation without its bias z_bias [n_heads x dim], and is overwritten
+// with the decays;
+// state [slots, n_heads, dim, vdim] float32; out [T, ldo] float32 gets o (n_heads x vdim).
+// chunk > 0: sequences are run in chunks of that many tokens, in parallel, through ``sums``
+// (n_seqs x max_chunks x n_heads x dim x vdim floats) and ``decays`` (n_seqs x max_chunks x n_heads x dim);
+// max_chunks = ceil(longest run of new tokens / chunk).
+SSB_API int ssb_gated_linear_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off,
+                                  float* z, int ldz, const float* z_bias, float tau, float q_scale,
+                                  float* state, const int* cu_new, const int* seq_slot, float* out, int ldo,
+                                  int n_seqs, int n_tokens, int n_heads, int dim, int vdim, int chunk, int max_chunks,
+                                  float* sums, float* decays, int pdl, cudaStream_t stream) {
+    if (n_seqs <= 0 || n_tokens <= 0) return 0;
+    if (dim <= 0 || dim > SCAN_MAX_ROWS * SCAN_GROUPS || vdim <= 0 || !(tau > 0.f)) return SSB_ERR_BAD_SIZE;
+    if (chunk < 0 || (chunk > 0 && (max_chunks <= 0 || sums == nullptr || decays == nullptr))) return SSB_ERR_BAD_SIZE;
     const long long items = chunk > 0 ? (long long)n_seqs * max_chunks : n_seqs;
     if (items > 0x7fffffffll) return SSB_ERR_BAD_SIZE;
     const dim3 grid((unsigned)items, n_heads, (vdim + SCAN_COLS - 1) / SCAN_COLS);
@@ -246,10 +227,17 @@ static int gated_scan_launches(const void* proj, int ld, int dtype, int q_off, i
     const int rpt = ((dim + SCAN_GROUPS - 1) / SCAN_GROUPS + 3) & ~3;
     const size_t smem = (size_t)SCAN_TOKENS * (3 * rpt * SCAN_GROUPS + SCAN_COLS + SCAN_COLS * SCAN_GROUPS) * sizeof(float);
     int rc = 0;
+    {
+        const size_t total = (size_t)n_tokens * n_heads * dim;
+        rc = ssb_launch(decay_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, pdl != 0, z, ldz, z_bias,
+                        1.0f / tau, n_heads * dim, total);
+        if (!rc) rc = ssb_launch_status();
+        if (rc) return rc;
+    }
 #define SSB_SCAN(T, OUT) \
-    rc = ssb_launch(gated_linear_scan_kernel<T, TIED>, grid, dim3(SCAN_COLS * SCAN_GROUPS), smem, stream, pdl != 0, \
+    rc = ssb_launch(gated_linear_scan_kernel<T>, grid, dim3(SCAN_COLS * SCAN_GROUPS), smem, stream, pdl != 0, \
                     (const T*)proj, ld, q_off, k_off, v_off, (const float*)z, ldz, q_scale, state, cu_new, seq_slot, \
-                    OUT, ldo, n_heads, dim, vdim, chunk, max_chunks, sums, decays, z_bias, lower)
+                    OUT, ldo, n_heads, dim, vdim, chunk, max_chunks, sums, decays)
 #define SSB_SCAN_BOTH(OUT) do { \
         if (dtype == SSB_F32) SSB_SCAN(float, OUT); \
         else if (dtype == SSB_BF16) SSB_SCAN(bf16, OUT); \
@@ -273,47 +261,262 @@ static int gated_scan_launches(const void* proj, int ld, int dtype, int q_off, i
     return 0;
 }
 
-// proj [T, ld] holds q, k (n_heads x dim each) and v (n_heads x vdim) from the given columns;
-// z [T, ldz] float32 is the decay's pre-activation without its bias z_bias [n_heads x dim], and is overwritten
-// with the decays;
-// state [slots, n_heads, dim, vdim] float32; out [T, ldo] float32 gets o (n_heads x vdim).
-// chunk > 0: sequences are run in chunks of that many tokens, in parallel, through ``sums``
-// (n_seqs x max_chunks x n_heads x dim x vdim floats) and ``decays`` (n_seqs x max_chunks x n_heads x dim);
-// max_chunks = ceil(longest run of new tokens / chunk).
-SSB_API int ssb_gated_linear_scan(const void* proj, int ld, int dtype, int q_off, int k_off, int v_off,
-                                  float* z, int ldz, const float* z_bias, float tau, float q_scale,
-                                  float* state, const int* cu_new, const int* seq_slot, float* out, int ldo,
-                                  int n_seqs, int n_tokens, int n_heads, int dim, int vdim, int chunk, int max_chunks,
-                                  float* sums, float* decays, int pdl, cudaStream_t stream) {
-    if (n_seqs <= 0 || n_tokens <= 0) return 0;
-    if (dim <= 0 || dim > SCAN_MAX_ROWS * SCAN_GROUPS || vdim <= 0 || !(tau > 0.f)) return SSB_ERR_BAD_SIZE;
-    if (chunk < 0 || (chunk > 0 && (max_chunks <= 0 || sums == nullptr || decays == nullptr))) return SSB_ERR_BAD_SIZE;
-    const long long items = chunk > 0 ? (long long)n_seqs * max_chunks : n_seqs;
-    if (items > 0x7fffffffll || n_seqs > 65535 || n_heads > 65535) return SSB_ERR_BAD_SIZE;
-    int rc = 0;
-    {
-        const size_t total = (size_t)n_tokens * n_heads * dim;
-        rc = ssb_launch(decay_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, pdl != 0, z, ldz, z_bias,
-                        1.0f / tau, n_heads * dim, total);
+// =======================================================================================
+// The tied form (HGRN2): a forget gate f per key channel that also says what is written,
+//     f_t = l + (1 - l) sigmoid(z_t + b),    S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T,    o_t = S_t^T silu(q_t)
+// walked as S <- S + k (v - S) with k = 1 - f = (1 - l) sigmoid(-z - b): a gate close to one loses nothing to the
+// rounding of 1 - f.
+//
+// A block takes one head of one sequence (or chunk of it) and up to 8 value columns a warp.  A lane owns a tile of the
+// state in registers, 4 columns by 4 R4 rows: sixteen lanes share four columns, so a token's k and q are read from
+// shared memory once for four columns, and the sums over rows are five shuffles for all four (the first two halve
+// the columns a lane still carries).  Eight tokens are staged per barrier, in two buffers, while the next eight are on
+// their way from memory.
+//   OUT = false: chunk sums, from zero, with the product of the chunk's decays;
+//   OUT = true: outputs from the state at the start (the slot's, or what the carry kernel left for the chunk).
+// norm_w given (one block holds all of the head's columns): the head norm is taken where the outputs meet in shared
+// memory, y = o / rms(o) * norm_w, a warp a token; else o itself goes out in float32.
+// =======================================================================================
+constexpr int TW_TOKENS = 8;
+
+// The written share 1 - f, from the gate's pre-activation (bias included) and the lower bound.
+__device__ __forceinline__ float tied_share(float z, float lower) { return (1.0f - lower) / (1.0f + expf(z)); }
+
+struct TiedArgs {
+    const void* proj; int ld, q_off, f_off, v_off;
+    const float* z_bias; const float* lower;
+    float* state; const int* cu_new; const int* seq_slot;
+    float* out; int ldo;
+    const float* norm_w; float eps; void* y; int ldy;
+    int n_heads, dim, vdim, chunk, max_chunks;
+    float* sums; float* decays;
+};
+
+template <typename T, int R4, int NT, bool OUT>
+__global__ void __launch_bounds__(NT)
+tied_walk_kernel(const TiedArgs a) {
+    constexpr int DIMP = 64 * R4, COLS = NT / 4;          // padded rows; columns a block owns
+    constexpr int KI = TW_TOKENS * DIMP / NT, VI = TW_TOKENS * COLS / NT;
+    extern __shared__ __align__(16) float tw_sm[];
+    float* k_s = tw_sm;                                    // [2][TW_TOKENS][DIMP]
+    float* q_s = k_s + 2 * TW_TOKENS * DIMP;               // [2][TW_TOKENS][DIMP]
+    float* v_s = q_s + 2 * TW_TOKENS * DIMP;               // [2][TW_TOKENS][COLS]
+    float* o_s = v_s + 2 * TW_TOKENS * COLS;               // [2][TW_TOKENS][COLS]
+    const int dim = a.dim, vdim = a.vdim, h = blockIdx.y, j0 = blockIdx.z * COLS;
+    const int b = a.chunk > 0 ? blockIdx.x / a.max_chunks : blockIdx.x, ch = a.chunk > 0 ? blockIdx.x % a.max_chunks : 0;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rg = lane & 15, cg = lane >> 4;
+    ssb_pdl_launch_dependents();
+    ssb_pdl_wait();
+    const int slot = a.seq_slot[b];
+    if (slot < 0) return;                                  // padding row
+    int t0 = a.cu_new[b], t1 = a.cu_new[b + 1];
+    if (a.chunk > 0) {
+        t0 += ch * a.chunk;
+        t1 = min(t1, t0 + a.chunk);
+    }
+    if (t0 >= t1) return;
+    const T* proj = reinterpret_cast<const T*>(a.proj);
+    float* S = a.chunk > 0 ? a.sums + (((size_t)blockIdx.x * a.n_heads + h) * dim) * vdim
+                           : a.state + ((size_t)slot * a.n_heads + h) * dim * vdim;
+    const int col0 = warp * 8 + cg * 4;                    // this lane's four columns, within the block's
+    float s[R4][4][4];
+#pragma unroll
+    for (int g = 0; g < R4; ++g)
+#pragma unroll
+        for (int r = 0; r < 4; ++r)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const int i = (g * 16 + rg) * 4 + r, j = j0 + col0 + c;
+                s[g][r][c] = (OUT && i < dim && j < vdim) ? S[(size_t)i * vdim + j] : 0.f;
+            }
+    float prod[R4][4];
+#pragma unroll
+    for (int g = 0; g < R4; ++g)
+#pragma unroll
+        for (int r = 0; r < 4; ++r) prod[g][r] = 1.f;
+    // this thread's channels among the staged items are the same in every turn: DIMP divides NT or is divided by it
+    float bias[KI], low[KI];
+#pragma unroll
+    for (int n = 0; n < KI; ++n) {
+        const int i = (n * NT + tid) % DIMP;
+        bias[n] = i < dim ? a.z_bias[h * dim + i] : 0.f;
+        low[n] = i < dim ? a.lower[h * dim + i] : 0.f;
+    }
+    float zz[KI], qq[KI], vv[VI];
+    auto fetch = [&](int t) {
+#pragma unroll
+        for (int n = 0; n < KI; ++n) {
+            const int item = n * NT + tid, tt = item / DIMP, i = item % DIMP;
+            const bool ok = t + tt < t1 && i < dim;
+            const T* row = proj + (size_t)(t + tt) * a.ld + h * dim + i;
+            zz[n] = ok ? ssb_to_float(row[a.f_off]) : 0.f;
+            qq[n] = OUT && ok ? ssb_to_float(row[a.q_off]) : 0.f;
+        }
+#pragma unroll
+        for (int n = 0; n < VI; ++n) {
+            const int item = n * NT + tid, tt = item / COLS, j = j0 + item % COLS;
+            vv[n] = t + tt < t1 && j < vdim ? ssb_to_float(proj[(size_t)(t + tt) * a.ld + a.v_off + h * vdim + j]) : 0.f;
+        }
+    };
+    auto finish = [&](int t, int buf) {                    // the outputs of the tokens from t on, which wait in buffer buf
+        const float* o_b = o_s + buf * TW_TOKENS * COLS;
+        const int n_tok = min(TW_TOKENS, t1 - t);
+        if (a.norm_w == nullptr) {
+            for (int e = tid; e < n_tok * COLS; e += NT) {
+                const int tt = e / COLS, j = j0 + e % COLS;
+                if (j < vdim) a.out[(size_t)(t + tt) * a.ldo + (size_t)h * vdim + j] = o_b[e];
+            }
+            return;
+        }
+        for (int tt = warp; tt < n_tok; tt += NT / 32) {
+            float sq = 0.f;
+            for (int j = lane; j < vdim; j += 32) sq = fmaf(o_b[tt * COLS + j], o_b[tt * COLS + j], sq);
+#pragma unroll
+            for (int m = 16; m > 0; m >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, m);
+            const float inv = 1.0f / sqrtf(sq / (float)vdim + a.eps);
+            T* y = reinterpret_cast<T*>(a.y) + (size_t)(t + tt) * a.ldy + (size_t)h * vdim;
+            for (int j = lane; j < vdim; j += 32) y[j] = ssb_from_float<T>(o_b[tt * COLS + j] * inv * a.norm_w[j]);
+        }
+    };
+    fetch(t0);
+    int buf = 0;
+    for (int t = t0; t < t1; t += TW_TOKENS, buf ^= 1) {
+        float* kb = k_s + buf * TW_TOKENS * DIMP;
+        float* qb = q_s + buf * TW_TOKENS * DIMP;
+        float* vb = v_s + buf * TW_TOKENS * COLS;
+        float* ob = o_s + buf * TW_TOKENS * COLS;
+#pragma unroll
+        for (int n = 0; n < KI; ++n) {
+            const int item = n * NT + tid, tt = item / DIMP, i = item % DIMP;
+            const bool ok = t + tt < t1 && i < dim;        // padding rows and tokens leave the state as it is: k = 0
+            kb[item] = ok ? tied_share(zz[n] + bias[n], low[n]) : 0.f;
+            if (OUT) qb[item] = qq[n] / (1.0f + expf(-qq[n]));
+        }
+#pragma unroll
+        for (int n = 0; n < VI; ++n) vb[n * NT + tid] = vv[n];
+        __syncthreads();
+        if (t + TW_TOKENS < t1) fetch(t + TW_TOKENS);
+        if (OUT && t > t0) finish(t - TW_TOKENS, buf ^ 1);
+        if (j0 + warp * 8 < vdim) {
+#pragma unroll 2
+            for (int tt = 0; tt < TW_TOKENS; ++tt) {
+                const float4 v4 = *reinterpret_cast<const float4*>(vb + tt * COLS + col0);
+                const float v[4] = {v4.x, v4.y, v4.z, v4.w};
+                float o[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                for (int g = 0; g < R4; ++g) {
+                    const float4 k4 = *reinterpret_cast<const float4*>(kb + tt * DIMP + (g * 16 + rg) * 4);
+                    const float k[4] = {k4.x, k4.y, k4.z, k4.w};
+                    float q[4] = {0.f, 0.f, 0.f, 0.f};
+                    if (OUT) {
+                        const float4 q4 = *reinterpret_cast<const float4*>(qb + tt * DIMP + (g * 16 + rg) * 4);
+                        q[0] = q4.x; q[1] = q4.y; q[2] = q4.z; q[3] = q4.w;
+                    }
+#pragma unroll
+                    for (int r = 0; r < 4; ++r) {
+#pragma unroll
+                        for (int c = 0; c < 4; ++c) {
+                            s[g][r][c] = fmaf(k[r], v[c] - s[g][r][c], s[g][r][c]);
+                            if (OUT) o[c] = fmaf(s[g][r][c], q[r], o[c]);
+                        }
+                        if (!OUT && warp == 0) prod[g][r] *= 1.0f - k[r];
+                    }
+                }
+                if (OUT) {
+                    // sums over the sixteen lanes of a column group; a lane ends with one of the four columns
+                    const bool hi8 = (lane & 8) != 0, hi4 = (lane & 4) != 0;
+                    const float p0 = (hi8 ? o[2] : o[0]) + __shfl_xor_sync(0xffffffffu, hi8 ? o[0] : o[2], 8);
+                    const float p1 = (hi8 ? o[3] : o[1]) + __shfl_xor_sync(0xffffffffu, hi8 ? o[1] : o[3], 8);
+                    float p = (hi4 ? p1 : p0) + __shfl_xor_sync(0xffffffffu, hi4 ? p0 : p1, 4);
+                    p += __shfl_xor_sync(0xffffffffu, p, 2);
+                    p += __shfl_xor_sync(0xffffffffu, p, 1);
+                    if ((lane & 3) == 0) ob[tt * COLS + col0 + (hi8 ? 2 : 0) + (hi4 ? 1 : 0)] = p;
+                }
+            }
+        }
+    }
+    if (OUT) {
+        __syncthreads();
+        const int last = t0 + (t1 - t0 - 1) / TW_TOKENS * TW_TOKENS;
+        finish(last, buf ^ 1);
+        if (a.chunk > 0) return;                           // the state was carried by the carry kernel
+    }
+#pragma unroll
+    for (int g = 0; g < R4; ++g)
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+            const int i = (g * 16 + rg) * 4 + r;
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const int j = j0 + col0 + c;
+                if (i < dim && j < vdim) S[(size_t)i * vdim + j] = s[g][r][c];
+            }
+            if (!OUT && blockIdx.z == 0 && warp == 0 && cg == 0 && i < dim)
+                a.decays[((size_t)blockIdx.x * a.n_heads + h) * dim + i] = prod[g][r];
+        }
+}
+
+template <typename T, int R4, int NT>
+static int launch_tied_walk(const TiedArgs& a, int n_seqs, bool pdl, cudaStream_t stream) {
+    constexpr int DIMP = 64 * R4, COLS = NT / 4;
+    constexpr size_t smem = (size_t)TW_TOKENS * (4 * DIMP + 4 * COLS) * sizeof(float);
+    const long long items = a.chunk > 0 ? (long long)n_seqs * a.max_chunks : n_seqs;
+    const dim3 grid((unsigned)items, a.n_heads, (a.vdim + COLS - 1) / COLS);
+    if (items > 0x7fffffffll || grid.y > 65535 || grid.z > 65535 || n_seqs > 65535) return SSB_ERR_BAD_SIZE;
+    static_assert(smem <= 200 * 1024, "");
+    auto sums = tied_walk_kernel<T, R4, NT, false>;
+    auto outs = tied_walk_kernel<T, R4, NT, true>;
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(sums, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(outs, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
+    int rc;
+    if (a.chunk > 0) {
+        rc = ssb_launch(sums, grid, dim3(NT), smem, stream, pdl, a);
+        if (!rc) rc = ssb_launch_status();
+        if (rc) return rc;
+        const size_t per = (size_t)a.n_heads * a.dim * a.vdim;
+        rc = ssb_launch(gated_linear_carry_kernel, dim3((unsigned)((per + 255) / 256), n_seqs), dim3(256), 0, stream, pdl, a.state,
+                        a.sums, (const float*)a.decays, a.cu_new, a.seq_slot, a.n_heads, a.dim, a.vdim, a.chunk, a.max_chunks);
         if (!rc) rc = ssb_launch_status();
         if (rc) return rc;
     }
-    return gated_scan_launches<false>(proj, ld, dtype, q_off, k_off, v_off, z, ldz, q_scale, state, cu_new, seq_slot, out, ldo,
-                                      n_seqs, n_heads, dim, vdim, chunk, max_chunks, sums, decays, nullptr, nullptr, pdl, stream);
+    rc = ssb_launch(outs, grid, dim3(NT), smem, stream, pdl, a);
+    return rc ? rc : ssb_launch_status();
 }
 
-// The tied form: f_off names the gate's pre-activation among proj's columns (bias z_bias, lower bounds `lower`, both
-// [n_heads x dim]); otherwise as ssb_gated_linear_scan.
+// proj [T, ld] holds q and the gate's pre-activation (n_heads x dim each) and v (n_heads x vdim) from the given columns;
+// z_bias and lower [n_heads x dim]; state [slots, n_heads, dim, vdim] float32.  norm_w null: out [T, ldo] float32 gets o;
+// else (vdim up to 128, up to 64 where dim is above 128) y [T, ldy] of proj's type gets the normed heads.  chunk, max_chunks, sums and decays as ssb_gated_linear_scan's.
 SSB_API int ssb_tied_scan(const void* proj, int ld, int dtype, int q_off, int f_off, int v_off, const float* z_bias,
                           const float* lower, float* state, const int* cu_new, const int* seq_slot, float* out, int ldo,
-                          int n_seqs, int n_tokens, int n_heads, int dim, int vdim, int chunk, int max_chunks, float* sums,
-                          float* decays, int pdl, cudaStream_t stream) {
+                          const float* norm_w, float eps, void* y, int ldy, int n_seqs, int n_tokens, int n_heads, int dim,
+                          int vdim, int chunk, int max_chunks, float* sums, float* decays, int pdl, cudaStream_t stream) {
     if (n_seqs <= 0 || n_tokens <= 0) return 0;
-    if (dim <= 0 || dim > SCAN_MAX_ROWS * SCAN_GROUPS || vdim <= 0 || n_heads <= 0 || z_bias == nullptr || lower == nullptr)
-        return SSB_ERR_BAD_SIZE;
+    if (dim <= 0 || dim > 256 || vdim <= 0 || n_heads <= 0 || z_bias == nullptr || lower == nullptr) return SSB_ERR_BAD_SIZE;
     if (chunk < 0 || (chunk > 0 && (max_chunks <= 0 || sums == nullptr || decays == nullptr))) return SSB_ERR_BAD_SIZE;
-    return gated_scan_launches<true>(proj, ld, dtype, q_off, f_off, v_off, nullptr, 0, 1.0f, state, cu_new, seq_slot, out, ldo,
-                                     n_seqs, n_heads, dim, vdim, chunk, max_chunks, sums, decays, z_bias, lower, pdl, stream);
+    if (norm_w != nullptr ? (y == nullptr || vdim > (dim > 128 ? 64 : 128)) : out == nullptr) return SSB_ERR_BAD_SIZE;
+    TiedArgs a;
+    a.proj = proj; a.ld = ld; a.q_off = q_off; a.f_off = f_off; a.v_off = v_off; a.z_bias = z_bias; a.lower = lower;
+    a.state = state; a.cu_new = cu_new; a.seq_slot = seq_slot; a.out = out; a.ldo = ldo; a.norm_w = norm_w; a.eps = eps;
+    a.y = y; a.ldy = ldy; a.n_heads = n_heads; a.dim = dim; a.vdim = vdim; a.chunk = chunk; a.max_chunks = max_chunks;
+    a.sums = sums; a.decays = decays;
+    const bool chain = pdl != 0;
+#define SSB_TW(T)                                                                                          \
+    {                                                                                                      \
+        if (vdim <= 64)                                                                                    \
+            return dim <= 64 ? launch_tied_walk<T, 1, 256>(a, n_seqs, chain, stream)                       \
+                 : dim <= 128 ? launch_tied_walk<T, 2, 256>(a, n_seqs, chain, stream)                      \
+                              : launch_tied_walk<T, 4, 256>(a, n_seqs, chain, stream);                     \
+        return dim <= 64 ? launch_tied_walk<T, 1, 512>(a, n_seqs, chain, stream)                           \
+             : dim <= 128 ? launch_tied_walk<T, 2, 512>(a, n_seqs, chain, stream)                          \
+                          : launch_tied_walk<T, 4, 256>(a, n_seqs, chain, stream);                         \
+    }
+    if (dtype == SSB_F32) SSB_TW(float)
+    if (dtype == SSB_BF16) SSB_TW(bf16)
+#undef SSB_TW
+    return SSB_ERR_BAD_DTYPE;
 }
 
 // ---------------------------------------------------------------------------------------

@@ -297,11 +297,113 @@ causal_conv_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ x
     }
 }
 
+// The same for bfloat16 rows in whole 16-byte pieces and two to four taps: a thread owns eight neighbouring channels
+// of CV_TILE tokens, with all its rows requested before the first is used.
+constexpr int CV_TILE = 8;
+constexpr int CV_THREADS = 128;
+
+template <int TAPS>
+__global__ void __launch_bounds__(CV_THREADS)
+causal_conv_vec_kernel(const bf16* __restrict__ x, int ldx, const float* __restrict__ w, float* __restrict__ tail,
+                       const int* __restrict__ cu_new, const int* __restrict__ seq_slot, bf16* __restrict__ u, int ldu,
+                       int channels, int pass_cols) {
+    constexpr int BACK = TAPS - 1;
+    const int b = blockIdx.x;
+    ssb_pdl_launch_dependents();
+    ssb_pdl_wait();
+    const int slot = seq_slot[b];
+    if (slot < 0) return;
+    const int t0 = cu_new[b], t1 = cu_new[b + 1];
+    const int lo = t0 + blockIdx.y * CV_TILE;
+    if (lo >= t1) return;
+    const int c = (blockIdx.z * CV_THREADS + threadIdx.x) * 8;
+    if (c >= channels + pass_cols) return;
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    uint4 raw[CV_TILE + BACK];
+#pragma unroll
+    for (int i = 0; i < CV_TILE + BACK; ++i) {
+        const int t = lo - BACK + i;
+        raw[i] = t >= t0 && t < t1 ? *reinterpret_cast<const uint4*>(x + (size_t)t * ldx + c) : zero;
+    }
+    if (c >= channels) {                                   // columns behind the channels pass through unchanged
+#pragma unroll
+        for (int i = 0; i < CV_TILE; ++i)
+            if (lo + i < t1) *reinterpret_cast<uint4*>(u + (size_t)(lo + i) * ldu + c) = raw[BACK + i];
+        return;
+    }
+    float wj[8][TAPS];
+#pragma unroll
+    for (int k = 0; k < 8; ++k)
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) wj[k][j] = w[(size_t)(c + k) * TAPS + j];
+    float* keep = tail + (size_t)slot * BACK * channels + c;
+    auto value = [](const uint4& r, int k) {
+        const uint32_t q = k < 2 ? r.x : k < 4 ? r.y : k < 6 ? r.z : r.w;
+        return __uint_as_float((k & 1) ? (q & 0xffff0000u) : (q << 16));
+    };
+    // inputs before the tile: rows of this step, or, in the sequence's first tile, its kept rows
+    float win[BACK][8];
+#pragma unroll
+    for (int i = 0; i < BACK; ++i)
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+            win[i][k] = lo - BACK + i >= t0 ? value(raw[i], k) : keep[(size_t)(lo - t0 + i) * channels + k];
+    if (lo == t0) {
+        // what the next step will need: the last BACK inputs of (kept rows, new inputs); places are written in rising
+        // order from places above them
+        const int n_new = t1 - t0;
+#pragma unroll
+        for (int i = 0; i < BACK; ++i) {
+            const int rel = n_new - BACK + i;
+            if (rel >= 0) {
+                const uint4 r = *reinterpret_cast<const uint4*>(x + (size_t)(t0 + rel) * ldx + c);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) keep[(size_t)i * channels + k] = value(r, k);
+            } else {
+#pragma unroll
+                for (int k = 0; k < 8; ++k) keep[(size_t)i * channels + k] = keep[(size_t)(rel + BACK) * channels + k];
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < CV_TILE; ++i) {
+        float v[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+            float acc = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                const int r = i + j - BACK;                // row of the tile that tap j sees
+                acc = fmaf(wj[k][j], r < 0 ? win[i + j < BACK ? i + j : 0][k] : value(raw[BACK + (r < 0 ? 0 : r)], k), acc);
+            }
+            v[k] = acc;
+        }
+        if (lo + i < t1) {
+            uint4 o;
+            __nv_bfloat162 p0 = __floats2bfloat162_rn(v[0], v[1]), p1 = __floats2bfloat162_rn(v[2], v[3]);
+            __nv_bfloat162 p2 = __floats2bfloat162_rn(v[4], v[5]), p3 = __floats2bfloat162_rn(v[6], v[7]);
+            o.x = *reinterpret_cast<uint32_t*>(&p0); o.y = *reinterpret_cast<uint32_t*>(&p1);
+            o.z = *reinterpret_cast<uint32_t*>(&p2); o.w = *reinterpret_cast<uint32_t*>(&p3);
+            *reinterpret_cast<uint4*>(u + (size_t)(lo + i) * ldu + c) = o;
+        }
+    }
+}
+
 SSB_API int ssb_causal_conv(const void* x, int ldx, int dtype, const float* x_bias, const float* w, const float* bias,
                             float* tail, const int* cu_new, const int* seq_slot, void* u, int ldu, int n_seqs,
                             int max_new, int channels, int taps, int pass_cols, int pdl, cudaStream_t stream) {
     if (n_seqs <= 0 || max_new <= 0) return 0;
     if (channels <= 0 || taps < 1 || taps > CONV_MAX_TAPS || pass_cols < 0) return SSB_ERR_BAD_SIZE;
+    if (dtype == SSB_BF16 && x_bias == nullptr && bias == nullptr && taps >= 2 && taps <= 4 && channels % 8 == 0 &&
+        pass_cols % 8 == 0 && ldx % 8 == 0 && ldu % 8 == 0 && (((uintptr_t)x | (uintptr_t)u) & 15) == 0 && x != u) {
+        const dim3 vgrid(n_seqs, (max_new + CV_TILE - 1) / CV_TILE, ((channels + pass_cols) / 8 + CV_THREADS - 1) / CV_THREADS);
+        if (vgrid.y <= 65535 && vgrid.z <= 65535) {
+            auto kern = taps == 2 ? causal_conv_vec_kernel<2> : taps == 3 ? causal_conv_vec_kernel<3> : causal_conv_vec_kernel<4>;
+            const int rcv = ssb_launch(kern, vgrid, dim3(CV_THREADS), 0, stream, pdl != 0, (const bf16*)x, ldx, w, tail, cu_new,
+                                       seq_slot, (bf16*)u, ldu, channels, pass_cols);
+            return rcv ? rcv : ssb_launch_status();
+        }
+    }
     const int tile = 32;                                  // at least taps - 1
     const dim3 grid(n_seqs, (max_new + tile - 1) / tile, (channels + pass_cols + SEQ_THREADS - 1) / SEQ_THREADS);
     if (grid.y > 65535 || grid.z > 65535) return SSB_ERR_BAD_SIZE;

@@ -36,8 +36,134 @@ struct SxArgs {
     int taps, width, streams;
 };
 
-// One block per token; u's row waits in shared memory for its sum of squares, which is taken in a fixed order.
-// SM: an upper bound of the number of streams (the loops over them are unrolled).
+// The convolution behind the norm, for one column of a token that is alone in its sequence's step.
+__device__ __forceinline__ float sx_convolve(const SxArgs& a, int slot, int c, float n) {
+    const int back = a.taps - 1;
+    const float* w = a.conv_w + (size_t)c * a.taps;
+    float acc = 0.f;
+    if (slot >= 0 && back > 0) {                           // the kept rows move down by one place
+        float* keep = a.tail + (size_t)slot * back * a.width + c;
+        for (int j = 0; j < back; ++j) {
+            const float v = keep[(size_t)j * a.width];
+            acc = fmaf(w[j], v, acc);
+            if (j > 0) keep[(size_t)(j - 1) * a.width] = v;
+        }
+        keep[(size_t)(back - 1) * a.width] = n;
+    }
+    return fmaf(w[back], n, acc);
+}
+
+__device__ __forceinline__ float sx_block_sum(float v, float* red) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float total = 0.f;
+    for (int w = 0; w < (int)blockDim.x / 32; ++w) total += red[w];
+    return total;
+}
+
+__device__ __forceinline__ void sx_store4(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void sx_store4(bf16* p, const float* v) {
+    const __nv_bfloat162 x = __floats2bfloat162_rn(v[0], v[1]), y = __floats2bfloat162_rn(v[2], v[3]);
+    uint2 u;
+    u.x = *reinterpret_cast<const uint32_t*>(&x);
+    u.y = *reinterpret_cast<const uint32_t*>(&y);
+    *reinterpret_cast<uint2*>(p) = u;
+}
+
+// Rows of whole float4s that a block's registers hold: everything is loaded before anything is stored (a loop that
+// zeroes a piece of the branch between its loads takes ten times as long: 211 against 20 us for 2,048 rows of 2,048
+// and two streams).  S: the number of streams; N: float4s a thread owns of a row.
+template <typename T, int S, int N, int NT>
+__global__ void __launch_bounds__(NT)
+stream_cross_vec_kernel(const SxArgs a) {
+    __shared__ float red[32];
+    const int tid = threadIdx.x, W = a.width, n4 = W / 4;
+    const bool writes = a.branch != nullptr;
+    ssb_pdl_launch_dependents();
+    // coefficients and the norm's weights: no kernel of a step writes them
+    float mix[S * S], out_w[S], in_w[S];
+#pragma unroll
+    for (int i = 0; i < S * S; ++i) mix[i] = writes ? a.mix[i] : 0.f;
+#pragma unroll
+    for (int i = 0; i < S; ++i) {
+        out_w[i] = writes ? a.out_w[i] : 0.f;
+        in_w[i] = a.in_w != nullptr ? a.in_w[i] : 1.0f;
+    }
+    ssb_pdl_wait();
+    const size_t row = (size_t)blockIdx.x * W;
+    float x[S][N][4], y[N][4];
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+        const int c = tid + n * NT;
+        const size_t at = row + 4 * (size_t)c;
+#pragma unroll
+        for (int s = 0; s < S; ++s) {
+            if (s > 0 && a.n_src == 1) {
+#pragma unroll
+                for (int k = 0; k < 4; ++k) x[s][n][k] = x[0][n][k];
+                continue;
+            }
+            const float4 v = c < n4 ? *reinterpret_cast<const float4*>(a.src + s * a.plane + at) : make_float4(0.f, 0.f, 0.f, 0.f);
+            x[s][n][0] = v.x; x[s][n][1] = v.y; x[s][n][2] = v.z; x[s][n][3] = v.w;
+        }
+        const float4 v = writes && c < n4 ? *reinterpret_cast<const float4*>(a.branch + at) : make_float4(0.f, 0.f, 0.f, 0.f);
+        y[n][0] = v.x; y[n][1] = v.y; y[n][2] = v.z; y[n][3] = v.w;
+    }
+    float sq = 0.f;
+#pragma unroll
+    for (int n = 0; n < N; ++n)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            float u = 0.f;
+            if (writes) {
+                float v[S];
+#pragma unroll
+                for (int to = 0; to < S; ++to) {
+                    v[to] = out_w[to] * y[n][k];
+#pragma unroll
+                    for (int s = 0; s < S; ++s) v[to] = fmaf(mix[s * S + to], x[s][n][k], v[to]);
+                    u = fmaf(in_w[to], v[to], u);
+                }
+#pragma unroll
+                for (int to = 0; to < S; ++to) x[to][n][k] = v[to];
+            } else {
+#pragma unroll
+                for (int s = 0; s < S; ++s) u = fmaf(in_w[s], x[s][n][k], u);
+            }
+            y[n][k] = u;
+            sq = fmaf(u, u, sq);
+        }
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+        const int c = tid + n * NT;
+        const size_t at = row + 4 * (size_t)c;
+        if (c >= n4) continue;
+        if (a.dst != nullptr)
+#pragma unroll
+            for (int s = 0; s < S; ++s) sx_store4(a.dst + s * a.plane + at, x[s][n]);
+        if (writes && a.clear) *reinterpret_cast<float4*>(a.branch + at) = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (a.norm_w == nullptr) sx_store4(reinterpret_cast<float*>(a.out) + at, y[n]);
+    }
+    if (a.norm_w == nullptr) return;
+    const float inv = 1.0f / sqrtf(sx_block_sum(sq, red) / (float)W + a.eps);
+    const int slot = a.conv_w != nullptr ? a.slot[blockIdx.x] : -1;
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+        const int c = tid + n * NT;
+        if (c >= n4) continue;
+        const float4 w = *reinterpret_cast<const float4*>(a.norm_w + 4 * c);
+        float v[4] = {y[n][0] * inv * w.x, y[n][1] * inv * w.y, y[n][2] * inv * w.z, y[n][3] * inv * w.w};
+        if (a.conv_w != nullptr)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) v[k] = sx_convolve(a, slot, 4 * c + k, v[k]);
+        sx_store4(reinterpret_cast<T*>(a.out) + row + 4 * c, v);
+    }
+}
+
+// Any width and number of streams (SM: an upper bound of it, the loops over the streams are unrolled).  u's row waits in
+// shared memory for its sum of squares, which is taken in a fixed order.
 template <typename T, int SM>
 __global__ void stream_cross_kernel(const SxArgs a) {
     extern __shared__ float sx_row[];
@@ -46,7 +172,6 @@ __global__ void stream_cross_kernel(const SxArgs a) {
     const int tid = threadIdx.x, nt = blockDim.x, S = a.streams, W = a.width;
     const bool writes = a.branch != nullptr;
     ssb_pdl_launch_dependents();
-    // the coefficients are weights: no kernel of a step writes them
     if (writes) {
         for (int i = tid; i < S * S; i += nt) c_mix[(i / S) * SM + i % S] = a.mix[i];
         for (int i = tid; i < S; i += nt) c_out[i] = a.out_w[i];
@@ -65,7 +190,6 @@ __global__ void stream_cross_kernel(const SxArgs a) {
         float u = 0.f;
         if (writes) {
             const float y = br[c];
-            if (a.clear) br[c] = 0.f;
 #pragma unroll
             for (int to = 0; to < SM; ++to)
                 if (to < S) {
@@ -81,42 +205,32 @@ __global__ void stream_cross_kernel(const SxArgs a) {
             for (int s = 0; s < SM; ++s)
                 if (s < S) u = fmaf(c_in[s], x[s], u);
         }
-        if (a.norm_w == nullptr) {
-            reinterpret_cast<float*>(a.out)[t * W + c] = u;
-            continue;
-        }
-        sx_row[c] = u;
+        if (a.norm_w == nullptr) reinterpret_cast<float*>(a.out)[t * W + c] = u;
+        else sx_row[c] = u;
         sq = fmaf(u, u, sq);
     }
+    if (writes && a.clear)
+        for (int c = tid; c < W; c += nt) br[c] = 0.f;
     if (a.norm_w == nullptr) return;
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
-    if ((tid & 31) == 0) red[tid >> 5] = sq;
-    __syncthreads();
-    float total = 0.f;
-    for (int w = 0; w < nt / 32; ++w) total += red[w];
-    const float inv = 1.0f / sqrtf(total / (float)W + a.eps);
+    const float inv = 1.0f / sqrtf(sx_block_sum(sq, red) / (float)W + a.eps);
     T* out = reinterpret_cast<T*>(a.out) + t * W;
-    if (a.conv_w == nullptr) {
-        for (int c = tid; c < W; c += nt) out[c] = ssb_from_float<T>(sx_row[c] * inv * a.norm_w[c]);
-        return;
-    }
-    const int slot = a.slot[t], back = a.taps - 1;
+    const int slot = a.conv_w != nullptr ? a.slot[t] : -1;
     for (int c = tid; c < W; c += nt) {
         const float n = sx_row[c] * inv * a.norm_w[c];
-        const float* w = a.conv_w + (size_t)c * a.taps;
-        float acc = 0.f;
-        if (slot >= 0 && back > 0) {                       // the kept rows move down by one place
-            float* keep = a.tail + (size_t)slot * back * W + c;
-            for (int j = 0; j < back; ++j) {
-                const float v = keep[(size_t)j * W];
-                acc = fmaf(w[j], v, acc);
-                if (j > 0) keep[(size_t)(j - 1) * W] = v;
-            }
-            keep[(size_t)(back - 1) * W] = n;
-        }
-        out[c] = ssb_from_float<T>(fmaf(w[back], n, acc));
+        out[c] = ssb_from_float<T>(a.conv_w != nullptr ? sx_convolve(a, slot, c, n) : n);
     }
+}
+
+template <typename T, int S>
+static int launch_stream_vec(const SxArgs& a, int n_tokens, bool pdl, cudaStream_t stream) {
+    const int n4 = a.width / 4;
+#define SSB_SXV(N, NT) return ssb_launch(stream_cross_vec_kernel<T, S, N, NT>, dim3(n_tokens), dim3(NT), 0, stream, pdl, a)
+    if (n4 <= 128) SSB_SXV(1, 128);
+    if (n4 <= 256) SSB_SXV(1, 256);
+    if (n4 <= 512) SSB_SXV(1, 512);
+    if (n4 <= 1024) SSB_SXV(2, 512);
+    SSB_SXV(4, 512);
+#undef SSB_SXV
 }
 
 // See SxArgs.  branch null: no write (mix, out_w and dst are not read).  norm_w null: out is float32 and gets u.
@@ -136,9 +250,18 @@ SSB_API int ssb_stream_cross(const float* src, int n_src, long long plane, float
     a.dst = branch != nullptr ? dst : nullptr;
     a.in_w = in_w; a.norm_w = norm_w; a.eps = eps; a.out = out; a.conv_w = conv_w; a.tail = tail; a.slot = slot;
     a.taps = taps; a.width = width; a.streams = streams;
-    // few tokens: a block's latency is the step's, so more threads share a row
-    const int threads = n_tokens <= 148 && width >= 1024 ? 512 : 256;
     int rc;
+    const uintptr_t align = (uintptr_t)src | (uintptr_t)branch | (uintptr_t)a.dst | (uintptr_t)norm_w | (uintptr_t)out;
+    if (width % 4 == 0 && width <= 8192 && streams <= 4 && (align & 15) == 0 && plane % 4 == 0) {
+        const bool chain = pdl != 0;
+#define SSB_SXT(S) rc = out_dtype == SSB_F32 ? launch_stream_vec<float, S>(a, n_tokens, chain, stream) \
+                                             : launch_stream_vec<bf16, S>(a, n_tokens, chain, stream)
+        if (out_dtype != SSB_F32 && out_dtype != SSB_BF16) return SSB_ERR_BAD_DTYPE;
+        if (streams == 1) SSB_SXT(1); else if (streams == 2) SSB_SXT(2); else if (streams == 3) SSB_SXT(3); else SSB_SXT(4);
+#undef SSB_SXT
+        return rc ? rc : ssb_launch_status();
+    }
+    const int threads = 256;
 #define SSB_SX(TYPE, SM)                                                                                             \
     {                                                                                                                \
         auto kern = stream_cross_kernel<TYPE, SM>;                                                                   \

@@ -194,8 +194,13 @@ def test_tied_scan_forms_agree():
         assert float((out - runs[0][0]).abs().max()) < 1e-4 * float(runs[0][0].abs().max())
         assert float((state - runs[0][1]).abs().max()) < 1e-4 * float(runs[0][1].abs().max())
     assert torch.equal(runs[0][1][[1, 3, 5]], state0[[1, 3, 5]])             # nobody else's state is touched
-    # token by token, with a padding row
+    # the head norm taken along
     w = torch.rand(dv, device=DEV, generator=g) + 0.5
+    y = torch.zeros(T, H * dv, device=DEV)
+    ops.tied_scan(proj, 0, H * d, 2 * H * d, bias, lower, state0.clone(), cu, slots, y, H, d, dv, norm_w=w, eps=1e-5)
+    want = (pr.unit_rms(runs[0][0].cpu().double().reshape(T, H, dv), 1e-5) * w.cpu().double()).reshape(T, -1)
+    assert float((y.cpu().double() - want).abs().max()) < 2e-4
+    # token by token, with a padding row
     state = state0.clone()
     for i in range(lens[2]):
         row = torch.stack([proj[271 + i], proj[0]]).contiguous()
