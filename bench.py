@@ -518,7 +518,8 @@ def _operation_work(model, tokens):
             add("feed_forward.expert_gate_up", 2 * T * ff.top * ff.w_gate_up[0].numel())
             add("feed_forward.grouped_linear", 2 * T * ff.top * ff.w_down[0].numel())
             if getattr(getattr(ff.router, "weight", None), "dim", lambda: 0)() == 2:   # a router that reads the token: a product of its own
-                add("feed_forward.linear", 2 * T * ff.router.weight.numel())
+                inside = type(ff.router).__name__ == "SoftmaxRouter"                  # ... taken with the choice as one operation
+                add("feed_forward.route_softmax" if inside else "feed_forward.linear", 2 * T * ff.router.weight.numel())
             if ff.shared is not None:
                 add("feed_forward.gate_up_swiglu", 2 * T * ff.shared.w_gate_up.numel())
                 add("feed_forward.linear", 2 * T * ff.shared.w_down.numel())

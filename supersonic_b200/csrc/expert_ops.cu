@@ -147,8 +147,8 @@ SSB_API int ssb_route_sigmoid_groups(const float* z, int ld, const float* correc
 // chosen scores (+ 1e-20).  One warp per token, lanes over experts.
 // ---------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(RG_THREADS)
-route_softmax_kernel(const float* __restrict__ z, int ld, int n_tokens, int n_experts, int top, int renormalize, float scale,
-                     int* __restrict__ expert_of, float* __restrict__ pair_weight) {
+route_softmax_kernel(float* __restrict__ z, int ld, int n_tokens, int n_experts, int top, int renormalize, float scale,
+                     int clear, int* __restrict__ expert_of, float* __restrict__ pair_weight) {
     extern __shared__ float rs_smem[];                   // per warp: [n_experts] scores, [top] chosen scores
     ssb_pdl_launch_dependents();
     ssb_pdl_wait();
@@ -157,14 +157,19 @@ route_softmax_kernel(const float* __restrict__ z, int ld, int n_tokens, int n_ex
     if (t >= n_tokens) return;
     float* s_s = rs_smem + (size_t)warp * (n_experts + top);
     float* w_s = s_s + n_experts;
-    const float* zr = z + (size_t)t * ld;
+    float* zr = z + (size_t)t * ld;
     float m = -INFINITY;
-    for (int e = lane; e < n_experts; e += 32) m = fmaxf(m, zr[e]);
+    for (int e = lane; e < n_experts; e += 32) {
+        s_s[e] = zr[e];
+        m = fmaxf(m, s_s[e]);
+    }
+    if (clear)
+        for (int e = lane; e < ld; e += 32) zr[e] = 0.f;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
     float sum = 0.f;
     for (int e = lane; e < n_experts; e += 32) {
-        const float p = expf(zr[e] - m);
+        const float p = expf(s_s[e] - m);
         s_s[e] = p;
         sum += p;
     }
@@ -203,7 +208,8 @@ route_softmax_kernel(const float* __restrict__ z, int ld, int n_tokens, int n_ex
     for (int k = lane; k < top; k += 32) pair_weight[(size_t)t * top + k] = w_s[k] * f;
 }
 
-SSB_API int ssb_route_softmax(const float* z, int ld, int n_tokens, int n_experts, int top, int renormalize, float scale,
+// clear: the whole row of z (ld columns) is zeroed behind the read.
+SSB_API int ssb_route_softmax(float* z, int ld, int n_tokens, int n_experts, int top, int renormalize, float scale, int clear,
                               int* expert_of, float* pair_weight, int pdl, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (n_experts <= 0 || top < 1 || top > n_experts || n_experts > 2048 || ld < n_experts) return SSB_ERR_BAD_SIZE;
@@ -214,7 +220,7 @@ SSB_API int ssb_route_softmax(const float* z, int ld, int n_tokens, int n_expert
     }
     const int rc = ssb_launch(route_softmax_kernel, dim3((n_tokens + RG_THREADS / 32 - 1) / (RG_THREADS / 32)),
                               dim3(RG_THREADS), smem, stream, pdl != 0, z, ld, n_tokens, n_experts, top, renormalize, scale,
-                              expert_of, pair_weight);
+                              clear, expert_of, pair_weight);
     return rc ? rc : ssb_launch_status();
 }
 

@@ -455,6 +455,19 @@ class FastKernels(PlainKernels):
     def route_table(self, token_ids, table, n_experts, expert_of, pair_weight):
         ops.route_table(token_ids, table, n_experts, expert_of, pair_weight, pdl=self.pdl)
 
+    def route_softmax(self, x, weight, n_experts, renormalize, scale, expert_of, pair_weight):
+        rows, n = x.shape[0], weight.shape[0]
+        if rows > STREAM_ROWS or self.deterministic:
+            super().route_softmax(x, weight, n_experts, renormalize, scale, expert_of, pair_weight)
+            return
+        # a few rows: K is split over blocks that add into sums which are zero between uses (the choice clears its rows)
+        logits = self._buffer("router_sums", rows * n, torch.float32, x.device, zero=True)[: rows * n].view(rows, n)
+        if not ops.gemm_tc_ok(x, weight, logits):
+            super().route_softmax(x, weight, n_experts, renormalize, scale, expert_of, pair_weight)
+            return
+        ops.gemv_tc(x, weight, logits, ops.TC_ACCUMULATE, splits=ops.gemv_tc_splits(n, weight.shape[1]), pdl=self.pdl)
+        ops.route_softmax(logits, n_experts, renormalize, scale, expert_of, pair_weight, clear=True, pdl=self._chain(rows))
+
     def group_by_expert(self, expert_of, n_experts, groups):
         ops.group_by_expert(expert_of, n_experts, groups["tile_rows"], groups["offsets"], groups["order"],
                             groups["tile_expert"], groups["tile_row0"], groups["meta"], pdl=self.pdl)

@@ -98,18 +98,19 @@ class PlainKernels:
     def stream_enter(self, src, streams, in_weights, branch, write, dst, norm, conv, tail, batch, out):
         """A sublayer's entry over several residual streams: the write of the sublayer before (``write`` = (mix,
         out_weights) with its ``branch``, or None), the next read, its RMS norm and the short convolution behind it
-        (``conv`` [width, taps] float32, ``tail`` its per-slot rows), into ``out``."""
+        (``conv`` float32 in two layouts, ([width, taps], [taps, width]); ``tail`` its per-slot rows), into ``out``."""
         mix, out_w = write if write is not None else (None, None)
         if write is None:
             branch = dst = None
         pdl = self._chain(batch.n_tokens)
         if batch.is_decode:                    # one token a sequence: the convolution reads its kept rows alone
-            ops.stream_cross(src, streams, in_weights, out, branch, mix, out_w, dst, True, norm.weight_f32, norm.eps, conv,
+            ops.stream_cross(src, streams, in_weights, out, branch, mix, out_w, dst, True, norm.weight_f32, norm.eps, conv[1],
                              tail, batch.slot_of_token, pdl=pdl)
             return
         normed = torch.empty_like(out)
         ops.stream_cross(src, streams, in_weights, normed, branch, mix, out_w, dst, True, norm.weight_f32, norm.eps, pdl=pdl)
-        ops.causal_conv(normed, None, conv, None, tail if conv.shape[1] > 1 else conv[:1, :0], batch.cu_new, batch.seq_slot,
+        w = conv[0]
+        ops.causal_conv(normed, None, w, None, tail if w.shape[1] > 1 else w[:1, :0], batch.cu_new, batch.seq_slot,
                         out, batch.max_new, pdl=pdl)
 
     def stream_sum(self, src, streams, branch, write, out, clear=True):
@@ -360,7 +361,10 @@ class PlainKernels:
         ops.route_sigmoid_groups(logits, n_experts, correction, n_groups, keep, scale, expert_of, pair_weight, extra_col,
                                  extra_out, pdl=self._chain(logits.shape[0]))
 
-    def route_softmax(self, logits, n_experts, renormalize, scale, expert_of, pair_weight):
+    def route_softmax(self, x, weight, n_experts, renormalize, scale, expert_of, pair_weight):
+        """The router's product (logits x @ weight^T in float32) and the choice."""
+        logits = torch.empty((x.shape[0], weight.shape[0]), dtype=torch.float32, device=x.device)
+        self.linear(x, weight, logits)
         ops.route_softmax(logits, n_experts, renormalize, scale, expert_of, pair_weight, pdl=self._chain(logits.shape[0]))
 
     def group_by_expert(self, expert_of, n_experts, groups):

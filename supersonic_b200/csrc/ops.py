@@ -588,8 +588,8 @@ def stream_cross(src: torch.Tensor, streams: int, in_weights: Optional[torch.Ten
     With a ``branch`` y [tokens, width] the streams become x_t = sum_s mix[s, t] x_s + out_weights[t] y, all at once from
     the old ones, stored into ``dst`` (``src`` itself, another tensor, or None: not stored), and ``clear`` zeroes the
     branch behind the read.  Then u = sum_t in_weights[t] x_t (None: their sum); ``out`` gets u (float32) or, with
-    ``norm_weight``, u / sqrt(mean(u^2) + eps) * norm_weight.  With ``conv`` [width, taps] (one token a sequence only) the
-    normed row n passes a causal convolution, out = sum_j conv[:, j] n_(t - taps + 1 + j), whose earlier rows are
+    ``norm_weight``, u / sqrt(mean(u^2) + eps) * norm_weight.  With ``conv`` [taps, width] (one token a sequence only) the
+    normed row n passes a causal convolution, out = sum_j conv[j] n_(t - taps + 1 + j), whose earlier rows are
     ``tail[slot]`` ([taps - 1, width], oldest first), brought up to date."""
     _need(src, "src", torch.float32, 3); _need(out, "out", None, 2)
     n_src, T, W = src.shape
@@ -621,9 +621,9 @@ def stream_cross(src: torch.Tensor, streams: int, in_weights: Optional[torch.Ten
     taps = 0
     if conv is not None:
         _need(conv, "conv", torch.float32, 2); _need(slot, "slot", torch.int32, 1)
-        taps = conv.shape[1]
-        if conv.shape[0] != W or not conv.is_contiguous() or not 1 <= taps <= CONV_MAX_TAPS or slot.shape[0] != T:
-            raise KernelError(f"stream_cross: conv [width, taps] of up to {CONV_MAX_TAPS} taps, one slot per token")
+        taps = conv.shape[0]
+        if conv.shape[1] != W or not conv.is_contiguous() or not 1 <= taps <= CONV_MAX_TAPS or slot.shape[0] != T:
+            raise KernelError(f"stream_cross: conv [taps, width] of up to {CONV_MAX_TAPS} taps, one slot per token")
         if taps > 1:
             _need(tail, "tail", torch.float32, 2)
             if tail.shape[1] != (taps - 1) * W or not tail.is_contiguous():
@@ -1426,9 +1426,10 @@ def route_sigmoid_groups(logits: torch.Tensor, n_experts: int, correction: Optio
 
 
 def route_softmax(logits: torch.Tensor, n_experts: int, renormalize: bool, scale: float, expert_of: torch.Tensor,
-                  pair_weight: torch.Tensor, pdl: bool = False) -> None:
+                  pair_weight: torch.Tensor, clear: bool = False, pdl: bool = False) -> None:
     """Per token, from float32 router logits [tokens, >= n_experts]: s = softmax(z) over all experts; the ``top`` experts
-    with the largest s; pair_weight = s * scale, with ``renormalize`` divided by the chosen scores' sum (+ 1e-20)."""
+    with the largest s; pair_weight = s * scale, with ``renormalize`` divided by the chosen scores' sum (+ 1e-20).
+    ``clear``: the logits' rows are zeroed behind the read."""
     _need(logits, "logits", torch.float32, 2)
     _need(expert_of, "expert_of", torch.int32, 2); _need(pair_weight, "pair_weight", torch.float32, 2)
     T, top = logits.shape[0], expert_of.shape[1]
@@ -1437,7 +1438,8 @@ def route_softmax(logits: torch.Tensor, n_experts: int, renormalize: bool, scale
         raise KernelError("route_softmax: logits [tokens, >= experts]; expert_of and pair_weight [tokens, top], contiguous")
     _check(_fn("expert_ops", "ssb_route_softmax")(
         _ptr(logits), c_int(logits.stride(0)), c_int(T), c_int(n_experts), c_int(top), c_int(1 if renormalize else 0),
-        c_float(scale), _ptr(expert_of), _ptr(pair_weight), c_int(1 if pdl else 0), _stream()), "route_softmax")
+        c_float(scale), c_int(1 if clear else 0), _ptr(expert_of), _ptr(pair_weight), c_int(1 if pdl else 0), _stream()),
+        "route_softmax")
 
 
 def expert_tiles_bound(n_pairs: int, n_experts: int, tile_rows: int) -> int:

@@ -333,9 +333,13 @@ causal_conv_vec_kernel(const bf16* __restrict__ x, int ldx, const float* __restr
     }
     float wj[8][TAPS];
 #pragma unroll
-    for (int k = 0; k < 8; ++k)
-#pragma unroll
-        for (int j = 0; j < TAPS; ++j) wj[k][j] = w[(size_t)(c + k) * TAPS + j];
+    for (int e = 0; e < 8 * TAPS; e += 4) {
+        const float4 v = *reinterpret_cast<const float4*>(w + (size_t)c * TAPS + e);
+        wj[e / TAPS][e % TAPS] = v.x;
+        wj[(e + 1) / TAPS][(e + 1) % TAPS] = v.y;
+        wj[(e + 2) / TAPS][(e + 2) % TAPS] = v.z;
+        wj[(e + 3) / TAPS][(e + 3) % TAPS] = v.w;
+    }
     float* keep = tail + (size_t)slot * BACK * channels + c;
     auto value = [](const uint4& r, int k) {
         const uint32_t q = k < 2 ? r.x : k < 4 ? r.y : k < 6 ? r.z : r.w;
@@ -344,25 +348,38 @@ causal_conv_vec_kernel(const bf16* __restrict__ x, int ldx, const float* __restr
     // inputs before the tile: rows of this step, or, in the sequence's first tile, its kept rows
     float win[BACK][8];
 #pragma unroll
-    for (int i = 0; i < BACK; ++i)
+    for (int i = 0; i < BACK; ++i) {
+        if (lo > t0) {                                     // CV_TILE >= BACK: the tile before this one holds them all
 #pragma unroll
-        for (int k = 0; k < 8; ++k)
-            win[i][k] = lo - BACK + i >= t0 ? value(raw[i], k) : keep[(size_t)(lo - t0 + i) * channels + k];
+            for (int k = 0; k < 8; ++k) win[i][k] = value(raw[i], k);
+        } else {
+            const float4 a = *reinterpret_cast<const float4*>(keep + (size_t)i * channels);
+            const float4 d = *reinterpret_cast<const float4*>(keep + (size_t)i * channels + 4);
+            win[i][0] = a.x; win[i][1] = a.y; win[i][2] = a.z; win[i][3] = a.w;
+            win[i][4] = d.x; win[i][5] = d.y; win[i][6] = d.z; win[i][7] = d.w;
+        }
+    }
     if (lo == t0) {
-        // what the next step will need: the last BACK inputs of (kept rows, new inputs); places are written in rising
-        // order from places above them
+        // what the next step will need: the last BACK inputs of (kept rows, new inputs)
         const int n_new = t1 - t0;
 #pragma unroll
         for (int i = 0; i < BACK; ++i) {
             const int rel = n_new - BACK + i;
+            float v[8];
             if (rel >= 0) {
                 const uint4 r = *reinterpret_cast<const uint4*>(x + (size_t)(t0 + rel) * ldx + c);
 #pragma unroll
-                for (int k = 0; k < 8; ++k) keep[(size_t)i * channels + k] = value(r, k);
+                for (int k = 0; k < 8; ++k) v[k] = value(r, k);
             } else {
 #pragma unroll
-                for (int k = 0; k < 8; ++k) keep[(size_t)i * channels + k] = keep[(size_t)(rel + BACK) * channels + k];
+                for (int k = 0; k < 8; ++k) {
+                    v[k] = 0.f;
+#pragma unroll
+                    for (int o = 0; o < BACK; ++o) v[k] = rel + BACK == o ? win[o][k] : v[k];
+                }
             }
+            *reinterpret_cast<float4*>(keep + (size_t)i * channels) = make_float4(v[0], v[1], v[2], v[3]);
+            *reinterpret_cast<float4*>(keep + (size_t)i * channels + 4) = make_float4(v[4], v[5], v[6], v[7]);
         }
     }
 #pragma unroll
@@ -395,7 +412,7 @@ SSB_API int ssb_causal_conv(const void* x, int ldx, int dtype, const float* x_bi
     if (n_seqs <= 0 || max_new <= 0) return 0;
     if (channels <= 0 || taps < 1 || taps > CONV_MAX_TAPS || pass_cols < 0) return SSB_ERR_BAD_SIZE;
     if (dtype == SSB_BF16 && x_bias == nullptr && bias == nullptr && taps >= 2 && taps <= 4 && channels % 8 == 0 &&
-        pass_cols % 8 == 0 && ldx % 8 == 0 && ldu % 8 == 0 && (((uintptr_t)x | (uintptr_t)u) & 15) == 0 && x != u) {
+        pass_cols % 8 == 0 && ldx % 8 == 0 && ldu % 8 == 0 && (((uintptr_t)x | (uintptr_t)u | (uintptr_t)w | (uintptr_t)tail) & 15) == 0 && x != u) {
         const dim3 vgrid(n_seqs, (max_new + CV_TILE - 1) / CV_TILE, ((channels + pass_cols) / 8 + CV_THREADS - 1) / CV_THREADS);
         if (vgrid.y <= 65535 && vgrid.z <= 65535) {
             auto kern = taps == 2 ? causal_conv_vec_kernel<2> : taps == 3 ? causal_conv_vec_kernel<3> : causal_conv_vec_kernel<4>;

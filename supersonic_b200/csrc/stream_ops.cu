@@ -30,7 +30,7 @@ struct SxArgs {
     const float* norm_w;         // [width], or null: u itself goes out (float32)
     float eps;
     void* out;                   // [tokens][width]
-    const float* conv_w;         // [width][taps], or null: no convolution behind the norm
+    const float* conv_w;         // [taps][width], or null: no convolution behind the norm
     float* tail;                 // [slots][taps - 1][width] the last taps - 1 normed rows, oldest first
     const int* slot;             // [tokens]
     int taps, width, streams;
@@ -39,18 +39,18 @@ struct SxArgs {
 // The convolution behind the norm, for one column of a token that is alone in its sequence's step.
 __device__ __forceinline__ float sx_convolve(const SxArgs& a, int slot, int c, float n) {
     const int back = a.taps - 1;
-    const float* w = a.conv_w + (size_t)c * a.taps;
+    const float* w = a.conv_w + c;
     float acc = 0.f;
     if (slot >= 0 && back > 0) {                           // the kept rows move down by one place
         float* keep = a.tail + (size_t)slot * back * a.width + c;
         for (int j = 0; j < back; ++j) {
             const float v = keep[(size_t)j * a.width];
-            acc = fmaf(w[j], v, acc);
+            acc = fmaf(w[(size_t)j * a.width], v, acc);
             if (j > 0) keep[(size_t)(j - 1) * a.width] = v;
         }
         keep[(size_t)(back - 1) * a.width] = n;
     }
-    return fmaf(w[back], n, acc);
+    return fmaf(w[(size_t)back * a.width], n, acc);
 }
 
 __device__ __forceinline__ float sx_block_sum(float v, float* red) {
@@ -75,9 +75,11 @@ __device__ __forceinline__ void sx_store4(bf16* p, const float* v) {
 // Rows of whole float4s that a block's registers hold: everything is loaded before anything is stored (a loop that
 // zeroes a piece of the branch between its loads takes ten times as long: 211 against 20 us for 2,048 rows of 2,048
 // and two streams).  S: the number of streams; N: float4s a thread owns of a row.
-template <typename T, int S, int N, int NT>
+// TAPS > 0: with a convolution of that many taps behind the norm, whose weights and kept rows are requested with the rest.
+template <typename T, int S, int N, int NT, int TAPS>
 __global__ void __launch_bounds__(NT)
 stream_cross_vec_kernel(const SxArgs a) {
+    constexpr int BACK = TAPS > 0 ? TAPS - 1 : 0;
     __shared__ float red[32];
     const int tid = threadIdx.x, W = a.width, n4 = W / 4;
     const bool writes = a.branch != nullptr;
@@ -91,8 +93,26 @@ stream_cross_vec_kernel(const SxArgs a) {
         out_w[i] = writes ? a.out_w[i] : 0.f;
         in_w[i] = a.in_w != nullptr ? a.in_w[i] : 1.0f;
     }
+    float4 cw[TAPS > 0 ? TAPS : 1][N], kept[BACK > 0 ? BACK : 1][N];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+            const int c = tid + n * NT;
+            if (c < n4) cw[j][n] = *reinterpret_cast<const float4*>(a.conv_w + (size_t)j * W + 4 * c);
+        }
     ssb_pdl_wait();
     const size_t row = (size_t)blockIdx.x * W;
+    const int slot = TAPS > 0 ? a.slot[blockIdx.x] : -1;
+    float* keep = BACK > 0 && slot >= 0 ? a.tail + (size_t)slot * BACK * W : nullptr;
+#pragma unroll
+    for (int j = 0; j < BACK; ++j)
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+            const int c = tid + n * NT;
+            kept[j][n] = keep != nullptr && c < n4 ? *reinterpret_cast<const float4*>(keep + (size_t)j * W + 4 * c)
+                                                   : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
     float x[S][N][4], y[N][4];
 #pragma unroll
     for (int n = 0; n < N; ++n) {
@@ -148,16 +168,28 @@ stream_cross_vec_kernel(const SxArgs a) {
     }
     if (a.norm_w == nullptr) return;
     const float inv = 1.0f / sqrtf(sx_block_sum(sq, red) / (float)W + a.eps);
-    const int slot = a.conv_w != nullptr ? a.slot[blockIdx.x] : -1;
 #pragma unroll
     for (int n = 0; n < N; ++n) {
         const int c = tid + n * NT;
         if (c >= n4) continue;
         const float4 w = *reinterpret_cast<const float4*>(a.norm_w + 4 * c);
         float v[4] = {y[n][0] * inv * w.x, y[n][1] * inv * w.y, y[n][2] * inv * w.z, y[n][3] * inv * w.w};
-        if (a.conv_w != nullptr)
+        if (TAPS > 0) {
+            const float4 now = make_float4(v[0], v[1], v[2], v[3]);
+            float acc[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-            for (int k = 0; k < 4; ++k) v[k] = sx_convolve(a, slot, 4 * c + k, v[k]);
+            for (int j = 0; j < TAPS; ++j) {
+                const float4 r = j < BACK ? kept[j < BACK ? j : 0][n] : now;
+                acc[0] = fmaf(cw[j][n].x, r.x, acc[0]); acc[1] = fmaf(cw[j][n].y, r.y, acc[1]);
+                acc[2] = fmaf(cw[j][n].z, r.z, acc[2]); acc[3] = fmaf(cw[j][n].w, r.w, acc[3]);
+            }
+            if (keep != nullptr)
+#pragma unroll
+                for (int j = 0; j < BACK; ++j)             // the kept rows move down by one place
+                    *reinterpret_cast<float4*>(keep + (size_t)j * W + 4 * c) = j + 1 < BACK ? kept[j + 1 < BACK ? j + 1 : 0][n] : now;
+#pragma unroll
+            for (int k = 0; k < 4; ++k) v[k] = acc[k];
+        }
         sx_store4(reinterpret_cast<T*>(a.out) + row + 4 * c, v);
     }
 }
@@ -221,16 +253,28 @@ __global__ void stream_cross_kernel(const SxArgs a) {
     }
 }
 
-template <typename T, int S>
+constexpr int SX_VEC_TAPS = 4;                             // taps the kernel above holds in registers
+
+template <typename T, int S, int TAPS>
 static int launch_stream_vec(const SxArgs& a, int n_tokens, bool pdl, cudaStream_t stream) {
     const int n4 = a.width / 4;
-#define SSB_SXV(N, NT) return ssb_launch(stream_cross_vec_kernel<T, S, N, NT>, dim3(n_tokens), dim3(NT), 0, stream, pdl, a)
+#define SSB_SXV(N, NT) return ssb_launch(stream_cross_vec_kernel<T, S, N, NT, TAPS>, dim3(n_tokens), dim3(NT), 0, stream, pdl, a)
     if (n4 <= 128) SSB_SXV(1, 128);
     if (n4 <= 256) SSB_SXV(1, 256);
     if (n4 <= 512) SSB_SXV(1, 512);
     if (n4 <= 1024) SSB_SXV(2, 512);
-    SSB_SXV(4, 512);
+    if constexpr (TAPS == 0) { SSB_SXV(4, 512); }
+    return SSB_ERR_UNSUPPORTED;
 #undef SSB_SXV
+}
+
+template <typename T, int S>
+static int launch_stream_taps(const SxArgs& a, int n_tokens, bool pdl, cudaStream_t stream) {
+    if (a.conv_w == nullptr) return launch_stream_vec<T, S, 0>(a, n_tokens, pdl, stream);
+    if (a.taps == 1) return launch_stream_vec<T, S, 1>(a, n_tokens, pdl, stream);
+    if (a.taps == 2) return launch_stream_vec<T, S, 2>(a, n_tokens, pdl, stream);
+    if (a.taps == 3) return launch_stream_vec<T, S, 3>(a, n_tokens, pdl, stream);
+    return launch_stream_vec<T, S, 4>(a, n_tokens, pdl, stream);
 }
 
 // See SxArgs.  branch null: no write (mix, out_w and dst are not read).  norm_w null: out is float32 and gets u.
@@ -252,10 +296,12 @@ SSB_API int ssb_stream_cross(const float* src, int n_src, long long plane, float
     a.taps = taps; a.width = width; a.streams = streams;
     int rc;
     const uintptr_t align = (uintptr_t)src | (uintptr_t)branch | (uintptr_t)a.dst | (uintptr_t)norm_w | (uintptr_t)out;
-    if (width % 4 == 0 && width <= 8192 && streams <= 4 && (align & 15) == 0 && plane % 4 == 0) {
+    const uintptr_t conv_align = conv_w == nullptr ? 0 : (uintptr_t)conv_w | (taps > 1 ? (uintptr_t)tail : 0);
+    if (width % 4 == 0 && width <= (conv_w != nullptr ? 4096 : 8192) && streams <= 4 && ((align | conv_align) & 15) == 0 &&
+        plane % 4 == 0 && (conv_w == nullptr || taps <= SX_VEC_TAPS)) {
         const bool chain = pdl != 0;
-#define SSB_SXT(S) rc = out_dtype == SSB_F32 ? launch_stream_vec<float, S>(a, n_tokens, chain, stream) \
-                                             : launch_stream_vec<bf16, S>(a, n_tokens, chain, stream)
+#define SSB_SXT(S) rc = out_dtype == SSB_F32 ? launch_stream_taps<float, S>(a, n_tokens, chain, stream) \
+                                             : launch_stream_taps<bf16, S>(a, n_tokens, chain, stream)
         if (out_dtype != SSB_F32 && out_dtype != SSB_BF16) return SSB_ERR_BAD_DTYPE;
         if (streams == 1) SSB_SXT(1); else if (streams == 2) SSB_SXT(2); else if (streams == 3) SSB_SXT(3); else SSB_SXT(4);
 #undef SSB_SXT

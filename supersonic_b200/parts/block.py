@@ -253,9 +253,9 @@ class HyperConnectionBlock:
             if self.taps:
                 w = stored(f"{sub}_conv", (self.size, self.taps)).clone()
                 w[:, -1] += 1.0
-                self.convs.append(w)
             else:
-                self.convs.append(torch.ones((self.size, 1), dtype=torch.float32, device=build.device))
+                w = torch.ones((self.size, 1), dtype=torch.float32, device=build.device)
+            self.convs.append((w, w.T.contiguous()))        # by channel, for prompts; by tap, for single tokens
         self.dtype = build.dtype
 
     @staticmethod

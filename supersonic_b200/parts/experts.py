@@ -113,7 +113,8 @@ class SigmoidGroupRouter:
 @register_router("softmax")
 class SoftmaxRouter:
     """params: ``renormalize`` (True), ``scale`` (1.0); weights: ``weight`` [experts, hidden].  The logits are a product of
-    their own with a float32 result, as ``sigmoid_groups``'."""
+    their own with a float32 result (in the bfloat16 path: bfloat16 operands, whose products are exact in float32,
+    summed in float32)."""
 
     def __init__(self, params, weights, build: BuildContext, n_experts: int, top: int):
         self.n_experts, self.top = n_experts, top
@@ -129,9 +130,7 @@ class SoftmaxRouter:
         self.weight = w.contiguous()
 
     def route(self, ctx, x, expert_of, pair_weight):
-        logits = torch.empty((x.shape[0], self.weight.shape[0]), dtype=torch.float32, device=x.device)
-        ctx.kernels.linear(x, self.weight, logits)
-        ctx.kernels.route_softmax(logits, self.n_experts, self.renormalize, self.scale, expert_of, pair_weight)
+        ctx.kernels.route_softmax(x, self.weight, self.n_experts, self.renormalize, self.scale, expert_of, pair_weight)
 
 
 @register_feed_forward("experts")

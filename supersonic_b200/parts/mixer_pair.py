@@ -4,7 +4,8 @@
 
 with the root mean square taken over the model width (eps inside the root) and a weight vector each, or, with
 ``join`` = ``"add"``, added as they are, result = left + right, each half with the constant factor its own parameters
-give it (``out_scale``): both then add straight into the stream.
+give it (``out_scale``): both then add straight into the stream.  Halves that keep their products apart from what lies
+between (``splits_products``) share them: one product over the input rows of both, one over the concatenated heads.
 Either half is any registered mixer; each keeps what it needs in the cache under the pair's id
 (``(cache_id, "left")`` and ``(cache_id, "right")``), and each gets the position encoding only if it asks for it.
 """
@@ -30,6 +31,16 @@ class MixerPair:
             sub = params[side]
             self.halves.append((side, lookup(MIXERS, sub["kind"], "mixer")(sub["params"], sub["weights"], build),
                                 bool(sub.get("position", False))))
+        self.shared = self.join == "add" and all(getattr(m, "splits_products", False) for _, m, _ in self.halves)
+        if self.shared:
+            (_, left, _), (_, right, _) = self.halves
+            self.in_cols, self.out_cols = left.in_weight.shape[0], left.out_weight.shape[1]
+            self.w_in = torch.cat([left.in_weight, right.in_weight], dim=0).contiguous()
+            self.w_o = torch.cat([left.out_weight, right.out_weight], dim=1).contiguous()
+            self.dtype = build.dtype
+            # the halves keep views: nothing is held twice
+            left.share_products(self.w_in[: self.in_cols], self.w_o[:, : self.out_cols])
+            right.share_products(self.w_in[self.in_cols:], self.w_o[:, self.out_cols:])
         if self.join == "add":
             return
         self.eps, self.scale = float(params["norm_eps"]), float(params.get("scale", 0.5))
@@ -59,6 +70,16 @@ class MixerPair:
 
     def forward(self, ctx, x, residual, cache_id, writes_cache, position):
         x = x.tensor() if hasattr(x, "tensor") else x
+        if self.shared:
+            T, dev, k = ctx.batch.n_tokens, residual.device, ctx.kernels
+            proj = torch.empty((T, self.w_in.shape[0]), dtype=self.dtype, device=dev)
+            k.linear(x, self.w_in, proj)
+            heads = torch.empty((T, self.w_o.shape[1]), dtype=self.dtype, device=dev)
+            for (side, mixer, wants_position), p, h in zip(self.halves, (proj[:, : self.in_cols], proj[:, self.in_cols:]),
+                                                           (heads[:, : self.out_cols], heads[:, self.out_cols:])):
+                mixer.inner(ctx, p, h, (cache_id, side), writes_cache, position if wants_position else None)
+            k.linear(heads, self.w_o, residual, accumulate=True)
+            return
         if self.join == "add":
             for side, mixer, wants_position in self.halves:
                 mixer.forward(ctx, x, residual, (cache_id, side), writes_cache, position if wants_position else None)

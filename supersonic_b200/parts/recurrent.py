@@ -317,6 +317,20 @@ class Hgrn2:
         self.q_off, self.f_off, self.v_off = 0, HD, 2 * HD
         self.dtype = dt
 
+    # what a pair of mixers that share their products asks for
+    splits_products = True
+
+    @property
+    def in_weight(self):
+        return self.w_in
+
+    @property
+    def out_weight(self):
+        return self.w_o
+
+    def share_products(self, w_in, w_o):
+        self.w_in, self.w_o = w_in, w_o
+
     def cache_need(self):
         return StateNeed(self.H * self.dim * self.vdim)
 
@@ -337,6 +351,12 @@ class Hgrn2:
         proj = torch.empty((T, self.w_in.shape[0]), dtype=self.dtype, device=dev)
         k.linear(x, self.w_in, proj)
         y = torch.empty((T, self.H * self.vdim), dtype=self.dtype, device=dev)
-        k.tied_scan(proj, self.q_off, self.f_off, self.v_off, self.f_bias, self.lower, ctx.cache.state(cache_id), ctx.batch,
-                    self.norm_w, self.eps, y, self.H, self.dim, self.vdim)
+        self.inner(ctx, proj, y, cache_id, writes_cache, position)
         k.linear(y, self.w_o, residual, accumulate=True)
+
+    def inner(self, ctx, proj, heads, cache_id, writes_cache, position):
+        """From the projected rows [q | f | v] to the normed heads that the output product reads."""
+        if not writes_cache:
+            raise ValueError("a recurrent mixer cannot read another layer's state without advancing it")
+        ctx.kernels.tied_scan(proj, self.q_off, self.f_off, self.v_off, self.f_bias, self.lower, ctx.cache.state(cache_id),
+                              ctx.batch, self.norm_w, self.eps, heads, self.H, self.dim, self.vdim)

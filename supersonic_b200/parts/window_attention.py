@@ -275,8 +275,37 @@ class WindowAttention:
             self.w_q = torch.cat([self._q_rows] + self._gate_rows, dim=0).contiguous()
         return self.w_q
 
+    # what a pair of mixers that share their products asks for; two maps are merged behind the heads
+    @property
+    def splits_products(self):
+        return self.own_kv and self.maps == 1
+
+    @property
+    def in_weight(self):
+        return self.w_qkv
+
+    @property
+    def out_weight(self):
+        return self.w_o
+
+    def share_products(self, w_in, w_o):
+        self.w_qkv, self.w_o = w_in, w_o
+        self.w_q = None if self.kv_cols and self.gate_cols else w_in[: self.n_q * self.dim]
+        self._q_rows = w_in[: self.n_q * self.dim]
+        self._gate_rows = [w_in[self.n_q * self.dim + self.kv_cols:]] if self.gate_cols else []
+
     def forward(self, ctx, x, residual, cache_id, writes_cache, position):
         T, dev, k = ctx.batch.n_tokens, residual.device, ctx.kernels
+        weight = self.w_qkv if writes_cache else self._read_weight()
+        qkv = torch.empty((T, weight.shape[0]), dtype=self.dtype, device=dev)
+        k.linear(x, weight, qkv)
+        heads = torch.empty((T, self.n_q * self.vdim), dtype=self.dtype, device=dev)
+        self.inner(ctx, qkv, heads, cache_id, writes_cache, position)
+        k.linear(heads, self.w_o, residual, accumulate=True)
+
+    def inner(self, ctx, qkv, heads, cache_id, writes_cache, position):
+        """From the projected rows [q | k | v | gate] to the heads that the output product reads."""
+        T, dev, k = ctx.batch.n_tokens, qkv.device, ctx.kernels
         if writes_cache and not self.own_kv:
             raise ValueError("window_attention: a mixer without keys of its own cannot write a cache entry")
         named = bool(self.pool or self.taps > 1)
@@ -288,14 +317,11 @@ class WindowAttention:
             kc = kv[0]
             kv = (kc.view(kc.shape[0], G * M, kc.shape[2], D),) + tuple(kv[1:])
         q_cols = H * M * D
-        weight = self.w_qkv if writes_cache else self._read_weight()
         kv_cols = self.kv_cols if writes_cache else 0
-        qkv = torch.empty((T, weight.shape[0]), dtype=self.dtype, device=dev)
-        k.linear(x, weight, qkv)
         if self.taps:
             if not writes_cache:
                 raise ValueError("window_attention: a convolution keeps state: its stop must write its cache entry")
-            conv = torch.empty_like(qkv)
+            conv = torch.empty(qkv.shape, dtype=qkv.dtype, device=dev)
             # a single tap keeps nothing from earlier tokens: it scales every channel
             tail = ctx.cache.state((cache_id, "conv")) if self.taps > 1 else self.conv_w[:1, :0]
             k.causal_conv(qkv, None, self.conv_w, None, tail, ctx.batch, conv,
@@ -320,13 +346,10 @@ class WindowAttention:
             k.pool_rows(kv, pooled, ctx.batch, G, D, V, PAGE_SHIFT, self.pool)
         n_gates = H * V if self.element_gate else H if self.head_gate else 0
         gate = qkv[:, q_cols + kv_cols: q_cols + kv_cols + n_gates] if n_gates else None
-        heads = torch.empty((T, H * M * V), dtype=self.dtype, device=dev)
-        k.window_attention(qkv, kv, pooled, ctx.batch, heads, H * M, G * M, D, V, PAGE_SHIFT,
+        maps = heads if M == 1 else torch.empty((T, H * M * V), dtype=self.dtype, device=dev)
+        k.window_attention(qkv, kv, pooled, ctx.batch, maps, H * M, G * M, D, V, PAGE_SHIFT,
                            self.window, self.keep_first, self.pool, self.scale, self.softcap,
                            self.sinks, self.value_position, self.out_scale if M == 1 else 1.0, v_share=M, gate=gate,
                            gate_elems=self.element_gate, slopes=self.slopes, head_mul=self.head_mul)
         if M > 1:
-            merged = torch.empty((T, H * V), dtype=self.dtype, device=dev)
-            k.map_difference(heads, merged, H, G, V, self.lam, self.eps, (1.0 - self.map_offset) * self.out_scale)
-            heads = merged
-        k.linear(heads, self.w_o, residual, accumulate=True)
+            k.map_difference(maps, heads, H, G, V, self.lam, self.eps, (1.0 - self.map_offset) * self.out_scale)

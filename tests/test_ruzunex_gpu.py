@@ -250,15 +250,40 @@ def test_window_attention_kernels_agree_with_biases_sinks_and_gates(heads, kv_he
         assert float((a.float() - b.float()).abs().max()) < 0.02 * max(1.0, float(a.float().abs().max())), decode
 
 
+@pytest.mark.parametrize("channels,taps,behind", [(64, 2, 0), (1536, 3, 64), (2048, 4, 8), (200, 4, 24), (60, 3, 0), (64, 6, 8)])
+def test_convolution_in_pieces_and_by_element(channels, taps, behind):
+    """The convolution over sequences of 1 to 70 tokens with kept rows from before, in bfloat16 (16-byte pieces where the
+    sizes allow it) against float64, and the rows kept for the next step; columns behind the channels pass through."""
+    from supersonic_b200.csrc import ops
+    g = torch.Generator().manual_seed(channels)
+    lens = [1, 70, 2, 8, 33, 3]
+    T, slots = sum(lens), [4, 0, 5, 2, 6, 1]
+    x = torch.randn(T, channels + behind, generator=g).bfloat16()
+    w, tail0 = torch.randn(channels, taps, generator=g), torch.randn(8, (taps - 1) * channels, generator=g)
+    tail, out = tail0.to(DEV), torch.zeros(T, channels + behind, dtype=torch.bfloat16, device=DEV)
+    cu = torch.tensor([0] + list(np.cumsum(lens)), dtype=torch.int32, device=DEV)
+    ops.causal_conv(x.to(DEV), None, w.to(DEV), None, tail, cu, torch.tensor(slots, dtype=torch.int32, device=DEV), out, max(lens),
+                    pass_cols=behind)
+    at = 0
+    for n, s in zip(lens, slots):
+        rows = torch.cat([tail0[s].double().view(taps - 1, channels), x[at:at + n, :channels].double()])
+        ref = pr.short_conv(rows, w.double())[taps - 1:]
+        assert float((out[at:at + n, :channels].cpu().double() - ref).abs().max()) < 0.01 * float(ref.abs().max()) + 1e-3
+        assert float((tail[s].cpu().double().view(taps - 1, channels) - rows[-(taps - 1):]).abs().max()) < 1e-6
+        at += n
+    assert torch.equal(out[:, channels:].cpu(), x[:, channels:]) and torch.equal(tail[[3, 7]].cpu(), tail0[[3, 7]])
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("streams", [1, 2, 3, 4, 6, 11, 16])
-def test_streams_alone(dtype, streams):
+@pytest.mark.parametrize("width,streams,taps", [(50, 1, 4), (48, 1, 4), (64, 2, 1), (516, 2, 3), (2048, 2, 4), (4096, 2, 4), (50, 3, 2),
+                                                (1032, 3, 2), (640, 4, 4), (64, 4, 5), (72, 6, 3), (40, 11, 2), (30, 16, 4)])
+def test_streams_alone(dtype, width, streams, taps):
     """The pass between two sublayers: first read of equal streams, first write from them, write over the streams in
     place, the sum at the end; the branch is zero behind every read; the convolution behind the norm with its kept rows
     over single tokens, a padding row among them."""
     from supersonic_b200.csrc import ops
     g = torch.Generator().manual_seed(streams)
-    T, W, S, taps = 9, 50, streams, 4
+    T, W, S = 9, width, streams
     e, y1, y2 = (torch.randn(T, W, generator=g) for _ in range(3))
     w = {f"{p}.{r}": t for p in ("a", "b") for r, t in (("in", torch.randn(S, generator=g)), ("out", torch.randn(S, generator=g)),
                                                          ("mix", torch.randn(S, S, generator=g)))}
@@ -286,7 +311,8 @@ def test_streams_alone(dtype, streams):
     slot = torch.tensor([3, 0, 9, -1, 5, 1, 2, 7, 8], dtype=torch.int32)
     tail0 = torch.randn(10, (taps - 1) * W, generator=g)
     tail = tail0.to(DEV)
-    ops.stream_cross(x, S, d["a.in"], out, br, d["b.mix"], d["b.out"], x, True, nw.to(DEV), 1e-4, conv.to(DEV), tail, slot.to(DEV))
+    ops.stream_cross(x, S, d["a.in"], out, br, d["b.mix"], d["b.out"], x, True, nw.to(DEV), 1e-4, conv.T.contiguous().to(DEV), tail,
+                     slot.to(DEV))
     xs = pr.write_streams(xs, y2.double(), w, "b")
     n = norm(pr.read_streams(xs, w, "a"))
     for t in range(T):
@@ -295,7 +321,7 @@ def test_streams_alone(dtype, streams):
         rows = torch.cat([tail0[slot[t]].double().view(taps - 1, W), n[t:t + 1]])
         ref = pr.short_conv(rows, conv.double())[-1]
         assert float((out[t].cpu().double() - ref).abs().max()) < tolerance(dtype, ref, 0.01)
-        assert float((tail[slot[t]].cpu().double().view(taps - 1, W) - rows[1:]).abs().max()) < 1e-4 * float(rows.abs().max())
+        assert torch.allclose(tail[slot[t]].cpu().double().view(taps - 1, W), rows[1:], rtol=0, atol=1e-4 * float(rows.abs().max()))
     assert torch.equal(tail[[4, 6]].cpu(), tail0[[4, 6]])
     total = torch.empty(T, W, device=DEV)
     br.copy_(y1)
@@ -370,7 +396,8 @@ def test_router_alone(experts, top):
     for renorm in (True, False):
         eo = torch.empty(T, top, dtype=torch.int32, device=DEV)
         pw = torch.empty(T, top, device=DEV)
-        ops.route_softmax(logits, experts, renorm, 1.0 if renorm else 2.5, eo, pw)
+        ops.route_softmax(logits, experts, renorm, 1.0 if renorm else 2.5, eo, pw, clear=not renorm)
+        assert bool((logits == 0).all()) == (not renorm)         # cleared behind the read, if asked
         for t in range(T):
             idx = sorted(range(experts), key=lambda e: (-float(z[t, e]), e))[:top]
             assert eo[t].tolist() == idx
