@@ -514,8 +514,8 @@ def _operation_work(model, tokens):
             if ff is not None:
                 add("feed_forward.stream_enter", 0, T * W * (4 * (2 * S + 2) + 2))
         if fk == "Experts":
-            per = ff.w_gate_up[0].numel() + ff.w_down[0].numel()
-            add("feed_forward.expert_gate_up", 2 * T * ff.top * ff.w_gate_up[0].numel())
+            per = ff.w_first[0].numel() + ff.w_down[0].numel()
+            add("feed_forward.expert_gate_up", 2 * T * ff.top * ff.w_first[0].numel())
             add("feed_forward.grouped_linear", 2 * T * ff.top * ff.w_down[0].numel())
             if getattr(getattr(ff.router, "weight", None), "dim", lambda: 0)() == 2:   # a router that reads the token: a product of its own
                 inside = type(ff.router).__name__ == "SoftmaxRouter"                  # ... taken with the choice as one operation
@@ -568,7 +568,7 @@ def design_comparison(args):
                 ff = b.feed_forward
                 if type(ff).__name__ == "Experts":
                     unused = (1.0 - ff.top / ff.E) ** batch
-                    nbytes -= int(unused * (ff.w_gate_up.numel() + ff.w_down.numel()) * ff.w_down.element_size())
+                    nbytes -= int(unused * (ff.w_first.numel() + ff.w_down.numel()) * ff.w_down.element_size())
             rec[f"decode_{batch}x{args.prompt_len}"] = {
                 "ms": round(ms, 4), "tokens_per_s": round(batch * 1000.0 / ms), "kernels": kernels,
                 "gbs": round(nbytes / ms / 1e6, 1), "of_measured_hbm": round(nbytes / ms / 1e6 / pk["hbm_gbs"], 3)}

@@ -20,6 +20,7 @@ from .ronelorn import ARCHITECTURE as _RONELORN, RonelornConfig
 from .vufadra import ARCHITECTURE as _VUFADRA, VufadraConfig
 from .kilisun import ARCHITECTURE as _KILISUN, KilisunConfig
 from .ruzunex import ARCHITECTURE as _RUZUNEX, RuzunexConfig
+from .ropulix import ARCHITECTURE as _ROPULIX, RopulixConfig
 
 _ARCHITECTURES: Dict[str, Type] = {}
 
@@ -74,6 +75,7 @@ register_architecture(_VUFADRA, VufadraConfig)
 register_architecture(_RONELORN, RonelornConfig)
 register_architecture(_KILISUN, KilisunConfig)
 register_architecture(_RUZUNEX, RuzunexConfig)
+register_architecture(_ROPULIX, RopulixConfig)
 
 
 _PRESET_DIR = os.path.join(os.path.dirname(os.path.abspath(__file__)), "presets")

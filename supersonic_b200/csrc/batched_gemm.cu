@@ -13,8 +13,9 @@
 // four stages of 32).  Two stages of 32 columns when the tiles are full: then what counts is how
 // many blocks an SM holds (seven of 30 KB against three of 61 KB: 2,048 tokens' gate/up of 64
 // experts 2.6 ms against 3.1 ms).
-// Epilogues: store (bfloat16 or float32), or SwiGLU: the matrix is [gate rows; up rows] and the
-// tile computes both halves for its columns and stores silu(gate) * up.
+// Epilogues: store (bfloat16 or float32), optionally through an activation or times the sigmoid of a gate row's
+// element, or SwiGLU: the matrix is [gate rows; up rows] and the tile computes both halves for its columns and
+// stores silu(gate) * up.
 #include "mma_helpers.cuh"
 #include <math.h>
 
@@ -30,8 +31,13 @@ struct BgArgs {
     const int* offsets; const int* tile_expert; const int* tile_row0; const int* meta;   // grouped form, else null
     int M, N, K;                                  // M: rows (per-head form); N: output columns; K
     int up_row0;                                  // SwiGLU: first row of the up half in a matrix
+    int act_kind;                                 // store: the activation on the sums (ssb_activate), or -1
+    const bf16* gate; int ldg;                    // store, per-head form: C[t, e, n] *= sigmoid(gate[t * ldg + e * N + n]), or null
     int gate_kind; float gate_limit;              // SwiGLU: the gated unit's inner step (ssb_gate_fast) and its clamp
 };
+
+__device__ __forceinline__ void bg_store2(float* d, float a, float b) { *reinterpret_cast<float2*>(d) = make_float2(a, b); }
+__device__ __forceinline__ void bg_store2(bf16* d, float a, float b) { *reinterpret_cast<uint32_t*>(d) = pack2(a, b); }
 
 template <bool SWIGLU, typename TC, int BG_STAGES, int BG_BK>
 __global__ void __launch_bounds__(BG_THREADS)
@@ -142,18 +148,31 @@ batched_gemm_kernel(const BgArgs g) {
             if (r >= r_end) continue;
             const size_t crow = g.c_index ? (size_t)g.c_index[r] : (size_t)r;
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
+            for (int j = 0; j < 4; ++j) {
+                const int n = n0 + wn + j * 8 + 2 * (lane & 3);
+                if (n >= N) continue;
+                float v[2];
 #pragma unroll
                 for (int x = 0; x < 2; ++x) {
-                    const int n = n0 + wn + j * 8 + 2 * (lane & 3) + x;
-                    if (n >= N) continue;
-                    float v = acc[0][i][j][hrow * 2 + x];
+                    v[x] = acc[0][i][j][hrow * 2 + x];
                     if (SWIGLU) {
                         const float u = acc[SWIGLU ? 1 : 0][i][j][hrow * 2 + x];
-                        v = ssb_gate_fast(v, u, g.gate_kind, g.gate_limit);
+                        v[x] = ssb_gate_fast(v[x], u, g.gate_kind, g.gate_limit);
+                    } else if (g.act_kind >= 0) {
+                        v[x] = ssb_activate(v[x], g.act_kind);
+                    } else if (g.gate != nullptr && n + x < N) {
+                        const float z = __bfloat162float(g.gate[(size_t)r * g.ldg + (size_t)e * N + n + x]);
+                        v[x] = __fdividef(v[x], 1.0f + __expf(-z));
                     }
-                    C[crow * g.ldc + n] = ssb_from_float<TC>(v);
                 }
+                TC* dst = C + crow * g.ldc + n;
+                if (n + 1 < N && (reinterpret_cast<uintptr_t>(dst) & (2 * sizeof(TC) - 1)) == 0) {
+                    bg_store2(dst, v[0], v[1]);
+                } else {
+                    dst[0] = ssb_from_float<TC>(v[0]);
+                    if (n + 1 < N) dst[1] = ssb_from_float<TC>(v[1]);
+                }
+            }
         }
 }
 
@@ -174,30 +193,32 @@ static int bg_launch(const BgArgs& a, int mode, int out_dtype, dim3 grid, int de
     } while (0)
 #define SSB_BG(SW, TC) do { if (deep) SSB_BG_ST(SW, TC, 3, 64); else SSB_BG_ST(SW, TC, 2, 32); } while (0)
     if (mode == 1 && out_dtype == SSB_BF16) SSB_BG(true, bf16);
-    else if (mode == 0 && out_dtype == SSB_BF16) SSB_BG(false, bf16);
-    else if (mode == 0 && out_dtype == SSB_F32) SSB_BG(false, float);
+    else if (mode != 1 && out_dtype == SSB_BF16) SSB_BG(false, bf16);
+    else if (mode != 1 && out_dtype == SSB_F32) SSB_BG(false, float);
     else return SSB_ERR_BAD_DTYPE;
 #undef SSB_BG
 #undef SSB_BG_ST
     return rc ? rc : ssb_launch_status();
 }
 
-// one matrix per head: C[t, h, :N] = W[h] (N x K) A[t, h, :K]; *_batch: elements between heads
+// one matrix per head: C[t, h, :N] = W[h] (N x K) A[t, h, :K]; *_batch: elements between heads; with a gate row per
+// token (columns of all heads side by side): times sigmoid(gate[t, h * N + n])
 SSB_API int ssb_head_gemm_mma(const void* A, int lda, long long a_batch, const void* W, int ldw, long long w_batch,
                               void* C, int ldc, long long c_batch, int out_dtype, int n_heads, int M, int N, int K,
-                              int pdl, cudaStream_t stream) {
+                              const void* gate, int ldg, int pdl, cudaStream_t stream) {
     // M rows of every head: a deep ring when the rows are few
     if (M <= 0 || N <= 0 || n_heads <= 0) return 0;
     BgArgs a = {};
     a.A = (const bf16*)A; a.lda = lda; a.a_batch = a_batch; a.a_index = nullptr; a.a_div = 1;
     a.W = (const bf16*)W; a.ldw = ldw; a.w_batch = w_batch;
     a.C = C; a.ldc = ldc; a.c_batch = c_batch; a.c_index = nullptr;
-    a.M = M; a.N = N; a.K = K;
+    a.M = M; a.N = N; a.K = K; a.act_kind = -1; a.gate = (const bf16*)gate; a.ldg = ldg;
     return bg_launch(a, 0, out_dtype, dim3((N + BG_BN - 1) / BG_BN, (M + BG_BM - 1) / BG_BM, n_heads), M <= 256, pdl, stream);
 }
 
 // one matrix per expert over the rows grouped for it (tiles of 64 rows).  mode 0: C = A W_e^T with N
-// columns; mode 1: W_e = [gate (N rows); up (N rows)], C = silu(A gate^T) * (A up^T)
+// columns; mode 1: W_e = [gate (N rows); up (N rows)], C = silu(A gate^T) * (A up^T); mode 2: C = act(A W_e^T), act the
+// activation `gate_kind`
 SSB_API int ssb_grouped_gemm_mma(const void* A, int lda, const int* a_index, int a_div, const void* W, int ldw,
                                  long long w_expert, void* C, int ldc, const int* c_index, int out_dtype,
                                  const int* offsets, const int* tile_expert, const int* tile_row0, const int* meta,
@@ -206,13 +227,14 @@ SSB_API int ssb_grouped_gemm_mma(const void* A, int lda, const int* a_index, int
     // n_rows: the rows of all groups together (what the host knows of their sizes); gate_kind, gate_limit: the
     // gated unit's inner step in mode 1 (0: silu(g) u)
     if (max_tiles <= 0 || N <= 0) return 0;
-    if (a_div <= 0 || gate_kind < 0 || gate_kind > SSB_GATE_LAST) return SSB_ERR_BAD_SIZE;
+    if (a_div <= 0 || mode < 0 || mode > 2 || gate_kind < 0 || gate_kind > (mode == 2 ? (int)SSB_ACT_SILU : (int)SSB_GATE_LAST)) return SSB_ERR_BAD_SIZE;
     BgArgs a = {};
     a.A = (const bf16*)A; a.lda = lda; a.a_batch = 0; a.a_index = a_index; a.a_div = a_div;
     a.W = (const bf16*)W; a.ldw = ldw; a.w_batch = w_expert;
     a.C = C; a.ldc = ldc; a.c_batch = 0; a.c_index = c_index;
     a.offsets = offsets; a.tile_expert = tile_expert; a.tile_row0 = tile_row0; a.meta = meta;
     a.M = 0; a.N = N; a.K = K; a.up_row0 = N;
+    a.act_kind = mode == 2 ? gate_kind : -1;
     a.gate_kind = gate_kind; a.gate_limit = gate_limit;
     return bg_launch(a, mode, out_dtype, dim3((N + BG_BN - 1) / BG_BN, max_tiles, 1), n_rows <= 1024, pdl, stream);
 }

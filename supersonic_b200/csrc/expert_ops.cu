@@ -142,12 +142,12 @@ SSB_API int ssb_route_sigmoid_groups(const float* z, int ld, const float* correc
 }
 
 // ---------------------------------------------------------------------------------------
-// softmax router.  s = softmax(z) over all experts (float32); the `top` experts with the largest scores win, the lower
+// softmax router.  s = softmax(z + bias) over all experts (float32; the bias is optional); the `top` experts with the largest scores win, the lower
 // index at equal scores; an expert's weight is its s times `scale`, with `renormalize` divided by the sum of the
 // chosen scores (+ 1e-20).  One warp per token, lanes over experts.
 // ---------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(RG_THREADS)
-route_softmax_kernel(float* __restrict__ z, int ld, int n_tokens, int n_experts, int top, int renormalize, float scale,
+route_softmax_kernel(float* __restrict__ z, int ld, const float* __restrict__ bias, int n_tokens, int n_experts, int top, int renormalize, float scale,
                      int clear, int* __restrict__ expert_of, float* __restrict__ pair_weight) {
     extern __shared__ float rs_smem[];                   // per warp: [n_experts] scores, [top] chosen scores
     ssb_pdl_launch_dependents();
@@ -160,7 +160,7 @@ route_softmax_kernel(float* __restrict__ z, int ld, int n_tokens, int n_experts,
     float* zr = z + (size_t)t * ld;
     float m = -INFINITY;
     for (int e = lane; e < n_experts; e += 32) {
-        s_s[e] = zr[e];
+        s_s[e] = zr[e] + (bias ? bias[e] : 0.f);
         m = fmaxf(m, s_s[e]);
     }
     if (clear)
@@ -209,7 +209,7 @@ route_softmax_kernel(float* __restrict__ z, int ld, int n_tokens, int n_experts,
 }
 
 // clear: the whole row of z (ld columns) is zeroed behind the read.
-SSB_API int ssb_route_softmax(float* z, int ld, int n_tokens, int n_experts, int top, int renormalize, float scale, int clear,
+SSB_API int ssb_route_softmax(float* z, int ld, const float* bias, int n_tokens, int n_experts, int top, int renormalize, float scale, int clear,
                               int* expert_of, float* pair_weight, int pdl, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (n_experts <= 0 || top < 1 || top > n_experts || n_experts > 2048 || ld < n_experts) return SSB_ERR_BAD_SIZE;
@@ -219,7 +219,7 @@ SSB_API int ssb_route_softmax(float* z, int ld, int n_tokens, int n_experts, int
         if (e != cudaSuccess) return (int)e;
     }
     const int rc = ssb_launch(route_softmax_kernel, dim3((n_tokens + RG_THREADS / 32 - 1) / (RG_THREADS / 32)),
-                              dim3(RG_THREADS), smem, stream, pdl != 0, z, ld, n_tokens, n_experts, top, renormalize, scale,
+                              dim3(RG_THREADS), smem, stream, pdl != 0, z, ld, bias, n_tokens, n_experts, top, renormalize, scale,
                               clear, expert_of, pair_weight);
     return rc ? rc : ssb_launch_status();
 }
@@ -409,5 +409,131 @@ SSB_API int ssb_expert_combine(float* residual, int ldr, const void* y, int ldy,
                         (const bf16*)y, ldy, pair_weight, top, width, total);
     else
         return SSB_ERR_BAD_DTYPE;
+    return rc ? rc : ssb_launch_status();
+}
+
+// ---------------------------------------------------------------------------------------
+// The same sum where it joins the stream through a norm of its own:
+//     v = sum_k pair_weight[t, k] * y[t * top + k],   residual[t] += v / sqrt(mean(v^2) + eps) * w,
+// and optionally the new stream rounded into next_out (what the next sublayer reads).  One block per token; the sums and
+// the stream's row stay in registers for rows of up to 256 x 4 x CN_MAX columns in 16-byte pieces.
+// ---------------------------------------------------------------------------------------
+constexpr int CN_THREADS = 256;
+constexpr int CN_MAX = 4;
+
+__device__ __forceinline__ float cn_block_sum(float v, float* red) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float s = 0.f;
+#pragma unroll
+    for (int w = 0; w < CN_THREADS / 32; ++w) s += red[w];
+    return s;
+}
+
+__device__ __forceinline__ void cn_store4(float* d, float4 o) { *reinterpret_cast<float4*>(d) = o; }
+__device__ __forceinline__ void cn_store4(bf16* d, float4 o) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(o.x, o.y), b = __floats2bfloat162_rn(o.z, o.w);
+    *reinterpret_cast<uint2*>(d) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(CN_THREADS)
+combine_rms_add_vec_kernel(float* __restrict__ residual, const float* __restrict__ y, const float* __restrict__ pair_weight,
+                           int top, const float* __restrict__ w, float eps, int width, T* __restrict__ next_out) {
+    __shared__ float red[CN_THREADS / 32];
+    ssb_pdl_launch_dependents();
+    ssb_pdl_wait();
+    const size_t t = blockIdx.x;
+    const int n4 = width / 4;
+    const float4* y4 = reinterpret_cast<const float4*>(y + t * top * (size_t)width);
+    float4* r4 = reinterpret_cast<float4*>(residual + t * width);
+    const float4* w4 = reinterpret_cast<const float4*>(w);
+    float4 v[CN_MAX], r[CN_MAX], g[CN_MAX];
+    float sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < CN_MAX; ++i) {
+        v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        const int c = threadIdx.x + i * CN_THREADS;
+        if (c < n4) { r[i] = r4[c]; g[i] = w4[c]; }
+    }
+    for (int k = 0; k < top; ++k) {
+        const float p = pair_weight[t * top + k];
+#pragma unroll
+        for (int i = 0; i < CN_MAX; ++i) {
+            const int c = threadIdx.x + i * CN_THREADS;
+            if (c < n4) {
+                const float4 a = y4[(size_t)k * n4 + c];
+                v[i].x = fmaf(p, a.x, v[i].x); v[i].y = fmaf(p, a.y, v[i].y);
+                v[i].z = fmaf(p, a.z, v[i].z); v[i].w = fmaf(p, a.w, v[i].w);
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < CN_MAX; ++i)
+        sq = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, sq))));
+    const float inv = 1.0f / sqrtf(cn_block_sum(sq, red) / (float)width + eps);
+#pragma unroll
+    for (int i = 0; i < CN_MAX; ++i) {
+        const int c = threadIdx.x + i * CN_THREADS;
+        if (c >= n4) continue;
+        float4 o;
+        o.x = r[i].x + v[i].x * inv * g[i].x; o.y = r[i].y + v[i].y * inv * g[i].y;
+        o.z = r[i].z + v[i].z * inv * g[i].z; o.w = r[i].w + v[i].w * inv * g[i].w;
+        r4[c] = o;
+        if (next_out != nullptr) {
+            cn_store4(next_out + t * width + 4 * (size_t)c, o);
+        }
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(CN_THREADS)
+combine_rms_add_kernel(float* __restrict__ residual, const float* __restrict__ y, const float* __restrict__ pair_weight,
+                       int top, const float* __restrict__ w, float eps, int width, T* __restrict__ next_out) {
+    extern __shared__ float cn_row[];
+    __shared__ float red[CN_THREADS / 32];
+    ssb_pdl_launch_dependents();
+    ssb_pdl_wait();
+    const size_t t = blockIdx.x;
+    float sq = 0.f;
+    for (int c = threadIdx.x; c < width; c += CN_THREADS) {
+        float v = 0.f;
+        for (int k = 0; k < top; ++k) v = fmaf(pair_weight[t * top + k], y[(t * top + k) * width + c], v);
+        cn_row[c] = v;
+        sq = fmaf(v, v, sq);
+    }
+    const float inv = 1.0f / sqrtf(cn_block_sum(sq, red) / (float)width + eps);
+    for (int c = threadIdx.x; c < width; c += CN_THREADS) {
+        const float o = residual[t * width + c] + cn_row[c] * inv * w[c];
+        residual[t * width + c] = o;
+        if (next_out != nullptr) next_out[t * width + c] = ssb_from_float<T>(o);
+    }
+}
+
+// residual [tokens, width], y [tokens * top, width], w [width], next_out [tokens, width] or null: all contiguous
+SSB_API int ssb_combine_rms_add(float* residual, const float* y, const float* pair_weight, int top, const float* w, float eps,
+                                int n_tokens, int width, void* next_out, int next_dtype, int pdl, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (top <= 0 || width <= 0 || (size_t)width * sizeof(float) > 200 * 1024) return SSB_ERR_BAD_SIZE;
+    const bool vec = width % 4 == 0 && width <= CN_THREADS * 4 * CN_MAX &&
+        (((uintptr_t)residual | (uintptr_t)y | (uintptr_t)w | (uintptr_t)next_out) & 15) == 0;
+    const size_t smem = vec ? 0 : (size_t)width * sizeof(float);
+    int rc;
+#define SSB_CN(TYPE)                                                                                                  \
+    {                                                                                                                 \
+        auto kern = vec ? combine_rms_add_vec_kernel<TYPE> : combine_rms_add_kernel<TYPE>;                            \
+        if (smem > 48 * 1024) {                                                                                       \
+            cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
+            if (e != cudaSuccess) return (int)e;                                                                      \
+        }                                                                                                             \
+        rc = ssb_launch(kern, dim3(n_tokens), dim3(CN_THREADS), smem, stream, pdl != 0, residual, y, pair_weight,     \
+                        top, w, eps, width, (TYPE*)next_out);                                                         \
+    }
+    if (next_out == nullptr || next_dtype == SSB_F32) SSB_CN(float)
+    else if (next_dtype == SSB_BF16) SSB_CN(bf16)
+    else return SSB_ERR_BAD_DTYPE;
+#undef SSB_CN
     return rc ? rc : ssb_launch_status();
 }

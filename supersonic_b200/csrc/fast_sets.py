@@ -358,18 +358,18 @@ class FastKernels(PlainKernels):
     # 64 x 520 keys: 55 us unsplit, 40 in 2 splits, 49 in 4; 8 x 520: 53, 37, 26, 24 and 22 us in 1, 2, 4, 8 and 16)
     LATENT_SPLIT_BLOCKS = 148
 
-    def head_linear(self, x, w, out):
+    def head_linear(self, x, w, out, gate=None):
         if ops.head_gemm_mma_ok(x, w, out):
-            ops.head_gemm_mma(x, w, out, pdl=self.pdl)
+            ops.head_gemm_mma(x, w, out, pdl=self.pdl, gate=gate)
         else:
-            super().head_linear(x, w, out)
+            super().head_linear(x, w, out, gate)
 
     def latent_prepare(self, proj, c_off, q_abs, norm_w, eps, position, batch, page_table, cache, n_heads, dim,
-                       rot_dim, kv_rank, page_shift, write_cache=True):
+                       rot_dim, kv_rank, page_shift, write_cache=True, q_latent=None):
         cos, sin, rot_dims = position.rotary_tables()
         ops.latent_prepare(proj, c_off, q_abs, norm_w, eps, cos, sin, batch.pos, batch.slot_of_token, page_table,
                            cache, n_heads, dim, rot_dim, rot_dims, kv_rank, page_shift, write_cache,
-                           getattr(position, "interleaved", False), pdl=self.pdl)
+                           getattr(position, "interleaved", False), pdl=self.pdl, q_latent=q_latent)
 
     def latent_attention(self, q_abs, cache, batch, page_table, out, n_heads, kv_rank, rot_dim, page_shift,
                          window, scale, sinks):
@@ -455,18 +455,19 @@ class FastKernels(PlainKernels):
     def route_table(self, token_ids, table, n_experts, expert_of, pair_weight):
         ops.route_table(token_ids, table, n_experts, expert_of, pair_weight, pdl=self.pdl)
 
-    def route_softmax(self, x, weight, n_experts, renormalize, scale, expert_of, pair_weight):
+    def route_softmax(self, x, weight, n_experts, renormalize, scale, expert_of, pair_weight, bias=None):
         rows, n = x.shape[0], weight.shape[0]
         if rows > STREAM_ROWS or self.deterministic:
-            super().route_softmax(x, weight, n_experts, renormalize, scale, expert_of, pair_weight)
+            super().route_softmax(x, weight, n_experts, renormalize, scale, expert_of, pair_weight, bias)
             return
         # a few rows: K is split over blocks that add into sums which are zero between uses (the choice clears its rows)
         logits = self._buffer("router_sums", rows * n, torch.float32, x.device, zero=True)[: rows * n].view(rows, n)
         if not ops.gemm_tc_ok(x, weight, logits):
-            super().route_softmax(x, weight, n_experts, renormalize, scale, expert_of, pair_weight)
+            super().route_softmax(x, weight, n_experts, renormalize, scale, expert_of, pair_weight, bias)
             return
         ops.gemv_tc(x, weight, logits, ops.TC_ACCUMULATE, splits=ops.gemv_tc_splits(n, weight.shape[1]), pdl=self.pdl)
-        ops.route_softmax(logits, n_experts, renormalize, scale, expert_of, pair_weight, clear=True, pdl=self._chain(rows))
+        ops.route_softmax(logits, n_experts, renormalize, scale, expert_of, pair_weight, clear=True, pdl=self._chain(rows),
+                          bias=bias)
 
     def group_by_expert(self, expert_of, n_experts, groups):
         ops.group_by_expert(expert_of, n_experts, groups["tile_rows"], groups["offsets"], groups["order"],
@@ -487,6 +488,13 @@ class FastKernels(PlainKernels):
                                  ops.GG_SWIGLU, pdl=self.pdl, act=act)
         else:
             super().expert_gate_up(x, top, w_gate_up, out, groups, act)
+
+    def expert_up(self, x, top, w_up, out, groups, act):
+        if ops.grouped_gemm_mma_ok(x, w_up, out, ops.GG_ACT):
+            ops.grouped_gemm_mma(x, groups["order"], top, w_up, out, None, groups["offsets"], groups["tile_expert"],
+                                 groups["tile_row0"], groups["meta"], groups["max_tiles"], ops.GG_ACT, pdl=self.pdl, act=act)
+        else:
+            super().expert_up(x, top, w_up, out, groups, act)
 
     def expert_combine(self, residual, y, pair_weight, top):
         ops.expert_combine(residual, y, pair_weight, top, pdl=self.pdl)

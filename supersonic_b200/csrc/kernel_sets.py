@@ -62,8 +62,8 @@ class PlainKernels:
     def _chain(self, rows) -> bool:
         return bool(self.pdl) and int(rows) <= self.PDL_MAX_ROWS
 
-    def embed(self, ids, table, out, scale=1.0):
-        ops.embed(ids, table, out, scale)
+    def embed(self, ids, table, out, scale=1.0, rounded=None):
+        ops.embed(ids, table, out, scale, rounded)
 
     def embed_norm(self, ids, table, weight, eps, out, scale=1.0):
         ops.embed_norm(ids, table, weight, eps, out, scale)
@@ -91,9 +91,17 @@ class PlainKernels:
 
     def rms_add(self, residual, branch, weight, eps, clear=False, next_norm=None, next_out=None):
         """residual += rmsnorm(branch) * weight; with ``next_norm`` (an RMS norm part) its output of the new stream
-        into ``next_out`` in the same pass."""
+        into ``next_out`` in the same pass; ``next_out`` alone: the new stream rounded to its type."""
         ops.rms_add(residual, branch, weight, eps, clear, None if next_norm is None else next_norm.weight_f32,
                     0.0 if next_norm is None else next_norm.eps, next_out, pdl=self._chain(residual.shape[0]))
+
+    def round_rows(self, x, out):
+        """float32 rows in out's type."""
+        ops.round_rows(x, out, pdl=self._chain(x.shape[0]))
+
+    def combine_rms_add(self, residual, y, pair_weight, top, weight, eps, next_out=None):
+        """residual += rmsnorm(sum_k pair_weight[:, k] y[k-th choice]) * weight; the new stream rounded into ``next_out``."""
+        ops.combine_rms_add(residual, y, pair_weight, top, weight, eps, next_out, pdl=self._chain(residual.shape[0]))
 
     def stream_enter(self, src, streams, in_weights, branch, write, dst, norm, conv, tail, batch, out):
         """A sublayer's entry over several residual streams: the write of the sublayer before (``write`` = (mix,
@@ -144,18 +152,22 @@ class PlainKernels:
         ops.swiglu(gate_up, out)
 
     # ---- latent attention ------------------------------------------------------------
-    def head_linear(self, x, w, out):
+    def head_linear(self, x, w, out, gate=None):
         """out[t, h] = w[h] @ x[t, h]: a matrix per head (``x`` [T, H, K] and ``out`` [T, H, N] may be views
-        into wider rows, ``w`` [H, N, K])."""
+        into wider rows, ``w`` [H, N, K]); with ``gate`` [T, H x N] times sigmoid(gate) element by element (``out`` then
+        holds whole rows)."""
         ops.head_linear_plain(x, w, out)
+        if gate is not None:
+            ops.sigmoid_gate(out.view(out.shape[0], -1), gate, pdl=self._chain(out.shape[0]))
 
     def latent_prepare(self, proj, c_off, q_abs, norm_w, eps, position, batch, page_table, cache, n_heads, dim,
-                       rot_dim, kv_rank, page_shift, write_cache=True):
-        """Rotated query parts into ``q_abs``; the token's cache row [normed latent | rotated key part]."""
+                       rot_dim, kv_rank, page_shift, write_cache=True, q_latent=None):
+        """Rotated query parts into ``q_abs``; the token's cache row [normed latent | rotated key part].  With ``n_heads`` 0
+        no queries; ``q_latent`` = (offset, rank, weight) norms a query latent in place."""
         cos, sin, rot_dims = position.rotary_tables()
         ops.latent_prepare(proj, c_off, q_abs, norm_w, eps, cos, sin, batch.pos, batch.slot_of_token, page_table,
                            cache, n_heads, dim, rot_dim, rot_dims, kv_rank, page_shift, write_cache,
-                           getattr(position, "interleaved", False))
+                           getattr(position, "interleaved", False), pdl=self._chain(batch.n_tokens), q_latent=q_latent)
 
     def latent_attention(self, q_abs, cache, batch, page_table, out, n_heads, kv_rank, rot_dim, page_shift,
                          window, scale, sinks):
@@ -361,11 +373,11 @@ class PlainKernels:
         ops.route_sigmoid_groups(logits, n_experts, correction, n_groups, keep, scale, expert_of, pair_weight, extra_col,
                                  extra_out, pdl=self._chain(logits.shape[0]))
 
-    def route_softmax(self, x, weight, n_experts, renormalize, scale, expert_of, pair_weight):
-        """The router's product (logits x @ weight^T in float32) and the choice."""
+    def route_softmax(self, x, weight, n_experts, renormalize, scale, expert_of, pair_weight, bias=None):
+        """The router's product (logits x @ weight^T + bias in float32) and the choice."""
         logits = torch.empty((x.shape[0], weight.shape[0]), dtype=torch.float32, device=x.device)
         self.linear(x, weight, logits)
-        ops.route_softmax(logits, n_experts, renormalize, scale, expert_of, pair_weight, pdl=self._chain(logits.shape[0]))
+        ops.route_softmax(logits, n_experts, renormalize, scale, expert_of, pair_weight, pdl=self._chain(logits.shape[0]), bias=bias)
 
     def group_by_expert(self, expert_of, n_experts, groups):
         """``groups``: the dict of int32 tensors a grouped product reads (offsets, order, tile_expert,
@@ -388,6 +400,11 @@ class PlainKernels:
         self.grouped_linear(x, True, top, w_gate_up, gate_up, False, groups)
         kind, limit = act if act else ("silu", 0.0)
         ops.gated_activation(gate_up, out, kind, limit, pdl=self._chain(out.shape[0]))
+
+    def expert_up(self, x, top, w_up, out, groups, act):
+        """out[sorted row] = act(x up_e^T) for the row's expert e: an expert without a gate; ``w_up`` [E, inter, hidden]."""
+        self.grouped_linear(x, True, top, w_up, out, False, groups)
+        ops.activation(out, out, act, 1.0, pdl=self._chain(out.shape[0]))
 
     def expert_combine(self, residual, y, pair_weight, top):
         ops.expert_combine(residual, y, pair_weight, top)

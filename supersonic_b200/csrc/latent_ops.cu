@@ -5,6 +5,8 @@
 // token's cache row [rms(first kv_rank) * w | rotate(last rot_dim)] at its position, and the
 // rotated rot_dim tails of the H queries behind the latent-space queries in q_abs.  The attention
 // that follows works on these rows directly (see parts/latent_attention.py for the algebra).
+// Where the queries go through a latent of their own, the kernel runs twice: before the queries exist (no heads), when
+// it norms the query latent in place and writes the cache row, and behind them, for their rotated parts alone.
 // All arithmetic is float32.
 #include "common.cuh"
 #include <math.h>
@@ -18,7 +20,8 @@ latent_prepare_kernel(T* __restrict__ proj, int ld, int c_off, T* __restrict__ q
                       const float* __restrict__ sin_t, int table_positions, const int* __restrict__ pos,
                       const int* __restrict__ slot, const int* __restrict__ page_table, int max_pages,
                       T* __restrict__ cache, int n_heads, int dim, int rot_dim, int rot_dims, int kv_rank,
-                      int page_shift, int write_cache, int interleaved) {
+                      int page_shift, int write_cache, int interleaved, int q_lat_off, int q_rank,
+                      const TW* __restrict__ q_norm_w) {
     __shared__ float red[256];
     const int t = blockIdx.x, tid = threadIdx.x;
     ssb_pdl_launch_dependents();
@@ -34,7 +37,7 @@ latent_prepare_kernel(T* __restrict__ proj, int ld, int c_off, T* __restrict__ q
     // queries: the rotated part of every head turned by the token's position, written behind the
     // head's latent-space query in q_abs ([head][kv_rank | rot_dim])
     const int qw = dim + rot_dim, aw = kv_rank + rot_dim;
-    T* qa = q_abs + (size_t)t * ldq;
+    T* qa = n_heads > 0 ? q_abs + (size_t)t * ldq : nullptr;
     for (int e = tid; e < n_heads * rot_dim; e += 256) {
         const int h = e / rot_dim, i = e % rot_dim;
         const T* x = row + (size_t)h * qw + dim;
@@ -50,21 +53,31 @@ latent_prepare_kernel(T* __restrict__ proj, int ld, int c_off, T* __restrict__ q
         }
         qa[(size_t)h * aw + kv_rank + i] = ssb_from_float<T>(v);
     }
+    auto mean_square = [&](const T* v, int n) {
+        float part = 0.f;
+        for (int c = tid; c < n; c += 256) {
+            const float x = ssb_to_float(v[c]);
+            part = fmaf(x, x, part);
+        }
+        red[tid] = part;
+        __syncthreads();
+        for (int st = 128; st > 0; st >>= 1) {
+            if (tid < st) red[tid] += red[tid + st];
+            __syncthreads();
+        }
+        const float ms = red[0] / (float)n;
+        __syncthreads();
+        return ms;
+    };
+    if (q_rank > 0) {                                    // the query latent, normed in place: a thread reads what it writes
+        T* ql = row + q_lat_off;
+        const float inv = 1.0f / sqrtf(mean_square(ql, q_rank) + eps);
+        for (int c = tid; c < q_rank; c += 256) ql[c] = ssb_from_float<T>(ssb_to_float(ql[c]) * inv * ssb_to_float(q_norm_w[c]));
+    }
     if (!write_cache) return;
     // the latent: x / sqrt(mean(x^2) + eps) * w
     const T* lat = row + c_off;
-    float part = 0.f;
-    for (int c = tid; c < kv_rank; c += 256) {
-        const float v = ssb_to_float(lat[c]);
-        part = fmaf(v, v, part);
-    }
-    red[tid] = part;
-    __syncthreads();
-    for (int st = 128; st > 0; st >>= 1) {
-        if (tid < st) red[tid] += red[tid + st];
-        __syncthreads();
-    }
-    const float inv = 1.0f / sqrtf(red[0] / (float)kv_rank + eps);
+    const float inv = 1.0f / sqrtf(mean_square(lat, kv_rank) + eps);
     T* dst = cache + ssb_cache_row(page_table, max_pages, s, p, page_shift, 1, 0, aw);
     for (int c = tid; c < kv_rank; c += 256)
         dst[c] = ssb_from_float<T>(ssb_to_float(lat[c]) * inv * ssb_to_float(norm_w[c]));
@@ -85,19 +98,23 @@ latent_prepare_kernel(T* __restrict__ proj, int ld, int c_off, T* __restrict__ q
 }
 
 // proj [T, ld]: queries from column 0, the low-rank row from column c_off; q_abs [T, ldq] gets the
-// rotated query parts; the cache entry [pages][1][tokens][kv_rank + rot_dim] gets the token's row
+// rotated query parts (none with n_heads 0); the cache entry [pages][1][tokens][kv_rank + rot_dim] gets the token's row;
+// q_rank > 0: the columns from q_lat_off are normed in place with q_norm_w
 SSB_API int ssb_latent_prepare(void* proj, int ld, int c_off, void* q_abs, int ldq, int dtype, const void* norm_w,
                                int w_dtype, float eps, const float* cos_t, const float* sin_t, int table_positions,
                                const int* pos, const int* slot, const int* page_table, int max_pages, void* cache,
                                int n_tokens, int n_heads, int dim, int rot_dim, int rot_dims, int kv_rank,
-                               int page_shift, int write_cache, int interleaved, int pdl, cudaStream_t stream) {
+                               int page_shift, int write_cache, int interleaved, int q_lat_off, int q_rank,
+                               const void* q_norm_w, int pdl, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (rot_dims % 2 || rot_dims > rot_dim || rot_dims < 0 || kv_rank <= 0) return SSB_ERR_BAD_SIZE;
+    if (rot_dims % 2 || rot_dims > rot_dim || rot_dims < 0 || kv_rank <= 0 || n_heads < 0 || q_rank < 0 ||
+        (n_heads > 0 && q_abs == nullptr) || (q_rank > 0 && q_norm_w == nullptr)) return SSB_ERR_BAD_SIZE;
     int rc = 0;
 #define SSB_PREP(T, TW) \
     rc = ssb_launch(latent_prepare_kernel<T, TW>, dim3(n_tokens), dim3(256), 0, stream, pdl != 0, (T*)proj, ld, c_off, \
                     (T*)q_abs, ldq, (const TW*)norm_w, eps, cos_t, sin_t, table_positions, pos, slot, page_table,  \
-                    max_pages, (T*)cache, n_heads, dim, rot_dim, rot_dims, kv_rank, page_shift, write_cache, interleaved)
+                    max_pages, (T*)cache, n_heads, dim, rot_dim, rot_dims, kv_rank, page_shift, write_cache, interleaved,  \
+                    q_lat_off, q_rank, (const TW*)q_norm_w)
     if (dtype == SSB_F32 && w_dtype == SSB_F32) SSB_PREP(float, float);
     else if (dtype == SSB_BF16 && w_dtype == SSB_BF16) SSB_PREP(bf16, bf16);
     else if (dtype == SSB_BF16 && w_dtype == SSB_F32) SSB_PREP(bf16, float);

@@ -83,15 +83,21 @@ def _fn(lib: str, name: str):
 
 
 # ---- plain ops -------------------------------------------------------------------------
-def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
-    """out[t] = table[ids[t]] * scale into the float32 residual stream (the product is float32)."""
+def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: float = 1.0,
+          rounded: Optional[torch.Tensor] = None) -> None:
+    """out[t] = table[ids[t]] * scale into the float32 residual stream (the product is float32); with ``rounded`` the
+    same rows in the table's type too."""
     _need(ids, "ids", torch.int32, 1); _need(table, "table", None, 2); _need(out, "out", torch.float32, 2)
     if not (table.is_contiguous() and out.is_contiguous()):
         raise KernelError("embed: table and out must be contiguous")
     if out.shape[0] != ids.shape[0] or out.shape[1] != table.shape[1]:
         raise KernelError(f"embed: out {tuple(out.shape)} does not fit {ids.shape[0]} ids of width {table.shape[1]}")
+    if rounded is not None:
+        _need(rounded, "rounded", table.dtype, 2)
+        if rounded.shape != out.shape or not rounded.is_contiguous():
+            raise KernelError("embed: rounded must be contiguous, of out's shape")
     _check(_fn("plain_ops", "ssb_embed_scaled")(
-        _ptr(ids), _ptr(table), c_int(dtype_code(table.dtype)), _ptr(out), c_int(ids.shape[0]),
+        _ptr(ids), _ptr(table), c_int(dtype_code(table.dtype)), _ptr(out), _ptr(rounded), c_int(ids.shape[0]),
         c_int(table.shape[1]), c_int(table.shape[0]), c_float(scale), _stream()), "embed")
 
 
@@ -254,20 +260,64 @@ def rms_add(residual: torch.Tensor, branch: torch.Tensor, weight: torch.Tensor, 
             pdl: bool = False) -> None:
     """residual[t] += branch[t] / sqrt(mean(branch[t]^2) + eps) * weight (both float32; ``weight`` is the multiplier
     itself).  ``clear``: the branch is zeroed behind the read.  With ``next_out``: next_out[t] = the new residual[t]
-    / sqrt(mean(.^2) + next_eps) * next_weight, the norm the next sublayer reads."""
+    / sqrt(mean(.^2) + next_eps) * next_weight, the norm the next sublayer reads; without ``next_weight`` the new
+    residual[t] itself, rounded to next_out's type."""
     _need(residual, "residual", torch.float32, 2); _need(branch, "branch", torch.float32, 2)
     _need(weight, "weight", torch.float32, 1)
     T, W = residual.shape
     if tuple(branch.shape) != (T, W) or weight.shape[0] != W or not (residual.is_contiguous() and branch.is_contiguous()):
         raise KernelError("rms_add: residual and branch [tokens, width] contiguous, one weight per column")
     if next_out is not None:
-        _need(next_out, "next_out", None, 2); _need(next_weight, "next_weight", torch.float32, 1)
-        if tuple(next_out.shape) != (T, W) or next_weight.shape[0] != W or not next_out.is_contiguous():
+        _need(next_out, "next_out", None, 2)
+        if next_weight is not None:
+            _need(next_weight, "next_weight", torch.float32, 1)
+        if tuple(next_out.shape) != (T, W) or (next_weight is not None and next_weight.shape[0] != W) \
+                or not next_out.is_contiguous():
             raise KernelError("rms_add: next_out [tokens, width] contiguous, one weight per column")
     _check(_fn("plain_ops", "ssb_rms_add")(
         _ptr(residual), _ptr(branch), _ptr(weight), c_float(eps), c_int(T), c_int(W), c_int(1 if clear else 0),
         _ptr(next_weight if next_out is not None else None), c_float(next_eps), _ptr(next_out),
         c_int(dtype_code(next_out.dtype) if next_out is not None else F32), c_int(1 if pdl else 0), _stream()), "rms_add")
+
+
+def combine_rms_add(residual: torch.Tensor, y: torch.Tensor, pair_weight: torch.Tensor, top: int, weight: torch.Tensor,
+                    eps: float, next_out: Optional[torch.Tensor] = None, pdl: bool = False) -> None:
+    """With v[t] = sum_k pair_weight[t, k] * y[t * top + k] (in the order of k): residual[t] += v[t] / sqrt(mean(v[t]^2) +
+    eps) * weight; ``next_out``: the new residual[t] in next_out's type."""
+    _need(residual, "residual", torch.float32, 2); _need(y, "y", torch.float32, 2)
+    _need(pair_weight, "pair_weight", torch.float32, 2); _need(weight, "weight", torch.float32, 1)
+    T, W = residual.shape
+    if tuple(y.shape) != (T * top, W) or tuple(pair_weight.shape) != (T, top) or weight.shape[0] != W \
+            or not (residual.is_contiguous() and y.is_contiguous() and pair_weight.is_contiguous()):
+        raise KernelError("combine_rms_add: residual [tokens, width], y [tokens * top, width], pair_weight [tokens, top]")
+    if next_out is not None:
+        _need(next_out, "next_out", None, 2)
+        if tuple(next_out.shape) != (T, W) or not next_out.is_contiguous():
+            raise KernelError("combine_rms_add: next_out must be [tokens, width], contiguous")
+    _check(_fn("expert_ops", "ssb_combine_rms_add")(
+        _ptr(residual), _ptr(y), _ptr(pair_weight), c_int(top), _ptr(weight), c_float(eps), c_int(T), c_int(W),
+        _ptr(next_out), c_int(dtype_code(next_out.dtype) if next_out is not None else F32), c_int(1 if pdl else 0),
+        _stream()), "combine_rms_add")
+
+
+def round_rows(x: torch.Tensor, out: torch.Tensor, pdl: bool = False) -> None:
+    """out = x rounded to out's type (x float32, both contiguous)."""
+    _need(x, "x", torch.float32, 2); _need(out, "out", None, 2)
+    if x.shape != out.shape or not (x.is_contiguous() and out.is_contiguous()):
+        raise KernelError("round_rows: contiguous rows of one shape")
+    _check(_fn("plain_ops", "ssb_round_rows")(
+        _ptr(x), _ptr(out), c_int(dtype_code(out.dtype)), c_longlong(x.numel()), c_int(1 if pdl else 0), _stream()),
+        "round_rows")
+
+
+def sigmoid_gate(y: torch.Tensor, gate: torch.Tensor, pdl: bool = False) -> None:
+    """y[t, c] *= sigmoid(gate[t, c])."""
+    _need(y, "y", None, 2); _need(gate, "gate", y.dtype, 2)
+    if y.shape != gate.shape:
+        raise KernelError("sigmoid_gate: one gate per element")
+    _check(_fn("plain_ops", "ssb_sigmoid_gate")(
+        _ptr(y), c_int(y.stride(0)), _ptr(gate), c_int(gate.stride(0)), c_int(dtype_code(y.dtype)), c_int(y.shape[0]),
+        c_int(y.shape[1]), c_int(1 if pdl else 0), _stream()), "sigmoid_gate")
 
 
 def add_into(out: torch.Tensor, x: torch.Tensor) -> None:
@@ -321,37 +371,46 @@ def head_linear_plain(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> No
 
 
 # ---- latent attention ------------------------------------------------------------------
-def latent_prepare(proj: torch.Tensor, c_off: int, q_abs: torch.Tensor, norm_w: torch.Tensor, eps: float,
+def latent_prepare(proj: torch.Tensor, c_off: int, q_abs: Optional[torch.Tensor], norm_w: torch.Tensor, eps: float,
                    cos: torch.Tensor, sin: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor,
                    page_table: torch.Tensor, cache: Optional[torch.Tensor], n_heads: int, dim: int, rot_dim: int,
                    rot_dims: int, kv_rank: int, page_shift: int, write_cache: bool = True,
-                   interleaved: bool = True, pdl: bool = False) -> None:
+                   interleaved: bool = True, pdl: bool = False, q_latent=None) -> None:
     """From a token's projected row ``proj`` ([queries: heads x (dim + rot_dim) | from ``c_off``: kv_rank latent,
     rot_dim key part]): the rotated query parts into ``q_abs`` ([heads x (kv_rank + rot_dim)], behind each
     head's first kv_rank columns), and the token's cache row [RMS-normed latent * norm_w | rotated key part]
-    at its position.  The first ``rot_dims`` coordinates of a rotated part turn, the rest pass."""
-    _need(proj, "proj", None, 2); _need(q_abs, "q_abs", proj.dtype, 2); _need(norm_w, "norm_w", None, 1)
+    at its position.  The first ``rot_dims`` coordinates of a rotated part turn, the rest pass.  ``n_heads`` 0: no
+    queries in the row (and no ``q_abs``).  ``q_latent`` = (offset, rank, weight): those columns are RMS-normed in place
+    times the weight, the latent that the queries are made from behind this call."""
+    _need(proj, "proj", None, 2); _need(norm_w, "norm_w", None, 1)
+    if n_heads:
+        _need(q_abs, "q_abs", proj.dtype, 2)
+    q_off, q_rank, q_norm_w = q_latent if q_latent is not None else (0, 0, None)
+    if q_latent is not None:
+        _need(q_norm_w, "q_norm_w", norm_w.dtype, 1)
+        if q_norm_w.shape[0] != q_rank or q_off < 0 or q_off + q_rank > proj.shape[1]:
+            raise KernelError("latent_prepare: the query latent's columns")
     _need(cos, "cos", torch.float32, 2); _need(sin, "sin", torch.float32, 2)
     _need(pos, "pos", torch.int32, 1); _need(slot, "slot", torch.int32, 1); _need(page_table, "page_table", torch.int32, 2)
     T = proj.shape[0]
-    if proj.shape[1] < max(n_heads * (dim + rot_dim), c_off + kv_rank + rot_dim) or \
-            q_abs.shape[0] != T or q_abs.shape[1] < n_heads * (kv_rank + rot_dim):
+    if proj.shape[1] < max(n_heads * (dim + rot_dim), c_off + kv_rank + rot_dim if write_cache else 0) or \
+            (n_heads and (q_abs.shape[0] != T or q_abs.shape[1] < n_heads * (kv_rank + rot_dim))):
         raise KernelError("latent_prepare: rows are too narrow")
     if cos.shape != sin.shape or cos.shape[1] * 2 != rot_dims or not (cos.is_contiguous() and sin.is_contiguous()):
         raise KernelError("latent_prepare: cos/sin must be [positions, rot_dims/2], contiguous")
-    if norm_w.shape[0] != kv_rank or pos.shape[0] != T or slot.shape[0] != T:
+    if (write_cache and norm_w.shape[0] != kv_rank) or pos.shape[0] != T or slot.shape[0] != T:
         raise KernelError("latent_prepare: sizes")
     if write_cache:
         _need(cache, "cache", proj.dtype)
         if not cache.is_contiguous() or cache.shape[-1] != kv_rank + rot_dim:
             raise KernelError("latent_prepare: the cache entry must be contiguous with rows of kv_rank + rot_dim")
     _check(_fn("latent_ops", "ssb_latent_prepare")(
-        _ptr(proj), c_int(proj.stride(0)), c_int(c_off), _ptr(q_abs), c_int(q_abs.stride(0)),
+        _ptr(proj), c_int(proj.stride(0)), c_int(c_off), _ptr(q_abs), c_int(q_abs.stride(0) if n_heads else 0),
         c_int(dtype_code(proj.dtype)), _ptr(norm_w), c_int(dtype_code(norm_w.dtype)), c_float(eps), _ptr(cos),
         _ptr(sin), c_int(cos.shape[0]), _ptr(pos), _ptr(slot), _ptr(page_table), c_int(page_table.shape[1]),
         _ptr(cache), c_int(T), c_int(n_heads), c_int(dim), c_int(rot_dim), c_int(rot_dims), c_int(kv_rank),
-        c_int(page_shift), c_int(1 if write_cache else 0), c_int(1 if interleaved else 0), c_int(1 if pdl else 0),
-        _stream()), "latent_prepare")
+        c_int(page_shift), c_int(1 if write_cache else 0), c_int(1 if interleaved else 0), c_int(q_off), c_int(q_rank),
+        _ptr(q_norm_w), c_int(1 if pdl else 0), _stream()), "latent_prepare")
 
 
 def latent_attention_mma_ok(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, n_heads: int, dk: int, dv: int,
@@ -406,19 +465,26 @@ def head_gemm_mma_ok(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> boo
             and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def head_gemm_mma(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, pdl: bool = False) -> None:
-    """``head_linear_plain`` on mma.sync: out[t, h] = w[h] @ x[t, h] for bfloat16 operands."""
+def head_gemm_mma(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, pdl: bool = False,
+                  gate: Optional[torch.Tensor] = None) -> None:
+    """``head_linear_plain`` on mma.sync: out[t, h] = w[h] @ x[t, h] for bfloat16 operands; with ``gate`` [T, H x N] times
+    the sigmoid of the element's gate, on the float32 sums."""
     T, H, K = x.shape
     N = w.shape[1]
     if not head_gemm_mma_ok(x, w, out) or tuple(w.shape) != (H, N, K) or tuple(out.shape) != (T, H, N):
         raise KernelError(f"head_gemm_mma: x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
+    if gate is not None:
+        _need(gate, "gate", torch.bfloat16, 2)
+        if tuple(gate.shape) != (T, H * N):
+            raise KernelError("head_gemm_mma: one gate per element of the concatenated heads")
     _check(_fn("batched_gemm", "ssb_head_gemm_mma")(
         _ptr(x), c_int(x.stride(0)), c_longlong(x.stride(1)), _ptr(w), c_int(K), c_longlong(N * K), _ptr(out),
         c_int(out.stride(0)), c_longlong(out.stride(1)), c_int(dtype_code(out.dtype)), c_int(H), c_int(T), c_int(N),
-        c_int(K), c_int(1 if pdl else 0), _stream()), "head_gemm_mma")
+        c_int(K), _ptr(gate), c_int(gate.stride(0) if gate is not None else 0), c_int(1 if pdl else 0), _stream()),
+        "head_gemm_mma")
 
 
-GG_STORE, GG_SWIGLU = 0, 1
+GG_STORE, GG_SWIGLU, GG_ACT = 0, 1, 2
 
 
 def order_rows(a, a_index, out, c_index) -> int:
@@ -430,7 +496,7 @@ def grouped_gemm_mma_ok(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mod
     return (a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous() and a.shape[1] % 8 == 0
             and a.stride(0) % 8 == 0 and a.stride(1) == 1 and out.stride(1) == 1 and a.data_ptr() % 16 == 0
             and w.data_ptr() % 16 == 0 and (w.shape[1] * w.shape[2]) % 8 == 0
-            and (out.dtype == torch.bfloat16 or (mode == GG_STORE and out.dtype == torch.float32)))
+            and (out.dtype == torch.bfloat16 or (mode != GG_SWIGLU and out.dtype == torch.float32)))
 
 
 def grouped_gemm_mma(a: torch.Tensor, a_index: Optional[torch.Tensor], a_div: int, w: torch.Tensor,
@@ -439,10 +505,13 @@ def grouped_gemm_mma(a: torch.Tensor, a_index: Optional[torch.Tensor], a_div: in
                      mode: int = GG_STORE, pdl: bool = False, act=None) -> None:
     """``grouped_gemm_plain`` on mma.sync (tiles of 64 rows).  mode GG_SWIGLU: ``w`` [E, 2N, K] holds gate rows then
     up rows and ``out`` [rows, N] gets silu(a gate^T) * (a up^T), or with ``act`` = (kind, limit) that inner step of
-    the gated unit (``gated_activation``)."""
-    kind, limit = act if act else ("silu", 0.0)
-    if kind not in GATE_KINDS_FF:
-        raise KernelError(f"grouped_gemm_mma: gate {kind!r} is not known (known: {sorted(GATE_KINDS_FF)})")
+    the gated unit (``gated_activation``).  mode GG_ACT: ``act`` names an activation on the sums (``ACTIVATIONS``)."""
+    if mode == GG_ACT:
+        kinds, kind, limit = ACTIVATIONS, act, 0.0
+    else:
+        kinds, (kind, limit) = GATE_KINDS_FF, act if act else ("silu", 0.0)
+    if kind not in kinds:
+        raise KernelError(f"grouped_gemm_mma: {kind!r} is not known (known: {sorted(kinds)})")
     E, n_w, K = w.shape
     N = n_w // 2 if mode == GG_SWIGLU else n_w
     if not grouped_gemm_mma_ok(a, w, out, mode) or a.shape[1] != K or out.shape[1] != N:
@@ -451,7 +520,7 @@ def grouped_gemm_mma(a: torch.Tensor, a_index: Optional[torch.Tensor], a_div: in
         _ptr(a), c_int(a.stride(0)), _ptr(a_index), c_int(a_div), _ptr(w), c_int(K), c_longlong(n_w * K), _ptr(out),
         c_int(out.stride(0)), _ptr(c_index), c_int(dtype_code(out.dtype)), _ptr(offsets), _ptr(tile_expert),
         _ptr(tile_row0), _ptr(meta), c_int(max_tiles), c_int(order_rows(a, a_index, out, c_index)), c_int(N), c_int(K),
-        c_int(mode), c_int(GATE_KINDS_FF[kind]), c_float(limit), c_int(1 if pdl else 0), _stream()), "grouped_gemm_mma")
+        c_int(mode), c_int(kinds[kind]), c_float(limit), c_int(1 if pdl else 0), _stream()), "grouped_gemm_mma")
 
 
 # ---- linear recurrences ----------------------------------------------------------------
@@ -1426,18 +1495,23 @@ def route_sigmoid_groups(logits: torch.Tensor, n_experts: int, correction: Optio
 
 
 def route_softmax(logits: torch.Tensor, n_experts: int, renormalize: bool, scale: float, expert_of: torch.Tensor,
-                  pair_weight: torch.Tensor, clear: bool = False, pdl: bool = False) -> None:
-    """Per token, from float32 router logits [tokens, >= n_experts]: s = softmax(z) over all experts; the ``top`` experts
+                  pair_weight: torch.Tensor, clear: bool = False, pdl: bool = False,
+                  bias: Optional[torch.Tensor] = None) -> None:
+    """Per token, from float32 router logits [tokens, >= n_experts]: s = softmax(z + bias) over all experts; the ``top`` experts
     with the largest s; pair_weight = s * scale, with ``renormalize`` divided by the chosen scores' sum (+ 1e-20).
     ``clear``: the logits' rows are zeroed behind the read."""
     _need(logits, "logits", torch.float32, 2)
     _need(expert_of, "expert_of", torch.int32, 2); _need(pair_weight, "pair_weight", torch.float32, 2)
     T, top = logits.shape[0], expert_of.shape[1]
+    if bias is not None:
+        _need(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != n_experts:
+            raise KernelError("route_softmax: one bias per expert")
     if logits.shape[1] < n_experts or not 1 <= top <= n_experts or tuple(expert_of.shape) != (T, top) \
             or tuple(pair_weight.shape) != (T, top) or not (expert_of.is_contiguous() and pair_weight.is_contiguous()):
         raise KernelError("route_softmax: logits [tokens, >= experts]; expert_of and pair_weight [tokens, top], contiguous")
     _check(_fn("expert_ops", "ssb_route_softmax")(
-        _ptr(logits), c_int(logits.stride(0)), c_int(T), c_int(n_experts), c_int(top), c_int(1 if renormalize else 0),
+        _ptr(logits), c_int(logits.stride(0)), _ptr(bias), c_int(T), c_int(n_experts), c_int(top), c_int(1 if renormalize else 0),
         c_float(scale), c_int(1 if clear else 0), _ptr(expert_of), _ptr(pair_weight), c_int(1 if pdl else 0), _stream()),
         "route_softmax")
 

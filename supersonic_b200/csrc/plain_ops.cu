@@ -19,32 +19,45 @@
 typedef __nv_bfloat16 bf16;
 
 // ---------------------------------------------------------------------------------------
-// embedding: out[t, :] = table[ids[t], :] * scale, written into the float32 residual stream
+// embedding: out[t, :] = table[ids[t], :] * scale, written into the float32 residual stream; optionally the same row in
+// the table's type (what a first sublayer without a norm in front of it reads)
 // ---------------------------------------------------------------------------------------
 template <typename T>
 __global__ void embed_kernel(const int* __restrict__ ids, const T* __restrict__ table,
-                             float* __restrict__ out, int hidden, int vocab, float scale) {
+                             float* __restrict__ out, T* __restrict__ rounded, int hidden, int vocab, float scale) {
     const int t = blockIdx.x;
     const int id = ids[t];
     float* dst = out + (size_t)t * hidden;
+    T* dst_r = rounded ? rounded + (size_t)t * hidden : nullptr;
     if (id < 0 || id >= vocab) {          // the host refuses such ids; never read out of range
-        for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = 0.f;
+        for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+            dst[c] = 0.f;
+            if (dst_r) dst_r[c] = ssb_from_float<T>(0.f);
+        }
         return;
     }
     const T* src = table + (size_t)id * hidden;
+    if (dst_r) {
+        for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+            const float v = ssb_to_float(src[c]) * scale;
+            dst[c] = v;
+            dst_r[c] = ssb_from_float<T>(v);
+        }
+        return;
+    }
     if (scale == 1.0f)
         for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = ssb_to_float(src[c]);
     else
         for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = ssb_to_float(src[c]) * scale;
 }
 
-SSB_API int ssb_embed_scaled(const int* ids, const void* table, int table_dtype, float* out, int n_tokens,
+SSB_API int ssb_embed_scaled(const int* ids, const void* table, int table_dtype, float* out, void* rounded, int n_tokens,
                              int hidden, int vocab, float scale, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (table_dtype == SSB_F32)
-        embed_kernel<float><<<n_tokens, 256, 0, stream>>>(ids, (const float*)table, out, hidden, vocab, scale);
+        embed_kernel<float><<<n_tokens, 256, 0, stream>>>(ids, (const float*)table, out, (float*)rounded, hidden, vocab, scale);
     else if (table_dtype == SSB_BF16)
-        embed_kernel<bf16><<<n_tokens, 256, 0, stream>>>(ids, (const bf16*)table, out, hidden, vocab, scale);
+        embed_kernel<bf16><<<n_tokens, 256, 0, stream>>>(ids, (const bf16*)table, out, (bf16*)rounded, hidden, vocab, scale);
     else
         return SSB_ERR_BAD_DTYPE;
     return ssb_launch_status();
@@ -92,7 +105,7 @@ SSB_API int ssb_embed_norm(const int* ids, const void* table, int table_dtype, c
 
 SSB_API int ssb_embed(const int* ids, const void* table, int table_dtype, float* out, int n_tokens,
                       int hidden, int vocab, cudaStream_t stream) {
-    return ssb_embed_scaled(ids, table, table_dtype, out, n_tokens, hidden, vocab, 1.0f, stream);
+    return ssb_embed_scaled(ids, table, table_dtype, out, nullptr, n_tokens, hidden, vocab, 1.0f, stream);
 }
 
 // ---------------------------------------------------------------------------------------
@@ -511,7 +524,8 @@ SSB_API int ssb_swiglu(const void* gate_up, int ld, void* z, int ldz, int dtype,
 // (w float32, the multiplier itself: a weight stored around zero arrives as 1 + w).  Optionally the branch row is
 // zeroed behind the read, so that the next sublayer's products can add into it again, and optionally the norm
 // that the next sublayer reads is taken of the new stream in the same pass:
-//     next_out[t] = residual[t] / sqrt(mean(residual[t]^2) + next_eps) * next_w.
+//     next_out[t] = residual[t] / sqrt(mean(residual[t]^2) + next_eps) * next_w,
+// or, where the next sublayer reads the stream without a norm (no next_w), the new stream itself in its type.
 // One block per token, the row in shared memory, sums in a fixed order.
 // ---------------------------------------------------------------------------------------
 constexpr int RA_THREADS = 256;
@@ -558,6 +572,10 @@ rms_add_kernel(float* __restrict__ residual, float* __restrict__ branch, const f
         sq2 = fmaf(v, v, sq2);
     }
     if (next_out == nullptr) return;
+    if (next_w == nullptr) {
+        for (int c = tid; c < width; c += RA_THREADS) next_out[t * width + c] = ssb_from_float<T>(ra_row[c]);
+        return;
+    }
     const float inv2 = 1.0f / sqrtf(ra_block_sum(sq2, red) / (float)width + next_eps);
     for (int c = tid; c < width; c += RA_THREADS)
         next_out[t * width + c] = ssb_from_float<T>(ra_row[c] * inv2 * next_w[c]);
@@ -566,8 +584,7 @@ rms_add_kernel(float* __restrict__ residual, float* __restrict__ branch, const f
 SSB_API int ssb_rms_add(float* residual, float* branch, const float* w, float eps, int n_tokens, int width, int clear,
                         const float* next_w, float next_eps, void* next_out, int next_dtype, int pdl, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (width <= 0 || (size_t)width * sizeof(float) > 200 * 1024 || (next_out != nullptr && next_w == nullptr))
-        return SSB_ERR_BAD_SIZE;
+    if (width <= 0 || (size_t)width * sizeof(float) > 200 * 1024) return SSB_ERR_BAD_SIZE;
     const size_t smem = (size_t)width * sizeof(float);
     int rc;
 #define SSB_RA(TYPE)                                                                                                 \
@@ -584,6 +601,61 @@ SSB_API int ssb_rms_add(float* residual, float* branch, const float* w, float ep
     else if (next_dtype == SSB_BF16) SSB_RA(bf16)
     else return SSB_ERR_BAD_DTYPE;
 #undef SSB_RA
+    return rc ? rc : ssb_launch_status();
+}
+
+// ---------------------------------------------------------------------------------------
+// y[t, c] *= sigmoid(g[t, c]): concatenated heads times a gate of their own, element by element
+// ---------------------------------------------------------------------------------------
+template <typename T>
+__global__ void sigmoid_gate_kernel(T* __restrict__ y, int ldy, const T* __restrict__ g, int ldg, int width, size_t total) {
+    ssb_pdl_launch_dependents();
+    ssb_pdl_wait();
+    const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= total) return;
+    const size_t t = idx / width;
+    const int c = (int)(idx % width);
+    T* p = y + t * ldy + c;
+    *p = ssb_from_float<T>(ssb_to_float(*p) / (1.0f + expf(-ssb_to_float(g[t * ldg + c]))));
+}
+
+// float32 rows in another type: a stream read without a norm
+template <typename T>
+__global__ void round_rows_kernel(const float* __restrict__ x, T* __restrict__ out, size_t total) {
+    ssb_pdl_launch_dependents();
+    ssb_pdl_wait();
+    const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx < total) out[idx] = ssb_from_float<T>(x[idx]);
+}
+
+SSB_API int ssb_round_rows(const float* x, void* out, int dtype, long long total, int pdl, cudaStream_t stream) {
+    if (total <= 0) return 0;
+    if (total > (1ll << 38)) return SSB_ERR_BAD_SIZE;
+    const dim3 grid((unsigned)((total + 255) / 256));
+    int rc;
+    if (dtype == SSB_F32)
+        rc = ssb_launch(round_rows_kernel<float>, grid, dim3(256), 0, stream, pdl != 0, x, (float*)out, (size_t)total);
+    else if (dtype == SSB_BF16)
+        rc = ssb_launch(round_rows_kernel<bf16>, grid, dim3(256), 0, stream, pdl != 0, x, (bf16*)out, (size_t)total);
+    else
+        return SSB_ERR_BAD_DTYPE;
+    return rc ? rc : ssb_launch_status();
+}
+
+SSB_API int ssb_sigmoid_gate(void* y, int ldy, const void* g, int ldg, int dtype, int n_tokens, int width, int pdl,
+                             cudaStream_t stream) {
+    const size_t total = (size_t)n_tokens * width;
+    if (n_tokens <= 0 || width <= 0) return 0;
+    const dim3 grid((unsigned)((total + 255) / 256));
+    int rc;
+    if (dtype == SSB_F32)
+        rc = ssb_launch(sigmoid_gate_kernel<float>, grid, dim3(256), 0, stream, pdl != 0, (float*)y, ldy, (const float*)g, ldg,
+                        width, total);
+    else if (dtype == SSB_BF16)
+        rc = ssb_launch(sigmoid_gate_kernel<bf16>, grid, dim3(256), 0, stream, pdl != 0, (bf16*)y, ldy, (const bf16*)g, ldg,
+                        width, total);
+    else
+        return SSB_ERR_BAD_DTYPE;
     return rc ? rc : ssb_launch_status();
 }
 

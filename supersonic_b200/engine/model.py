@@ -217,7 +217,7 @@ class Model:
         for b in spec.blocks:
             mixer = part(MIXERS, "mixer", b.mixer)
             ff = part(FEED_FORWARDS, "feed-forward", b.feed_forward) if b.feed_forward else None
-            n1 = part(NORMS, "norm", b.mixer_norm)
+            n1 = part(NORMS, "norm", b.mixer_norm) if b.mixer_norm else None
             n2 = part(NORMS, "norm", b.feed_forward_norm) if b.feed_forward_norm else None
             pos = part(POSITION_ENCODINGS, "position encoding", b.position) if b.position else None
             # an arrangement with constants or tensors of its own gets them like any other part

@@ -2,6 +2,7 @@
 the residual stream kept and summed in float32 (crates/runner/src/prefill_engine.rs:1116-1222).
 ``sandwich``: h += norm_b(mixer(norm_a(h))); h += norm_d(feed_forward(norm_c(h))): a sublayer's result passes a
 norm of its own before it joins the stream.
+``post_norm``: h += norm_b(mixer(h)); h += norm_d(feed_forward(h)): the sublayers read the stream as it is.
 ``parallel``: h += mixer(n) + feed_forward(n) with the one n = norm(h), or with a norm each (both of the
 same h); optionally the mixer's input is mixed with the previous token's (token shift), and optionally the
 layer is followed by a learned weighted sum over the results of all layers so far.
@@ -93,6 +94,73 @@ class SandwichBlock:
             x2 = self._give(NormedInput(ctx, residual, self.feed_forward_norm), self.feed_forward)
         self.feed_forward.forward(ctx, x2, branch)
         ctx.kernels.rms_add(residual, branch, self.feed_forward_out, self.eps, clear=True)
+
+
+@register_block("post_norm")
+class PostNormBlock:
+    """x <- x + norm_1(mixer(x)), then x <- x + norm_2(feed_forward(x)): RMS norms behind the sublayers alone, which read
+    the stream itself (the feed-forward may be absent).
+
+    ``params``: ``size``, ``eps``, ``takes_rounded``, ``leaves_rounded``; tensors ``mixer_out`` and ``feed_forward_out``
+    [size].  The stream is float32.  Where the activations are too, the sublayers read it in place; else they read a
+    rounded copy, which the kernel that adds a normed result to the stream writes in the same pass.  ``takes_rounded``: the
+    stop before this one (a block of this kind with ``leaves_rounded``, or an embedding with it) left the copy of the
+    stream in ``ctx.carried``; without it the block rounds the stream itself.  As in a sandwich, the sublayers' products
+    add into a float32 row of zeros per token, which the norm zeroes again behind its read; a feed-forward that ends in a
+    weighted sum over its choices (``terms``) hands the norm the choices instead, and its result is never stored."""
+
+    ENTRY = "rounded_stream"
+
+    def __init__(self, mixer, feed_forward, mixer_norm, feed_forward_norm, position, params=None, weights=None, build=None):
+        if mixer_norm is not None or feed_forward_norm is not None:
+            raise ValueError("post_norm: the sublayers read the stream itself, without a norm in front of them")
+        self.mixer, self.feed_forward, self.position = mixer, feed_forward, position
+        self.size, self.eps = int(params["size"]), float(params["eps"])
+        self.takes, self.leaves = bool(params.get("takes_rounded")), bool(params.get("leaves_rounded"))
+
+        def multiplier(role):
+            w = build.weights.stored(weights[role]).float().contiguous()
+            if tuple(w.shape) != (self.size,):
+                raise ValueError(f"{weights[role]} has shape {tuple(w.shape)}, expected ({self.size},)")
+            return w
+        self.mixer_out = multiplier("mixer_out")
+        self.feed_forward_out = multiplier("feed_forward_out") if feed_forward is not None else None
+        self.dtype = build.dtype
+
+    def forward(self, ctx, residual, cache_id, writes_cache):
+        k = ctx.kernels
+        branch = ctx.streams
+        if not (isinstance(branch, torch.Tensor) and branch.shape == residual.shape and branch.dtype == torch.float32):
+            branch = ctx.streams = torch.zeros_like(residual)         # zero again behind every use
+        rounds = self.dtype != residual.dtype
+
+        def copy(wanted):
+            return torch.empty(residual.shape, dtype=self.dtype, device=residual.device) if rounds and wanted else None
+        x = residual
+        if rounds:
+            x = ctx.carried.pop(self.ENTRY, None) if self.takes else None
+            if self.takes and (x is None or x.shape != residual.shape):
+                raise RuntimeError("post_norm: the stop before this one left no rounded stream")
+            if x is None:
+                x = copy(True)
+                k.round_rows(residual, x)
+        ff = self.feed_forward
+        ctx.stage = "mixer"
+        self.mixer.forward(ctx, x, branch, cache_id, writes_cache, self.position)
+        nxt = copy(ff is not None or self.leaves)
+        k.rms_add(residual, branch, self.mixer_out, self.eps, clear=True, next_out=nxt)
+        if ff is not None:
+            x = residual if nxt is None else nxt
+            ctx.stage = "feed_forward"
+            nxt = copy(self.leaves)
+            if getattr(ff, "sums_choices", False):
+                y, pair_weight, top = ff.terms(ctx, x)
+                k.combine_rms_add(residual, y, pair_weight, top, self.feed_forward_out, self.eps, next_out=nxt)
+            else:
+                ff.forward(ctx, x, branch)
+                k.rms_add(residual, branch, self.feed_forward_out, self.eps, clear=True, next_out=nxt)
+        if self.leaves and rounds:
+            ctx.carried[self.ENTRY] = nxt
 
 
 @register_block("parallel")

@@ -13,7 +13,8 @@ from .registry import BuildContext, register_embedding
 class Embedding:
     """params: ``vocab_size``, ``hidden_size``, ``scale`` (optional: the rows are multiplied by it in float32),
     ``norm`` (optional, ``{"eps", "unit_offset"}``: the rows pass an RMS norm on their way into the stream, in the
-    same kernel); weights: ``weight`` [vocab, hidden], with a norm ``norm`` [hidden]."""
+    same kernel), ``leaves_rounded`` (the rows in the activation type go to ``ctx.carried["rounded_stream"]`` as well, for a
+    first block that reads the stream without a norm); weights: ``weight`` [vocab, hidden], with a norm ``norm`` [hidden]."""
 
     def __init__(self, params, weights, build: BuildContext):
         self.vocab, self.hidden = int(params["vocab_size"]), int(params["hidden_size"])
@@ -25,6 +26,9 @@ class Embedding:
                 raise ValueError(f"{weights['norm']} has shape {tuple(w.shape)}, expected ({self.hidden},)")
             self.norm_weight = (w + (1.0 if params["norm"].get("unit_offset") else 0.0)).contiguous()
             self.norm_eps = float(params["norm"]["eps"])
+        self.leaves_rounded = bool(params.get("leaves_rounded"))
+        if self.leaves_rounded and self.norm_weight is not None:
+            raise ValueError("embedding: rows that pass a norm are not left rounded")
         self.table = build.weights.as_dtype(weights["weight"], build.dtype, share=True)
         if tuple(self.table.shape) != (self.vocab, self.hidden):
             raise ValueError(f"{weights['weight']} has shape {tuple(self.table.shape)}, "
@@ -34,6 +38,10 @@ class Embedding:
         out = torch.empty((token_ids.shape[0], self.hidden), dtype=torch.float32, device=token_ids.device)
         if self.norm_weight is not None:
             ctx.kernels.embed_norm(token_ids, self.table, self.norm_weight, self.norm_eps, out, self.scale)
+        elif self.leaves_rounded and self.table.dtype != out.dtype:
+            rounded = torch.empty(out.shape, dtype=self.table.dtype, device=out.device)
+            ctx.kernels.embed(token_ids, self.table, out, self.scale, rounded)
+            ctx.carried["rounded_stream"] = rounded
         else:
             ctx.kernels.embed(token_ids, self.table, out, self.scale)
         return out

@@ -2,7 +2,8 @@
 token out of ``n_experts``, plus E_shared(x) if the layer has a shared expert.
 
 An expert is a gated unit without biases, E(x) = Wdown (silu(Wgate x) * (Wup x)), or with ``activation`` another
-inner step (see the ``swiglu`` feed-forward).  Routers are registered by name and fill two arrays per step, the
+inner step (see the ``swiglu`` feed-forward); with ``gated`` False it has no gate, E(x) = Wdown act(Wup x) with a named
+activation (see the ``dense`` feed-forward).  Routers are registered by name and fill two arrays per step, the
 chosen experts and their weights:
 
 * ``table``: nothing is learned and nothing is computed from x: row ``token id`` of an integer table
@@ -10,8 +11,9 @@ chosen experts and their weights:
 * ``sigmoid_groups``: scores s = sigmoid(W x) in float32; experts are chosen by s + correction (a stored vector),
   but only among the experts of the ``keep`` best of ``groups`` equal groups of neighbours, a group's score being
   the sum of its two largest choice scores; the weights are the chosen experts' s times ``scale``, not renormalized.
-* ``softmax``: scores s = softmax(W x) over all experts in float32; the experts with the largest scores are chosen;
-  the weights are their s times ``scale``, with ``renormalize`` divided by their sum (+ 1e-20).
+* ``softmax``: scores s = softmax(W x + b) over all experts in float32 (the bias b is optional); the experts with the largest scores are chosen;
+  the weights are their s times ``scale``, with ``renormalize`` divided by their sum (+ 1e-20), which is the softmax over
+  the chosen experts' logits alone.
 
 A shared expert runs for every token; with ``shared.gate`` its result is multiplied by sigmoid(w_sg . x), one number
 per token.
@@ -112,9 +114,9 @@ class SigmoidGroupRouter:
 
 @register_router("softmax")
 class SoftmaxRouter:
-    """params: ``renormalize`` (True), ``scale`` (1.0); weights: ``weight`` [experts, hidden].  The logits are a product of
-    their own with a float32 result (in the bfloat16 path: bfloat16 operands, whose products are exact in float32,
-    summed in float32)."""
+    """params: ``renormalize`` (True), ``scale`` (1.0); weights: ``weight`` [experts, hidden], ``bias`` [experts] (optional).
+    The logits are a product of their own with a float32 result (in the bfloat16 path: bfloat16 operands, whose products
+    are exact in float32, summed in float32)."""
 
     def __init__(self, params, weights, build: BuildContext, n_experts: int, top: int):
         self.n_experts, self.top = n_experts, top
@@ -128,16 +130,22 @@ class SoftmaxRouter:
         if pad:
             w = torch.cat([w, torch.zeros((pad, w.shape[1]), dtype=w.dtype, device=w.device)], dim=0)
         self.weight = w.contiguous()
+        self.bias = None
+        if weights.get("bias"):
+            self.bias = build.weights.stored(weights["bias"]).float().contiguous()
+            if tuple(self.bias.shape) != (n_experts,):
+                raise ValueError(f"{weights['bias']} has shape {tuple(self.bias.shape)}, expected ({n_experts},)")
 
     def route(self, ctx, x, expert_of, pair_weight):
-        ctx.kernels.route_softmax(x, self.weight, self.n_experts, self.renormalize, self.scale, expert_of, pair_weight)
+        ctx.kernels.route_softmax(x, self.weight, self.n_experts, self.renormalize, self.scale, expert_of, pair_weight,
+                                  bias=self.bias)
 
 
 @register_feed_forward("experts")
 class Experts:
     """params: ``hidden_size``, ``n_experts``, ``top``, ``expert_size``, ``activation`` (None, or as the ``swiglu``
-    feed-forward's), ``router`` ({"kind": ..., its own parameters}), ``shared`` (None or {"intermediate_size": ...,
-    "activation": ..., "gate": bool}); weights: ``gate.<e>``, ``up.<e>``, ``down.<e>`` for every expert e, the router's
+    feed-forward's; the name of one with ``gated`` False), ``gated`` (True), ``router`` ({"kind": ..., its own parameters}), ``shared`` (None or {"intermediate_size": ...,
+    "activation": ..., "gate": bool}); weights: ``gate.<e>`` (gated), ``up.<e>``, ``down.<e>`` for every expert e, the router's
     own, and ``shared.gate`` / ``shared.up`` / ``shared.down`` (with a gate ``shared.sg`` [1, hidden])."""
 
     takes_lazy_input = True
@@ -146,23 +154,31 @@ class Experts:
         self.hidden, self.E = int(params["hidden_size"]), int(params["n_experts"])
         self.top, self.inter = int(params["top"]), int(params["expert_size"])
         w, dt = build.weights, build.dtype
+        self.gated = bool(params.get("gated", True))
         first, second = [], []
         for e in range(self.E):
-            gate, up, down = (w.as_dtype(weights[f"{r}.{e}"], dt) for r in ("gate", "up", "down"))
-            for name, t, want in ((f"gate.{e}", gate, (self.inter, self.hidden)), (f"up.{e}", up, (self.inter, self.hidden)),
-                                  (f"down.{e}", down, (self.hidden, self.inter))):
+            rows = []
+            for r in ("gate", "up", "down") if self.gated else ("up", "down"):
+                t, want = w.as_dtype(weights[f"{r}.{e}"], dt), (self.hidden, self.inter) if r == "down" else (self.inter, self.hidden)
                 if tuple(t.shape) != want:
-                    raise ValueError(f"{weights[name]} has shape {tuple(t.shape)}, expected {want}")
-            first.append(torch.cat([gate, up], dim=0))
-            second.append(down)
-        self.w_gate_up = torch.stack(first).contiguous()       # [E, 2 * inter, hidden]: gate rows, then up rows
+                    raise ValueError(f"{weights[f'{r}.{e}']} has shape {tuple(t.shape)}, expected {want}")
+                rows.append(t)
+            first.append(torch.cat(rows[:-1], dim=0))
+            second.append(rows[-1])
+        self.w_first = torch.stack(first).contiguous()         # [E, 2 * inter, hidden]: gate rows, then up rows; up rows alone
         self.w_down = torch.stack(second).contiguous()         # [E, hidden, inter]
         router = dict(params["router"])
         if router.get("kind") not in ROUTERS:
             raise KeyError(f"unknown router {router.get('kind')!r}; registered: {sorted(ROUTERS)}")
         self.router = ROUTERS[router["kind"]](router, weights, build, self.E, self.top)
         from .feed_forward import SwiGLU, gated_activation_of
-        self.act = gated_activation_of(params.get("activation"))
+        if self.gated:
+            self.act = gated_activation_of(params.get("activation"))
+        else:
+            from ..csrc.ops import ACTIVATIONS
+            self.act = str(params.get("activation"))
+            if self.act not in ACTIVATIONS:
+                raise ValueError(f"experts: activation {self.act!r} is not known (known: {sorted(ACTIVATIONS)})")
         self.shared, self.shared_gate = None, False
         if params.get("shared"):
             sh = params["shared"]
@@ -182,14 +198,32 @@ class Experts:
 
     @staticmethod
     def activation_elements(params) -> int:
-        """Elements per token while the part runs: per choice gate, up, their product and the expert's output
-        (float32: counted twice); the shared expert's rows."""
+        """Elements per token while the part runs: per choice gate, up, their product (without a gate the inner row alone)
+        and the expert's output (float32: counted twice); the shared expert's rows."""
+        inner = 3 if params.get("gated", True) else 1
         shared = 3 * int(params["shared"]["intermediate_size"]) if params.get("shared") else 0
-        return int(params["top"]) * (3 * int(params["expert_size"]) + 2 * int(params["hidden_size"])) + shared
+        return int(params["top"]) * (inner * int(params["expert_size"]) + 2 * int(params["hidden_size"])) + shared
+
+    @property
+    def sums_choices(self) -> bool:
+        """Whether the result is the weighted sum over the choices alone: a block may then take ``terms`` and sum itself."""
+        return self.shared is None
+
+    def terms(self, ctx, x):
+        """(y [tokens x top, hidden] float32, the choices' weights [tokens, top], top)."""
+        return self._choices(ctx, as_tensor(x))[:2] + (self.top,)
 
     def forward(self, ctx, x, residual):
-        T, dev, top = residual.shape[0], residual.device, self.top
-        xt = as_tensor(x)
+        y, pair_weight, shared_scale = self._choices(ctx, as_tensor(x))
+        ctx.kernels.expert_combine(residual, y, pair_weight, self.top)
+        if self.shared is not None:
+            if shared_scale is None:
+                self.shared.forward(ctx, x, residual)
+            else:
+                self.shared.forward(ctx, x, residual, row_scale=shared_scale)
+
+    def _choices(self, ctx, xt):
+        T, dev, top = xt.shape[0], xt.device, self.top
         P = T * top
         expert_of = torch.empty((T, top), dtype=torch.int32, device=dev)
         pair_weight = torch.empty((T, top), dtype=torch.float32, device=dev)
@@ -208,15 +242,12 @@ class Experts:
                   "tile_row0": ints[self.E + 1 + P + max_tiles: self.E + 1 + P + 2 * max_tiles], "meta": ints[-1:]}
         ctx.kernels.group_by_expert(expert_of, self.E, groups)
         z = torch.empty((P, self.inter), dtype=self.dtype, device=dev)
-        if self.act is None:
-            ctx.kernels.expert_gate_up(xt, top, self.w_gate_up, z, groups)
+        if not self.gated:
+            ctx.kernels.expert_up(xt, top, self.w_first, z, groups, self.act)
+        elif self.act is None:
+            ctx.kernels.expert_gate_up(xt, top, self.w_first, z, groups)
         else:
-            ctx.kernels.expert_gate_up(xt, top, self.w_gate_up, z, groups, act=self.act)
+            ctx.kernels.expert_gate_up(xt, top, self.w_first, z, groups, act=self.act)
         y = torch.empty((P, self.hidden), dtype=torch.float32, device=dev)
         ctx.kernels.grouped_linear(z, False, top, self.w_down, y, True, groups)
-        ctx.kernels.expert_combine(residual, y, pair_weight, top)
-        if self.shared is not None:
-            if shared_scale is None:
-                self.shared.forward(ctx, x, residual)
-            else:
-                self.shared.forward(ctx, x, residual, row_scale=shared_scale)
+        return y, pair_weight, shared_scale

@@ -15,7 +15,7 @@ Visible to position p, with window W, F kept first tokens and runs of P tokens:
     its key is the mean of the run's P keys as the cache holds them, its value the mean of their values.
 
 A token that has left the window while its run is not yet wholly before it is not visible.  ``norm`` is an RMS norm
-of q and of k with a plain weight: per head over ``dim`` with one weight vector for all heads (``"head"``), or over
+of q and of k with a plain weight (none stored: all ones): per head over ``dim`` with one weight vector for all heads (``"head"``), or over
 the whole projection of all heads at once with a weight of that size (``"row"``).  ``rot`` turns the first
 coordinates of q and k (the position encoding of the block); ``vrot`` turns every value over its whole width by
 its own position, so that a value enters a head's sum by its distance to the query.  ``sink`` (True): a key of score 0
@@ -71,7 +71,7 @@ class WindowAttention:
     ``out_scale`` (1.0), ``conv`` (0), ``values`` (``"projection"`` or ``"keys"``), ``query_temperature`` (None),
     ``head_gate`` (False), ``element_gate`` (False), ``score_maps`` (1 or 2), ``map_offset``, ``own_kv`` (True),
     ``cache_window``, ``conv_values`` (False), ``head_scale`` (False), ``distance_bias`` (None), ``value_mix`` (None); weights:
-    ``q``, ``k``, ``v``, ``o``, with a norm ``q_norm``, ``k_norm``, with a convolution ``q_conv``, ``k_conv`` (and ``v_conv``)
+    ``q``, ``k``, ``v``, ``o``, with a norm ``q_norm``, ``k_norm`` (both may be absent), with a convolution ``q_conv``, ``k_conv`` (and ``v_conv``)
     [channels, taps], with a gate ``g`` [heads, hidden] or [heads x value_dim, hidden], with two maps ``lq1``, ``lk1``,
     ``lq2``, ``lk2`` [dim], with learned sinks ``sink`` [heads], with a head scale ``temp`` [heads], mixing values of an
     earlier layer ``vmix`` (one number)."""
@@ -165,17 +165,21 @@ class WindowAttention:
         self._q_rows, self._gate_rows = q, gate_rows
         self.q_norm = self.k_norm = None
         if self.qk_norm:
-            self.q_norm = w.stored(weights["q_norm"]).float().contiguous()
+            def multiplier(role, n):
+                if weights.get(role) is None:            # a norm without a weight
+                    return torch.ones(n, dtype=torch.float32, device=build.device)
+                return w.stored(weights[role]).float().contiguous()
+            self.q_norm = multiplier("q_norm", D if self.qk_norm == "head" else H * D)
             sizes = [D if self.qk_norm == "head" else H * D]
             norms = [self.q_norm]
             if self.own_kv:
-                self.k_norm = w.stored(weights["k_norm"]).float().contiguous()
+                self.k_norm = multiplier("k_norm", D if self.qk_norm == "head" else G * D)
                 sizes.append(D if self.qk_norm == "head" else G * D)
                 norms.append(self.k_norm)
             else:
                 self.k_norm = self.q_norm    # never applied: the stop does not write keys
             if [n.numel() for n in norms] != sizes or any(n.dim() != 1 for n in norms):
-                raise ValueError(f"{weights['q_norm']} / {weights.get('k_norm')}: expected {sizes} weights")
+                raise ValueError(f"{weights.get('q_norm')} / {weights.get('k_norm')}: expected {sizes} weights")
         self.conv_w = None
         if self.taps:
             cq, ck = (w.stored(weights[r]).float() for r in ("q_conv", "k_conv"))
