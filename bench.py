@@ -425,6 +425,40 @@ def _ruzunex_sizes(name):
     return ruz, kil
 
 
+def _ropulix_sizes(name):
+    """(Ropulix config.json, the Sotavik configuration of the same width, layer count, vocabulary and weights per expert: the
+    closest existing design, whose latent attention and expert products run on the same kernels; its shared expert, which
+    this design does not have, left out).  A gated recurrence, a latent layer inside a window, a window attention layer and
+    a latent layer that reads the first one's rows with a longer window, all with experts."""
+    def latent(heads, dim, rot, vdim, rank, q_rank, window, kv_from=None):
+        m = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "q_rank": q_rank, "mask": {"size": window},
+             "rot": {"base": 10000.0, "dims": rot}, "scale": (dim + rot) ** -0.5}
+        if kv_from is not None:
+            m["kv_from"] = kv_from
+        return {"type": "latent_attention", "mixer": m}
+
+    def window(heads, kv, dim, vdim, size):
+        return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": dim ** -0.5,
+                                               "mask": {"size": size}}}
+
+    def rglru(width, blocks):
+        return {"type": "rglru", "mixer": {"width": width, "conv": 4, "blocks": blocks}}
+    sot, _ = _sotavik_sizes(name)
+    theirs = sot["layers"][0]["mlp"]
+    sot = dict(sot, layers=[dict(l, mlp=dict(l["mlp"], shared=None)) for l in sot["layers"]])
+    if name == "2048":
+        mixers = [rglru(2048, 16), latent(16, 128, 64, 128, 512, 768, 512), window(16, 4, 64, 128, 512),
+                  latent(16, 128, 64, 128, 512, 768, 1024, kv_from=1)]
+    else:
+        mixers = [rglru(1024, 8), latent(8, 64, 32, 64, 256, 384, 256), window(8, 2, 64, 128, 256),
+                  latent(8, 64, 32, 64, 256, 384, 512, kv_from=1)]
+    # two matrices an expert instead of three: half as wide again for the same weights
+    experts = {"kind": "moe", "expert": {"ff": theirs["expert"]["ff"] * 3 // 2}, "router": dict(theirs["router"])}
+    rop = {"architecture": "Ropulix", "vocab": sot["vocab"], "width": sot["width"], "norm": {"eps": 1e-5},
+           "layers": [dict(m, mlp=experts) for m in mixers]}
+    return rop, sot
+
+
 def _operation_work(model, tokens):
     """Algorithmic work of one prompt of ``tokens`` tokens per operation of the model's parts: (FLOPs, bytes).
     Matrix products count 2 per multiply-add; attention counts its scores and weighted sums over the causal
@@ -456,9 +490,15 @@ def _operation_work(model, tokens):
         m, ff = b.mixer, b.feed_forward
         kind = type(m).__name__
         if kind == "LatentAttention":
-            add("mixer.linear", 2 * T * (m.w_in.numel() + m.w_o.numel()))
+            w_in = m.w_in if m.own_kv else m._read_weight()
+            add("mixer.linear", 2 * T * (w_in.numel() + m.w_o.numel() + (m.w_uq.numel() if m.q_rank else 0)))
             add("mixer.head_linear", 2 * T * (m.w_absorb.numel() + m.w_uv.numel()))
-            add("mixer.latent_attention", 2 * causal * m.H * (2 * m.rank + m.rot))
+            w = int(m.window or T)
+            pairs = sum(min(i + 1, w) for i in range(T))
+            add("mixer.latent_attention", 2 * pairs * m.H * (2 * m.rank + m.rot))
+            if m.q_rank:    # the query latent in and out, the low-rank row in and its cache row out, the rotated query parts in and out
+                row = 4 * (m.rank + m.rot) if m.own_kv else 0
+                add("mixer.latent_prepare", 0, T * (4 * m.q_rank + row + 4 * m.H * m.rot))
         elif kind == "GatedLinearAttention":
             add("mixer.linear", 2 * T * (m.w_in.numel() + m.w_a2.numel() + m.w_o.numel()))
             add("mixer.gated_linear_scan", 4 * T * m.H * m.dim * m.vdim,
@@ -507,6 +547,13 @@ def _operation_work(model, tokens):
             # behind each sublayer: the float32 branch in, zeros back, the stream in and out; once with the next norm's rows out
             W = model.spec.hidden_size
             add("feed_forward.rms_add", 0, T * W * ((4 * 4 + 2) + (4 * 4 if ff is not None else 0)))
+        if type(b).__name__ == "PostNormBlock":
+            # behind the mixer: the float32 branch in, zeros back, the stream in and out, its rounded copy out; behind the
+            # experts: the choices' float32 rows in instead of the branch
+            W = model.spec.hidden_size
+            add("mixer.rms_add", 0, T * W * (4 * 4 + 2))
+            if ff is not None:
+                add("feed_forward.combine_rms_add", 0, T * W * (4 * (ff.top + 2) + (2 if b.leaves else 0)))
         if type(b).__name__ == "HyperConnectionBlock":
             # a sublayer's entry: the streams and the branch in, the streams and zeros out, the normed and convolved row out
             W, S = model.spec.hidden_size, b.streams
@@ -515,7 +562,7 @@ def _operation_work(model, tokens):
                 add("feed_forward.stream_enter", 0, T * W * (4 * (2 * S + 2) + 2))
         if fk == "Experts":
             per = ff.w_first[0].numel() + ff.w_down[0].numel()
-            add("feed_forward.expert_gate_up", 2 * T * ff.top * ff.w_first[0].numel())
+            add("feed_forward.expert_gate_up" if ff.gated else "feed_forward.expert_up", 2 * T * ff.top * ff.w_first[0].numel())
             add("feed_forward.grouped_linear", 2 * T * ff.top * ff.w_down[0].numel())
             if getattr(getattr(ff.router, "weight", None), "dim", lambda: 0)() == 2:   # a router that reads the token: a product of its own
                 inside = type(ff.router).__name__ == "SoftmaxRouter"                  # ... taken with the choice as one operation
@@ -542,12 +589,14 @@ def design_comparison(args):
     from supersonic_b200.weights import RandomWeightStore
     pk, pk_src = peaks()
     sizes = {"vufadra": _vufadra_sizes, "sotavik": _sotavik_sizes, "ronelorn": _ronelorn_sizes,
-             "kilisun": _kilisun_sizes, "ruzunex": _ruzunex_sizes}[args.design]
+             "kilisun": _kilisun_sizes, "ruzunex": _ruzunex_sizes, "ropulix": _ropulix_sizes}[args.design]
     sot, lla = sizes(args.design_size)
-    beside = {"ronelorn": "vufadra", "kilisun": "ronelorn", "ruzunex": "kilisun"}.get(args.design, "llama")
+    beside = {"ronelorn": "vufadra", "kilisun": "ronelorn", "ruzunex": "kilisun", "ropulix": "sotavik"}.get(args.design, "llama")
     models = [(args.design, sot), (beside, lla)]
     if args.design in ("kilisun", "ruzunex"):                              # its experts beside the design whose expert products they run on
         models.append(("sotavik", _sotavik_sizes(args.design_size)[0]))
+    if args.design == "ropulix":                                           # the likes of its window attention and of its recurrence
+        models += [("kilisun", _kilisun_sizes(args.design_size)[0]), ("vufadra", _vufadra_sizes(args.design_size)[0])]
     out = {"metric": "design_comparison", "design": args.design, "beside": beside, "size": args.design_size,
            "layers": len(sot["layers"]), "dtype": "bf16", "data": "synthetic", "peaks": pk, "peaks_source": pk_src,
            "models": {}}
@@ -721,7 +770,7 @@ def main():
                     help="also time decode and prompts at further sizes (adds a 'sweep' key to the line)")
     ap.add_argument("--deterministic", action="store_true",
                     help="time the bfloat16 path without float atomics and with one kernel choice whatever the batch")
-    ap.add_argument("--design", default=None, choices=["sotavik", "vufadra", "ronelorn", "kilisun", "ruzunex"],
+    ap.add_argument("--design", default=None, choices=["sotavik", "vufadra", "ronelorn", "kilisun", "ruzunex", "ropulix"],
                     help="instead of the headline workload: this design beside the closest existing model at equal size")
     ap.add_argument("--design-size", default="2048", help="width of the compared models: 1024 or 2048")
     args = ap.parse_args()

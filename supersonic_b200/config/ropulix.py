@@ -276,15 +276,15 @@ class RopulixConfig:
         return name.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2")
 
     def special_random_tensor(self, name: str, seed: int, device, std: float) -> Optional[torch.Tensor]:
-        """Random values for what is neither a matrix nor a norm weight: biases of order one half, gate matrices and
-        convolution taps of order one over their fan-in's root, decay rates that keep a state for a few to a few hundred
-        tokens."""
+        """Random values for what is neither a matrix nor a norm weight: biases of the matrices' spread (so that they do not
+        drown what the matrices say of a token), gate matrices and convolution taps of order one over their fan-in's root,
+        decay rates that keep a state for a few to a few hundred tokens."""
         from ..weights.random_fill import fnv1a64
         shape = self.tensor_shapes()[name]
         g = torch.Generator().manual_seed((seed * 0x9E3779B1 + fnv1a64(name)) % (1 << 62))
         last = name.rsplit(".", 1)[-1]
         if last == "b":
-            t = 0.5 * torch.randn(shape, generator=g)
+            t = std * torch.randn(shape, generator=g)
         elif last == "lam":
             t = -1.0 - 5.0 * torch.rand(shape, generator=g)
         elif last in ("conv", "ra", "ri"):

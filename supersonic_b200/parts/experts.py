@@ -141,6 +141,17 @@ class SoftmaxRouter:
                                   bias=self.bias)
 
 
+def group_buffers(kernels, n_pairs: int, n_experts: int, device) -> dict:
+    """The int32 buffers that sorting ``n_pairs`` (token, choice) pairs by expert fills and the grouped products read, with
+    the sizes a kernel set asks for."""
+    tile_rows, P, E = kernels.expert_tile_rows, n_pairs, n_experts
+    max_tiles = P // tile_rows + min(E, P)
+    ints = torch.empty(E + 1 + P + 2 * max_tiles + 1, dtype=torch.int32, device=device)
+    return {"tile_rows": tile_rows, "max_tiles": max_tiles, "offsets": ints[: E + 1], "order": ints[E + 1: E + 1 + P],
+            "tile_expert": ints[E + 1 + P: E + 1 + P + max_tiles],
+            "tile_row0": ints[E + 1 + P + max_tiles: E + 1 + P + 2 * max_tiles], "meta": ints[-1:]}
+
+
 @register_feed_forward("experts")
 class Experts:
     """params: ``hidden_size``, ``n_experts``, ``top``, ``expert_size``, ``activation`` (None, or as the ``swiglu``
@@ -233,13 +244,7 @@ class Experts:
             self.router.route(ctx, xt, expert_of, pair_weight, extra_out=shared_scale)
         else:
             self.router.route(ctx, xt, expert_of, pair_weight)
-        tile_rows = ctx.kernels.expert_tile_rows
-        max_tiles = P // tile_rows + min(self.E, P)
-        ints = torch.empty(self.E + 1 + P + 2 * max_tiles + 1, dtype=torch.int32, device=dev)
-        groups = {"tile_rows": tile_rows, "max_tiles": max_tiles, "offsets": ints[: self.E + 1],
-                  "order": ints[self.E + 1: self.E + 1 + P],
-                  "tile_expert": ints[self.E + 1 + P: self.E + 1 + P + max_tiles],
-                  "tile_row0": ints[self.E + 1 + P + max_tiles: self.E + 1 + P + 2 * max_tiles], "meta": ints[-1:]}
+        groups = group_buffers(ctx.kernels, P, self.E, dev)
         ctx.kernels.group_by_expert(expert_of, self.E, groups)
         z = torch.empty((P, self.inter), dtype=self.dtype, device=dev)
         if not self.gated:

@@ -93,7 +93,8 @@ class LatentAttention:
             self.norm_w = torch.ones(rank, dtype=dt, device=build.device)
         # Wuk_g^T [rank, dim] per head carries a plain query into the latent space; Wuv_g [vdim, rank] carries
         # the summed latent out of it
-        self.w_absorb = got["uk"].view(H, d, rank).transpose(1, 2).contiguous()
+        self.w_absorb = torch.empty((H, rank, d), dtype=dt, device=got["uk"].device)      # (a copy whose strides hold for d = 1 too)
+        self.w_absorb.copy_(got["uk"].view(H, d, rank).transpose(1, 2))
         self.w_uv = got["uv"].view(H, dv, rank).contiguous()
         self.w_o = got["o"]
         self.sinks = None
