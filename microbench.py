@@ -189,21 +189,32 @@ def latent_attention(args):
 
 def grouped_gemm(args):
     """The experts' gate/up product with SwiGLU (--kernel swiglu) or a plain one: --tokens tokens, --top of
-    --experts experts each, matrices of --n x --k."""
+    --experts experts each, matrices of --n x --k.  --kernel tc / tc_swiglu: on tcgen05, tiles of --tile rows, the rows
+    sorted beforehand."""
     T, top, E, K, N = args.tokens, args.top, args.experts, args.k, args.n
     expert_of = torch.rand(T, E, device=DEV).argsort(1)[:, :top].int().contiguous()
     P = T * top
-    mt = ops.expert_tiles_bound(P, E, 64)
+    tc = args.kernel.startswith("tc")
+    tile = args.tile if tc else 64
+    mt = ops.expert_tiles_bound(P, E, tile)
     offsets, order, te, tr, meta = [torch.zeros(n, dtype=torch.int32, device=DEV) for n in (E + 1, P, mt, mt, 1)]
-    ops.group_by_expert(expert_of, E, 64, offsets, order, te, tr, meta)
-    swiglu = args.kernel == "swiglu"
+    ops.group_by_expert(expert_of, E, tile, offsets, order, te, tr, meta)
+    swiglu = args.kernel.endswith("swiglu")
     x = torch.randn(T, K, device=DEV).bfloat16()
     w = (torch.randn(E, (2 if swiglu else 1) * N, K, device=DEV) * 0.05).bfloat16()
     out = torch.empty(P, N, dtype=torch.bfloat16, device=DEV)
-    us = _time(lambda i: ops.grouped_gemm_mma(x, order, top, w, out, None, offsets, te, tr, meta, mt,
-                                              ops.GG_SWIGLU if swiglu else ops.GG_STORE), args.iters)
+    if tc:
+        groups = {"offsets": offsets, "order": order, "tile_expert": te, "tile_row0": tr, "meta": meta, "max_tiles": mt, "tile_rows": tile}
+        rows = torch.empty(P, K, dtype=torch.bfloat16, device=DEV)
+        sort_us = _time(lambda i: ops.group_gather(expert_of, E, tile, offsets, order, te, tr, meta, x, rows), args.iters)
+        us = _time(lambda i: ops.grouped_gemm_tc(rows, w, out, None, groups, ops.GG_SWIGLU if swiglu else ops.GG_STORE), args.iters)
+        ops.check_device_errors()
+    else:
+        sort_us = _time(lambda i: ops.group_by_expert(expert_of, E, tile, offsets, order, te, tr, meta), args.iters)
+        us = _time(lambda i: ops.grouped_gemm_mma(x, order, top, w, out, None, offsets, te, tr, meta, mt,
+                                                  ops.GG_SWIGLU if swiglu else ops.GG_STORE), args.iters)
     used = E * (1.0 - (1.0 - top / E) ** T)
-    return {"kernel": "grouped_gemm_mma", "swiglu": swiglu, "tokens": T, "top": top, "experts": E, "n": N, "k": K,
+    return {"kernel": "grouped_gemm_tc" if tc else "grouped_gemm_mma", "tile": tile, "sort_us": round(sort_us, 2), "swiglu": swiglu, "tokens": T, "top": top, "experts": E, "n": N, "k": K,
             "us": round(us, 2), "TFLOP/s": round(2.0 * P * w.shape[1] * K / us / 1e6, 1),
             "GB/s": round(used * w.shape[1] * K * 2 / us / 1e3, 1)}
 

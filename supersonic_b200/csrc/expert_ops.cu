@@ -273,6 +273,100 @@ SSB_API int ssb_group_by_expert(const int* expert_of, int n_pairs, int n_experts
 }
 
 // ---------------------------------------------------------------------------------------
+// The same grouping over many blocks, with the rows of x copied into sorted order on the way (what the products that fetch
+// whole boxes of rows read).  A block owns a run of neighbouring pairs.  It counts all pairs per expert and those before
+// its own; an expert's first row is the sum of the counts of the experts before it, and a pair's place behind it is the
+// number of pairs of its expert that come earlier: the order is stable, whatever the number of blocks.  Block 0 writes
+// the offsets and the tile list.
+// ---------------------------------------------------------------------------------------
+constexpr int GR_THREADS = 256;
+
+__global__ void __launch_bounds__(GR_THREADS)
+group_gather_kernel(const int* __restrict__ expert_of, int n_pairs, int n_experts, int tile_rows, int chunk,
+                    const uint4* __restrict__ x, int ldx, int top, int width, uint4* __restrict__ rows,
+                    int* __restrict__ offsets, int* __restrict__ order, int* __restrict__ tile_expert,
+                    int* __restrict__ tile_row0, int* __restrict__ meta) {
+    extern __shared__ int gr_s[];                        // all [E], before [E], then [chunk] experts, [chunk] places
+    int* all = gr_s;
+    int* before = all + n_experts;
+    int* mine = before + n_experts;
+    int* place = mine + chunk;
+    ssb_pdl_launch_dependents();
+    ssb_pdl_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int lo = blockIdx.x * chunk, n = min(chunk, n_pairs - lo);
+    for (int e = tid; e < 2 * n_experts; e += GR_THREADS) gr_s[e] = 0;
+    __syncthreads();
+    for (int p = tid; p < n_pairs; p += GR_THREADS) {
+        const int e = expert_of[p];
+        atomicAdd(&all[e], 1);
+        if (p < lo) atomicAdd(&before[e], 1);
+        if (p >= lo && p < lo + n) mine[p - lo] = e;
+    }
+    __syncthreads();
+    if (warp == 0) {                                     // first rows (and tiles) of the experts, 32 at a time
+        int row = 0, tile = 0;
+        for (int e0 = 0; e0 < n_experts; e0 += 32) {
+            const int e = e0 + lane, cnt = e < n_experts ? all[e] : 0, tiles = (cnt + tile_rows - 1) / tile_rows;
+            int r = cnt, t = tiles;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int ru = __shfl_up_sync(0xffffffffu, r, o), tu = __shfl_up_sync(0xffffffffu, t, o);
+                if (lane >= o) { r += ru; t += tu; }
+            }
+            const int first = row + r - cnt, tile0 = tile + t - tiles;
+            if (e < n_experts) {
+                before[e] += first;
+                if (blockIdx.x == 0) {
+                    offsets[e] = first;
+                    for (int k = 0; k < tiles; ++k) {
+                        tile_expert[tile0 + k] = e;
+                        tile_row0[tile0 + k] = first + k * tile_rows;
+                    }
+                }
+            }
+            row += __shfl_sync(0xffffffffu, r, 31);
+            tile += __shfl_sync(0xffffffffu, t, 31);
+        }
+        if (blockIdx.x == 0 && lane == 0) {
+            offsets[n_experts] = row;
+            meta[0] = tile;
+        }
+    }
+    __syncthreads();
+    for (int i = tid; i < n; i += GR_THREADS) {
+        const int e = mine[i];
+        int rank = 0;
+        for (int j = 0; j < i; ++j) rank += mine[j] == e ? 1 : 0;
+        const int at = before[e] + rank;
+        place[i] = at;
+        order[at] = lo + i;
+    }
+    if (rows == nullptr) return;
+    __syncthreads();
+    for (int i = warp; i < n; i += GR_THREADS / 32) {
+        const uint4* src = x + (size_t)((lo + i) / top) * ldx;
+        uint4* dst = rows + (size_t)place[i] * width;
+#pragma unroll 4
+        for (int c = lane; c < width; c += 32) dst[c] = src[c];
+    }
+}
+
+// x [tokens, ldx] and rows [n_pairs, width] bfloat16 (columns and strides multiples of 8), or both null; chunk: pairs a block
+SSB_API int ssb_group_gather(const int* expert_of, int n_pairs, int n_experts, int tile_rows, int chunk, const void* x, int ldx,
+                             int top, int width, void* rows, int* offsets, int* order, int* tile_expert, int* tile_row0,
+                             int* meta, int pdl, cudaStream_t stream) {
+    if (n_pairs <= 0) return 0;
+    if (n_experts <= 0 || n_experts > 2048 || tile_rows <= 0 || chunk < 1 || chunk > 4096 || top < 1) return SSB_ERR_BAD_SIZE;
+    if (rows != nullptr && (x == nullptr || width % 8 || ldx % 8 || (((uintptr_t)x | (uintptr_t)rows) & 15))) return SSB_ERR_BAD_SIZE;
+    const size_t smem = (size_t)(2 * n_experts + 2 * chunk) * sizeof(int);
+    const int rc = ssb_launch(group_gather_kernel, dim3((n_pairs + chunk - 1) / chunk), dim3(GR_THREADS), smem, stream, pdl != 0,
+                              expert_of, n_pairs, n_experts, tile_rows, chunk, (const uint4*)x, ldx / 8, top, width / 8,
+                              (uint4*)rows, offsets, order, tile_expert, tile_row0, meta);
+    return rc ? rc : ssb_launch_status();
+}
+
+// ---------------------------------------------------------------------------------------
 // grouped product: for sorted row r of expert e, C[c_row(r), n] = sum_k A[a_row(r), k] W_e[n, k].
 // a_row(r) = a_index ? a_index[r] / a_div : r;  c_row(r) = c_index ? c_index[r] : r.
 // 64 x 64 tiles, the arithmetic of the plain matrix product (FMA sums of 16, added with compensation).

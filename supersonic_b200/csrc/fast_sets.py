@@ -20,6 +20,8 @@ TARGET_BLOCKS = 1184           # eight small blocks per SM
 DETERMINISTIC_CHUNK_PAGES = 16 # ... and its fixed chunk size (1,024 keys) when results must not depend on the batch
 STREAM_ROWS = ops.GEMV_TC_MAX_ROWS   # steps of up to this many rows take the projections that stream the weights once
 CLUSTER_CHUNK_PAGES = 8       # the most pages a chunk holds when a sequence's chunks run as a cluster
+EXPERT_NARROW_ROWS = 24       # mean rows an expert up to which its products take tiles of 64 rows ...
+EXPERT_MIDDLE_ROWS = 64       # ... and of 128
 TC_ATTENTION_MIN_NEW = 96     # prompts at least this long take the tcgen05 attention (tiles of 128 rows)
 
 
@@ -469,12 +471,31 @@ class FastKernels(PlainKernels):
         ops.route_softmax(logits, n_experts, renormalize, scale, expert_of, pair_weight, clear=True, pdl=self._chain(rows),
                           bias=bias)
 
-    def group_by_expert(self, expert_of, n_experts, groups):
+    grouped_tc = True        # the experts' products on tcgen05, where their sizes are whole 16-byte pieces
+
+    def expert_grouping(self, n_tokens, top, n_experts, hidden, inter):
+        if not (self.grouped_tc and ops.grouped_gemm_tc_ok(hidden, inter, n_experts)):
+            return super().expert_grouping(n_tokens, top, n_experts, hidden, inter)
+        # a token picks an expert once: a step of up to 64 tokens has no group of more rows.  Narrow tiles leave room for
+        # more stages of weights in flight, wide ones read the weights less often
+        mean = n_tokens * top / n_experts
+        return (64 if n_tokens <= 64 or mean <= EXPERT_NARROW_ROWS else 128 if mean <= EXPERT_MIDDLE_ROWS else 256), True
+
+    def group_by_expert(self, expert_of, n_experts, groups, x=None):
+        if groups.get("sorts_rows") and x is not None:
+            P = expert_of.numel()
+            groups["rows"] = torch.empty((P, x.shape[1]), dtype=x.dtype, device=x.device)
+            ops.group_gather(expert_of, n_experts, groups["tile_rows"], groups["offsets"], groups["order"], groups["tile_expert"],
+                             groups["tile_row0"], groups["meta"], x, groups["rows"], pdl=self._chain(expert_of.shape[0]))
+            return
         ops.group_by_expert(expert_of, n_experts, groups["tile_rows"], groups["offsets"], groups["order"],
                             groups["tile_expert"], groups["tile_row0"], groups["meta"], pdl=self.pdl)
 
     def grouped_linear(self, a, gather, top, w, out, scatter, groups):
-        if ops.grouped_gemm_mma_ok(a, w, out, ops.GG_STORE):
+        if "rows" in groups:
+            ops.grouped_gemm_tc(groups["rows"] if gather else a, w, out, groups["order"] if scatter else None, groups,
+                                pdl=self._chain(a.shape[0] // (1 if gather else top)))
+        elif ops.grouped_gemm_mma_ok(a, w, out, ops.GG_STORE):
             ops.grouped_gemm_mma(a, groups["order"] if gather else None, top if gather else 1, w, out,
                                  groups["order"] if scatter else None, groups["offsets"], groups["tile_expert"],
                                  groups["tile_row0"], groups["meta"], groups["max_tiles"], ops.GG_STORE, pdl=self.pdl)
@@ -482,7 +503,9 @@ class FastKernels(PlainKernels):
             super().grouped_linear(a, gather, top, w, out, scatter, groups)
 
     def expert_gate_up(self, x, top, w_gate_up, out, groups, act=None):
-        if ops.grouped_gemm_mma_ok(x, w_gate_up, out, ops.GG_SWIGLU):
+        if "rows" in groups:
+            ops.grouped_gemm_tc(groups["rows"], w_gate_up, out, None, groups, ops.GG_SWIGLU, act, pdl=self._chain(x.shape[0]))
+        elif ops.grouped_gemm_mma_ok(x, w_gate_up, out, ops.GG_SWIGLU):
             ops.grouped_gemm_mma(x, groups["order"], top, w_gate_up, out, None, groups["offsets"],
                                  groups["tile_expert"], groups["tile_row0"], groups["meta"], groups["max_tiles"],
                                  ops.GG_SWIGLU, pdl=self.pdl, act=act)
@@ -490,7 +513,9 @@ class FastKernels(PlainKernels):
             super().expert_gate_up(x, top, w_gate_up, out, groups, act)
 
     def expert_up(self, x, top, w_up, out, groups, act):
-        if ops.grouped_gemm_mma_ok(x, w_up, out, ops.GG_ACT):
+        if "rows" in groups:
+            ops.grouped_gemm_tc(groups["rows"], w_up, out, None, groups, ops.GG_ACT, act, pdl=self._chain(x.shape[0]))
+        elif ops.grouped_gemm_mma_ok(x, w_up, out, ops.GG_ACT):
             ops.grouped_gemm_mma(x, groups["order"], top, w_up, out, None, groups["offsets"], groups["tile_expert"],
                                  groups["tile_row0"], groups["meta"], groups["max_tiles"], ops.GG_ACT, pdl=self.pdl, act=act)
         else:

@@ -363,7 +363,9 @@ class PlainKernels:
                         max_new=batch.max_new, scratch=scratch)
 
     # ---- experts ---------------------------------------------------------------------
-    expert_tile_rows = 64
+    def expert_grouping(self, n_tokens, top, n_experts, hidden, inter):
+        """(rows of a tile, whether the grouping copies the tokens' rows into sorted order) for an expert layer's step."""
+        return 64, False
 
     def route_table(self, token_ids, table, n_experts, expert_of, pair_weight):
         ops.route_table(token_ids, table, n_experts, expert_of, pair_weight)
@@ -379,9 +381,9 @@ class PlainKernels:
         self.linear(x, weight, logits)
         ops.route_softmax(logits, n_experts, renormalize, scale, expert_of, pair_weight, pdl=self._chain(logits.shape[0]), bias=bias)
 
-    def group_by_expert(self, expert_of, n_experts, groups):
+    def group_by_expert(self, expert_of, n_experts, groups, x=None):
         """``groups``: the dict of int32 tensors a grouped product reads (offsets, order, tile_expert,
-        tile_row0, meta) plus ``max_tiles``."""
+        tile_row0, meta) plus ``max_tiles``; ``x``: the tokens' rows, which a set may copy into sorted order here."""
         ops.group_by_expert(expert_of, n_experts, groups["tile_rows"], groups["offsets"], groups["order"],
                             groups["tile_expert"], groups["tile_row0"], groups["meta"])
 

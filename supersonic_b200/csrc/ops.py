@@ -1540,6 +1540,69 @@ def group_by_expert(expert_of: torch.Tensor, n_experts: int, tile_rows: int, off
         _ptr(tile_expert), _ptr(tile_row0), _ptr(meta), c_int(1 if pdl else 0), _stream()), "group_by_expert")
 
 
+GROUP_BLOCKS = 592               # four blocks an SM
+
+
+def group_gather(expert_of: torch.Tensor, n_experts: int, tile_rows: int, offsets: torch.Tensor, order: torch.Tensor,
+                 tile_expert: torch.Tensor, tile_row0: torch.Tensor, meta: torch.Tensor, x: Optional[torch.Tensor] = None,
+                 rows: Optional[torch.Tensor] = None, pdl: bool = False) -> None:
+    """``group_by_expert`` over many blocks, in a stable order; with ``rows`` [pairs, width] the pairs' rows of ``x`` [tokens,
+    width] (bfloat16) in sorted order."""
+    for t, n in ((expert_of, "expert_of"), (offsets, "offsets"), (order, "order"), (tile_expert, "tile_expert"),
+                 (tile_row0, "tile_row0"), (meta, "meta")):
+        _need(t, n, torch.int32)
+        if not t.is_contiguous():
+            raise KernelError(f"group_gather: {n} must be contiguous")
+    _need(expert_of, "expert_of", torch.int32, 2)
+    P, top = expert_of.numel(), expert_of.shape[1]
+    bound = expert_tiles_bound(P, n_experts, tile_rows)
+    if offsets.numel() < n_experts + 1 or order.numel() < P or tile_expert.numel() < bound or tile_row0.numel() < bound:
+        raise KernelError("group_gather: outputs are too small")
+    width = ldx = 8
+    if rows is not None:
+        _need(x, "x", torch.bfloat16, 2); _need(rows, "rows", torch.bfloat16, 2)
+        width, ldx = x.shape[1], x.stride(0)
+        if tuple(rows.shape) != (P, width) or not rows.is_contiguous() or x.shape[0] * top != P or width % 8 or ldx % 8:
+            raise KernelError("group_gather: x [tokens, width], rows [pairs, width], widths and strides multiples of 8")
+    chunk = min(4096, max(1, -(-P // GROUP_BLOCKS)))
+    _check(_fn("expert_ops", "ssb_group_gather")(
+        _ptr(expert_of), c_int(P), c_int(n_experts), c_int(tile_rows), c_int(chunk), _ptr(x if rows is not None else None),
+        c_int(ldx), c_int(top), c_int(width), _ptr(rows), _ptr(offsets), _ptr(order), _ptr(tile_expert), _ptr(tile_row0),
+        _ptr(meta), c_int(1 if pdl else 0), _stream()), "group_gather")
+
+
+def grouped_gemm_tc_ok(hidden: int, inter: int, n_experts: int) -> bool:
+    """Whether the tcgen05 grouped products take an expert layer of these sizes (bfloat16)."""
+    return hidden % 8 == 0 and inter % 8 == 0 and n_experts <= 2048 and n_experts * max(2 * inter, hidden) < 2 ** 31 - 256
+
+
+def grouped_gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, c_index: Optional[torch.Tensor], groups: dict,
+                    mode: int = 0, act=None, pdl: bool = False) -> None:
+    """Grouped products on tcgen05: for sorted row r of expert e, out[c_index[r] or r] = w[e] @ a[r]; ``a`` [pairs, K] sorted,
+    ``w`` [E, N, K], ``groups`` with tiles of 64, 128 or 256 rows.  mode GG_SWIGLU: ``w`` [E, 2N, K] holds gate rows, then
+    up rows, ``act`` = (kind, limit) names the inner step (None: silu(g) u); mode GG_ACT: ``act`` names an activation."""
+    _need(a, "a", torch.bfloat16, 2); _need(w, "w", torch.bfloat16, 3); _need(out, "out", None, 2)
+    E, n_w, K = w.shape
+    N = n_w // 2 if mode == GG_SWIGLU else n_w
+    if mode == GG_ACT:
+        kinds, kind, limit = ACTIVATIONS, act, 0.0
+    else:
+        kinds, (kind, limit) = GATE_KINDS_FF, act if act else ("silu", 0.0)
+    if kind not in kinds:
+        raise KernelError(f"grouped_gemm_tc: {kind!r} is not known (known: {sorted(kinds)})")
+    P = groups["order"].shape[0]
+    if tuple(a.shape) != (P, K) or tuple(out.shape) != (P, N) or not w.is_contiguous() \
+            or (c_index is not None and c_index.numel() < P):
+        raise KernelError(f"grouped_gemm_tc: a{tuple(a.shape)} w{tuple(w.shape)} out{tuple(out.shape)} for {P} pairs")
+    global _tc_unchecked
+    _tc_unchecked += 1
+    _check(_fn("grouped_gemm_tc", "ssb_grouped_gemm_tc")(
+        _ptr(a), c_int(a.stride(0)), _ptr(w), c_int(E), c_int(n_w), _ptr(out), c_int(out.stride(0)), _ptr(c_index),
+        c_int(dtype_code(out.dtype)), _ptr(groups["offsets"]), _ptr(groups["tile_expert"]), _ptr(groups["tile_row0"]),
+        _ptr(groups["meta"]), c_int(groups["max_tiles"]), c_int(groups["tile_rows"]), c_int(P), c_int(N), c_int(K), c_int(mode),
+        c_int(kinds[kind]), c_float(limit), _ptr(tc_error_word(a.device)), c_int(1 if pdl else 0), _stream()), "grouped_gemm_tc")
+
+
 def grouped_gemm_plain(a: torch.Tensor, a_index: Optional[torch.Tensor], a_div: int, w: torch.Tensor,
                        out: torch.Tensor, c_index: Optional[torch.Tensor], offsets: torch.Tensor,
                        tile_expert: torch.Tensor, tile_row0: torch.Tensor, meta: torch.Tensor, max_tiles: int) -> None:

@@ -141,13 +141,14 @@ class SoftmaxRouter:
                                   bias=self.bias)
 
 
-def group_buffers(kernels, n_pairs: int, n_experts: int, device) -> dict:
-    """The int32 buffers that sorting ``n_pairs`` (token, choice) pairs by expert fills and the grouped products read, with
+def group_buffers(kernels, n_tokens: int, top: int, n_experts: int, hidden: int, inter: int, device) -> dict:
+    """The int32 buffers that sorting the step's (token, choice) pairs by expert fills and the grouped products read, with
     the sizes a kernel set asks for."""
-    tile_rows, P, E = kernels.expert_tile_rows, n_pairs, n_experts
+    P, E = n_tokens * top, n_experts
+    tile_rows, sorts_rows = kernels.expert_grouping(n_tokens, top, n_experts, hidden, inter)
     max_tiles = P // tile_rows + min(E, P)
     ints = torch.empty(E + 1 + P + 2 * max_tiles + 1, dtype=torch.int32, device=device)
-    return {"tile_rows": tile_rows, "max_tiles": max_tiles, "offsets": ints[: E + 1], "order": ints[E + 1: E + 1 + P],
+    return {"tile_rows": tile_rows, "sorts_rows": sorts_rows, "max_tiles": max_tiles, "offsets": ints[: E + 1], "order": ints[E + 1: E + 1 + P],
             "tile_expert": ints[E + 1 + P: E + 1 + P + max_tiles],
             "tile_row0": ints[E + 1 + P + max_tiles: E + 1 + P + 2 * max_tiles], "meta": ints[-1:]}
 
@@ -209,11 +210,11 @@ class Experts:
 
     @staticmethod
     def activation_elements(params) -> int:
-        """Elements per token while the part runs: per choice gate, up, their product (without a gate the inner row alone)
-        and the expert's output (float32: counted twice); the shared expert's rows."""
+        """Elements per token while the part runs: per choice gate, up, their product (without a gate the inner row alone),
+        the token's row in sorted order and the expert's output (float32: counted twice); the shared expert's rows."""
         inner = 3 if params.get("gated", True) else 1
         shared = 3 * int(params["shared"]["intermediate_size"]) if params.get("shared") else 0
-        return int(params["top"]) * (inner * int(params["expert_size"]) + 2 * int(params["hidden_size"])) + shared
+        return int(params["top"]) * (inner * int(params["expert_size"]) + 3 * int(params["hidden_size"])) + shared
 
     @property
     def sums_choices(self) -> bool:
@@ -244,8 +245,8 @@ class Experts:
             self.router.route(ctx, xt, expert_of, pair_weight, extra_out=shared_scale)
         else:
             self.router.route(ctx, xt, expert_of, pair_weight)
-        groups = group_buffers(ctx.kernels, P, self.E, dev)
-        ctx.kernels.group_by_expert(expert_of, self.E, groups)
+        groups = group_buffers(ctx.kernels, T, top, self.E, self.hidden, self.inter, dev)
+        ctx.kernels.group_by_expert(expert_of, self.E, groups, xt)
         z = torch.empty((P, self.inter), dtype=self.dtype, device=dev)
         if not self.gated:
             ctx.kernels.expert_up(xt, top, self.w_first, z, groups, self.act)

@@ -255,8 +255,8 @@ def test_expert_products_with_the_activation_inside(dtype, rows, experts, top, h
     chosen = torch.stack([torch.cat([torch.zeros(1, dtype=torch.long), 1 + torch.randperm(pool - 1, generator=g)[: top - 1]])
                           if top > 1 else torch.zeros(1, dtype=torch.long) for _ in range(rows)]).int()
     chosen = chosen[:, torch.randperm(top, generator=g)].contiguous()
-    groups = group_buffers(k, rows * top, experts, DEV)
-    k.group_by_expert(chosen.to(DEV), experts, groups)
+    groups = group_buffers(k, rows, top, experts, hidden, inter, DEV)
+    k.group_by_expert(chosen.to(DEV), experts, groups, x.to(DEV))
     z = torch.empty(rows * top, inter, dtype=dtype, device=DEV)
     k.expert_up(x.to(DEV), top, w.to(DEV), z, groups, "relu_squared")
     y = torch.full((rows * top, hidden), float("nan"), dtype=torch.float32, device=DEV)
@@ -275,6 +275,46 @@ def test_expert_products_with_the_activation_inside(dtype, rows, experts, top, h
         out[at] = ref[at].to(dtype).double() @ down[i].double().T
     assert float((z.cpu().double() - ref[order]).abs().max()) < (1e-5 if dtype == torch.float32 else 0.01) * float(ref.abs().max())
     assert float((y.cpu().double() - out).abs().max()) < (1e-5 if dtype == torch.float32 else 0.01) * float(out.abs().max())
+
+
+@pytest.mark.parametrize("act", [None, ("clamped_swish", 0.75), ("gelu_tanh", 0.0)])
+@pytest.mark.parametrize("tile_rows", [64, 128, 256])
+def test_gated_expert_products_on_tcgen05(tile_rows, act):
+    """Gate and up rows of an expert met inside the product, for every tile height: groups of one row, of whole tiles, of one
+    row more and of none; widths that are not whole column tiles, an inner size that is not whole k-blocks."""
+    from supersonic_b200.csrc import ops
+    g = torch.Generator().manual_seed(tile_rows)
+    sizes = [1, tile_rows, 0, tile_rows + 1, 3 * tile_rows - 5, 16, 17]
+    E, P, K, I = len(sizes), sum(sizes), 136, 88
+    expert_of = torch.cat([torch.full((n,), e, dtype=torch.int32) for e, n in enumerate(sizes)])[torch.randperm(P, generator=g)]
+    x = (torch.randn(P, K, generator=g) * 1.5).bfloat16()
+    w = (torch.randn(E, 2 * I, K, generator=g) * 0.15).bfloat16()
+    mt = ops.expert_tiles_bound(P, E, tile_rows)
+    groups = {k: torch.full((n,), -7, dtype=torch.int32, device=DEV) for k, n in
+              (("offsets", E + 1), ("order", P), ("tile_expert", mt), ("tile_row0", mt), ("meta", 1))}
+    rows = torch.empty(P, K, dtype=torch.bfloat16, device=DEV)
+    ops.group_gather(expert_of.view(P, 1).to(DEV), E, tile_rows, groups["offsets"], groups["order"], groups["tile_expert"],
+                     groups["tile_row0"], groups["meta"], x.to(DEV), rows)
+    order = torch.sort(expert_of, stable=True).indices
+    assert torch.equal(groups["order"].cpu().long(), order) and torch.equal(rows.cpu(), x[order])
+    assert groups["offsets"].tolist() == [sum(sizes[:i]) for i in range(E + 1)]
+    tiles = [(e, sum(sizes[:e]) + r) for e, n in enumerate(sizes) for r in range(0, n, tile_rows)]
+    assert int(groups["meta"]) == len(tiles)
+    assert list(zip(groups["tile_expert"].tolist(), groups["tile_row0"].tolist()))[: len(tiles)] == tiles
+    groups.update(max_tiles=mt, tile_rows=tile_rows)
+    out = torch.full((P, I), float("nan"), dtype=torch.bfloat16, device=DEV)
+    ops.grouped_gemm_tc(rows, w.to(DEV), out, None, groups, ops.GG_SWIGLU, act)
+    ops.check_device_errors()
+    kind, limit = act or ("silu", 0.0)
+    for i, p in enumerate(order.tolist()):
+        h = w[expert_of[p]].double() @ x[p].double()
+        gate, up = h[:I], h[I:]
+        if kind == "clamped_swish":
+            gate, up = gate.clamp(max=limit), up.clamp(-limit, limit) + 1.0
+            gate = gate * pr.sigmoid(1.702 * gate)
+        else:
+            gate = pr.gelu(gate) if kind == "gelu_tanh" else gate * pr.sigmoid(gate)
+        assert float((out[i].cpu().double() - gate * up).abs().max()) < 0.02 * max(1.0, float((gate * up).abs().max())), (i, p)
 
 
 @pytest.mark.parametrize("experts,top", [(1, 1), (2, 1), (12, 3), (70, 5), (33, 33)])
