@@ -361,7 +361,9 @@ class FastKernels(PlainKernels):
     LATENT_SPLIT_BLOCKS = 148
 
     def head_linear(self, x, w, out, gate=None):
-        if ops.head_gemm_mma_ok(x, w, out):
+        if self.head_tc and not self.deterministic and ops.head_gemm_tc_ok(x, w, out):
+            ops.head_gemm_tc(x, w, out, pdl=self._chain(x.shape[0]), gate=gate)
+        elif ops.head_gemm_mma_ok(x, w, out):
             ops.head_gemm_mma(x, w, out, pdl=self.pdl, gate=gate)
         else:
             super().head_linear(x, w, out, gate)
@@ -459,18 +461,25 @@ class FastKernels(PlainKernels):
 
     def route_softmax(self, x, weight, n_experts, renormalize, scale, expert_of, pair_weight, bias=None):
         rows, n = x.shape[0], weight.shape[0]
-        if rows > STREAM_ROWS or self.deterministic:
+        tile_n = 64 if n <= 64 else self._tile_n(rows, n)
+        splits = ops.gemv_tc_splits(n, weight.shape[1]) if rows <= STREAM_ROWS else self._gemm_splits(rows, n, weight.shape[1], tile_n)
+        if self.deterministic or (rows > STREAM_ROWS and splits == 1):
             super().route_softmax(x, weight, n_experts, renormalize, scale, expert_of, pair_weight, bias)
             return
-        # a few rows: K is split over blocks that add into sums which are zero between uses (the choice clears its rows)
+        # fewer output tiles than SMs: K is split over blocks that add into sums which are zero between uses (the choice
+        # clears its rows); 2,048 rows of 2,048 columns and 64 experts: 28 us with the product in one part, 20 so
         logits = self._buffer("router_sums", rows * n, torch.float32, x.device, zero=True)[: rows * n].view(rows, n)
         if not ops.gemm_tc_ok(x, weight, logits):
             super().route_softmax(x, weight, n_experts, renormalize, scale, expert_of, pair_weight, bias)
             return
-        ops.gemv_tc(x, weight, logits, ops.TC_ACCUMULATE, splits=ops.gemv_tc_splits(n, weight.shape[1]), pdl=self.pdl)
+        if rows <= STREAM_ROWS:
+            ops.gemv_tc(x, weight, logits, ops.TC_ACCUMULATE, splits=splits, pdl=self.pdl)
+        else:
+            ops.gemm_tc(x, weight, logits, ops.TC_ACCUMULATE, tile_n=tile_n, splits=splits)
         ops.route_softmax(logits, n_experts, renormalize, scale, expert_of, pair_weight, clear=True, pdl=self._chain(rows),
                           bias=bias)
 
+    head_tc = True           # prompts' per-head products on tcgen05
     grouped_tc = True        # the experts' products on tcgen05, where their sizes are whole 16-byte pieces
 
     def expert_grouping(self, n_tokens, top, n_experts, hidden, inter):

@@ -484,6 +484,33 @@ def head_gemm_mma(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, pdl: bool
         "head_gemm_mma")
 
 
+HEAD_GEMM_TC_MIN_ROWS = 129      # tokens from which the per-head products run on tcgen05
+
+
+def head_gemm_tc_ok(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> bool:
+    return head_gemm_mma_ok(x, w, out) and x.shape[0] >= HEAD_GEMM_TC_MIN_ROWS and w.shape[0] * w.shape[1] < 2 ** 31 - 256
+
+
+def head_gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, pdl: bool = False,
+                 gate: Optional[torch.Tensor] = None) -> None:
+    """``head_gemm_mma`` on tcgen05, for prompts."""
+    T, H, K = x.shape
+    N = w.shape[1]
+    if not head_gemm_tc_ok(x, w, out) or tuple(w.shape) != (H, N, K) or tuple(out.shape) != (T, H, N):
+        raise KernelError(f"head_gemm_tc: x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
+    if gate is not None:
+        _need(gate, "gate", torch.bfloat16, 2)
+        if tuple(gate.shape) != (T, H * N):
+            raise KernelError("head_gemm_tc: one gate per element of the concatenated heads")
+    global _tc_unchecked
+    _tc_unchecked += 1
+    _check(_fn("grouped_gemm_tc", "ssb_head_gemm_tc")(
+        _ptr(x), c_int(x.stride(0)), c_int((H - 1) * x.stride(1) + K), c_int(x.stride(1) if H > 1 else 0), _ptr(w), _ptr(out),
+        c_int(out.stride(0)), c_int(out.stride(1)), c_int(dtype_code(out.dtype)), c_int(H), c_int(T), c_int(N), c_int(K),
+        _ptr(gate), c_int(gate.stride(0) if gate is not None else 0), _ptr(tc_error_word(x.device)), c_int(1 if pdl else 0),
+        _stream()), "head_gemm_tc")
+
+
 GG_STORE, GG_SWIGLU, GG_ACT = 0, 1, 2
 
 

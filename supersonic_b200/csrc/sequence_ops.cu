@@ -302,9 +302,10 @@ causal_conv_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ x
 constexpr int CV_TILE = 8;
 constexpr int CV_THREADS = 128;
 
-template <int TAPS>
+template <int TAPS, bool BIAS>
 __global__ void __launch_bounds__(CV_THREADS)
-causal_conv_vec_kernel(const bf16* __restrict__ x, int ldx, const float* __restrict__ w, float* __restrict__ tail,
+causal_conv_vec_kernel(const bf16* __restrict__ x, int ldx, const float* __restrict__ x_bias, const float* __restrict__ w,
+                       const float* __restrict__ bias, float* __restrict__ tail,
                        const int* __restrict__ cu_new, const int* __restrict__ seq_slot, bf16* __restrict__ u, int ldu,
                        int channels, int pass_cols) {
     constexpr int BACK = TAPS - 1;
@@ -341,9 +342,16 @@ causal_conv_vec_kernel(const bf16* __restrict__ x, int ldx, const float* __restr
         wj[(e + 3) / TAPS][(e + 3) % TAPS] = v.w;
     }
     float* keep = tail + (size_t)slot * BACK * channels + c;
-    auto value = [](const uint4& r, int k) {
+    float xb[8], cb[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+        xb[k] = BIAS && x_bias ? x_bias[c + k] : 0.f;
+        cb[k] = BIAS && bias ? bias[c + k] : 0.f;
+    }
+    auto value = [&](const uint4& r, int k) {
         const uint32_t q = k < 2 ? r.x : k < 4 ? r.y : k < 6 ? r.z : r.w;
-        return __uint_as_float((k & 1) ? (q & 0xffff0000u) : (q << 16));
+        const float v = __uint_as_float((k & 1) ? (q & 0xffff0000u) : (q << 16));
+        return BIAS ? v + xb[k] : v;
     };
     // inputs before the tile: rows of this step, or, in the sequence's first tile, its kept rows
     float win[BACK][8];
@@ -387,7 +395,7 @@ causal_conv_vec_kernel(const bf16* __restrict__ x, int ldx, const float* __restr
         float v[8];
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
-            float acc = 0.f;
+            float acc = BIAS ? cb[k] : 0.f;
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) {
                 const int r = i + j - BACK;                // row of the tile that tap j sees
@@ -411,12 +419,15 @@ SSB_API int ssb_causal_conv(const void* x, int ldx, int dtype, const float* x_bi
                             int max_new, int channels, int taps, int pass_cols, int pdl, cudaStream_t stream) {
     if (n_seqs <= 0 || max_new <= 0) return 0;
     if (channels <= 0 || taps < 1 || taps > CONV_MAX_TAPS || pass_cols < 0) return SSB_ERR_BAD_SIZE;
-    if (dtype == SSB_BF16 && x_bias == nullptr && bias == nullptr && taps >= 2 && taps <= 4 && channels % 8 == 0 &&
+    if (dtype == SSB_BF16 && taps >= 2 && taps <= 4 && channels % 8 == 0 &&
         pass_cols % 8 == 0 && ldx % 8 == 0 && ldu % 8 == 0 && (((uintptr_t)x | (uintptr_t)u | (uintptr_t)w | (uintptr_t)tail) & 15) == 0 && x != u) {
         const dim3 vgrid(n_seqs, (max_new + CV_TILE - 1) / CV_TILE, ((channels + pass_cols) / 8 + CV_THREADS - 1) / CV_THREADS);
         if (vgrid.y <= 65535 && vgrid.z <= 65535) {
-            auto kern = taps == 2 ? causal_conv_vec_kernel<2> : taps == 3 ? causal_conv_vec_kernel<3> : causal_conv_vec_kernel<4>;
-            const int rcv = ssb_launch(kern, vgrid, dim3(CV_THREADS), 0, stream, pdl != 0, (const bf16*)x, ldx, w, tail, cu_new,
+            const bool biased = x_bias != nullptr || bias != nullptr;
+            auto kern = taps == 2 ? (biased ? causal_conv_vec_kernel<2, true> : causal_conv_vec_kernel<2, false>)
+                      : taps == 3 ? (biased ? causal_conv_vec_kernel<3, true> : causal_conv_vec_kernel<3, false>)
+                                  : (biased ? causal_conv_vec_kernel<4, true> : causal_conv_vec_kernel<4, false>);
+            const int rcv = ssb_launch(kern, vgrid, dim3(CV_THREADS), 0, stream, pdl != 0, (const bf16*)x, ldx, x_bias, w, bias, tail, cu_new,
                                        seq_slot, (bf16*)u, ldu, channels, pass_cols);
             return rcv ? rcv : ssb_launch_status();
         }

@@ -55,7 +55,7 @@ class TimedKernels:
 
     def __getattr__(self, name):
         attr = getattr(self._inner, name)
-        if name.startswith("_") or not callable(attr) or name == "pack_gate_up":
+        if name.startswith("_") or not callable(attr) or name in ("pack_gate_up", "expert_grouping"):
             return attr
 
         def timed(*args, **kwargs):

@@ -371,9 +371,11 @@ def test_joining_the_stream(dtype, width, top):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("T,H,K,N", [(5, 3, 24, 16), (70, 4, 128, 64), (300, 5, 80, 48), (33, 2, 20, 9)])
+@pytest.mark.parametrize("T,H,K,N", [(5, 3, 24, 16), (70, 4, 128, 64), (300, 5, 80, 48), (33, 2, 20, 9), (129, 1, 64, 200),
+                                     (1000, 3, 128, 256), (257, 16, 72, 33)])
 def test_per_head_products_with_a_gate_inside(dtype, T, H, K, N):
-    """out[t, h] = (W_h x[t, h]) * sigmoid(gate): inside the product where it takes the sizes, else behind it."""
+    """out[t, h] = (W_h x[t, h]) * sigmoid(gate): inside the product where it takes the sizes, else behind it; without a gate
+    from and into parts of wider heads."""
     from supersonic_b200.csrc.kernel_sets import kernel_set_for
     g = torch.Generator().manual_seed(T)
     x, w = torch.randn(T, H, K, generator=g).to(dtype), (torch.randn(H, N, K, generator=g) * K ** -0.5).to(dtype)
@@ -382,6 +384,14 @@ def test_per_head_products_with_a_gate_inside(dtype, T, H, K, N):
     kernel_set_for(dtype).head_linear(x.to(DEV), w.to(DEV), out, gate=rows[:, 3:])
     ref = torch.einsum("thk,hnk->thn", x.double(), w.double()) * pr.sigmoid(rows[:, 3:].cpu().double()).view(T, H, N)
     assert float((out.cpu().double() - ref).abs().max()) < (1e-5 if dtype == torch.float32 else 0.02) * max(1.0, float(ref.abs().max()))
+    wide_x, wide_out = torch.full((T, H, K + 8), 9.0, dtype=dtype, device=DEV), torch.full((T, H, N + 5), 7.0, device=DEV)
+    wide_x[:, :, :K] = x.to(DEV)
+    kernel_set_for(dtype).head_linear(wide_x[:, :, :K], w.to(DEV), wide_out[:, :, :N])
+    ref = torch.einsum("thk,hnk->thn", x.double(), w.double())
+    assert float((wide_out[:, :, :N].cpu().double() - ref).abs().max()) < (1e-5 if dtype == torch.float32 else 1e-4) * max(1.0, float(ref.abs().max()))
+    assert bool((wide_out[:, :, N:] == 7.0).all())
+    from supersonic_b200.csrc import ops
+    ops.check_device_errors()
 
 
 @pytest.mark.parametrize("heads,rank,rot,window", [(4, 128, 32, 100), (5, 80, 16, 33), (16, 512, 64, 64), (1, 16, 16, 1), (8, 256, 32, 65),
